@@ -373,20 +373,25 @@ def gemm_heads(a, w, out):
     return out
 
 
-def moe_route(x, w_router, correction, w_shared_gate, groups, keep, top, weight_eps=1e-20, scores="sigmoid"):
+def moe_route(x, w_router, correction, w_shared_gate, groups, keep, top, weight_eps=1e-20, scores="sigmoid",
+              group_score="two_best", renorm=True):
     xf = x.to(torch.float32)
-    s = xf @ w_router.t() if scores == "softmax_chosen" else torch.sigmoid(xf @ w_router.t())
+    z = xf @ w_router.t()
+    s = {"softmax_chosen": lambda: z, "sigmoid": lambda: torch.sigmoid(z), "softmax": lambda: torch.softmax(z, dim=-1)}[scores]()
     n, experts = s.shape
     pick = s + correction if correction is not None else s.clone()
     if groups:
         per = pick.view(n, groups, experts // groups)
-        strength = per.topk(min(2, experts // groups), dim=-1).values.sum(-1)
+        strength = per.topk(1 if group_score == "best" else min(2, experts // groups), dim=-1).values.sum(-1)
         best = strength.topk(keep, dim=-1).indices
         ok = torch.zeros((n, groups), dtype=torch.bool).scatter_(1, best, True)
         pick = per.masked_fill(~ok[:, :, None], float("-inf")).reshape(n, experts)
     chosen = pick.topk(top, dim=-1).indices
     w = s.gather(1, chosen)
-    w = torch.softmax(w, dim=-1) if scores == "softmax_chosen" else w / (w.sum(-1, keepdim=True) + weight_eps)
+    if scores == "softmax_chosen":
+        w = torch.softmax(w, dim=-1)
+    elif renorm:
+        w = w / (w.sum(-1, keepdim=True) + weight_eps)
     shared = torch.sigmoid(xf @ w_shared_gate) if w_shared_gate is not None else None
     return chosen.to(torch.int32), w, shared
 
@@ -399,7 +404,15 @@ def _act(z, kind):
     return z * torch.sigmoid(z)
 
 
-def moe_gate_up(x, chosen, w_gate_up, act=None):
+def gated(g, u, form=None):
+    """A gated unit in the form ``kernels.ops.GateForm`` (silu unless given), from its definition."""
+    if form is None:
+        return g * torch.sigmoid(g) * u
+    g = torch.clamp(g, max=form.limit)
+    return g * torch.sigmoid(g * (form.c1 + form.c3 * g * g)) * (torch.clamp(u, min=-form.limit, max=form.limit) + form.shift)
+
+
+def moe_gate_up(x, chosen, w_gate_up, act=None, form=None):
     n, top = chosen.shape
     xf = x.to(torch.float32)
     if act is not None:
@@ -408,11 +421,11 @@ def moe_gate_up(x, chosen, w_gate_up, act=None):
     w = w_gate_up.to(torch.float32)[chosen.long()]                      # (n, top, 2, F, d)
     g = torch.einsum("ntfd,nd->ntf", w[:, :, 0], xf)
     u = torch.einsum("ntfd,nd->ntf", w[:, :, 1], xf)
-    return (g * torch.sigmoid(g) * u).reshape(n * top, -1).to(x.dtype)
+    return gated(g, u, form).reshape(n * top, -1).to(x.dtype)
 
 
-def moe_experts(x, chosen, weights, w_gate_up, w_down, shared, shared_gate, act=None):
-    return moe_down(moe_gate_up(x, chosen, w_gate_up, act), chosen, weights, w_down, shared, shared_gate)
+def moe_experts(x, chosen, weights, w_gate_up, w_down, shared, shared_gate, act=None, form=None):
+    return moe_down(moe_gate_up(x, chosen, w_gate_up, act, form), chosen, weights, w_down, shared, shared_gate)
 
 
 def gated_linear_attention(qkv, a_in, power, a_bias, gate, norm_weight, eps, q_scale, state, out, row_slot, row_last,
@@ -522,6 +535,44 @@ def rotate_tie_store(qk, num_heads, kv_heads, dim, rot, cos, sin, k_pages, v_pag
         v_pages[page, :, pos % page_size, :] = k.to(v_pages.dtype)
 
 
+def add_layer_norm(residual, delta_a, delta_b, w, b, eps, out):
+    for delta in (delta_a, delta_b):
+        if delta is not None:
+            residual += delta.to(torch.float32)
+    mean = residual.mean(-1, keepdim=True)
+    var = (residual - mean).pow(2).mean(-1, keepdim=True)
+    out.copy_(((residual - mean) / torch.sqrt(var + eps) * w + b).to(out.dtype))
+    return out
+
+
+def rotate_norm_store(qkv, num_heads, kv_heads, dim, v_dim, cos, sin, interleaved, norm, eps, k_pages, v_pages, block_table,
+                      positions, row_slot, page_size, fault):
+    def prepared(z, pos):               # (heads, dim)
+        out = z.to(torch.float32).clone()
+        if cos is not None:
+            half = cos.shape[1]
+            ia = torch.arange(half) * 2 if interleaved else torch.arange(half)
+            ib = ia + 1 if interleaved else ia + half
+            a, b = out[:, ia].clone(), out[:, ib].clone()
+            out[:, ia] = a * cos[pos] - b * sin[pos]
+            out[:, ib] = b * cos[pos] + a * sin[pos]
+        if norm:
+            out = out / torch.sqrt(out.pow(2).mean(-1, keepdim=True) + eps)
+        return out
+
+    H, G = num_heads, kv_heads
+    for r in range(qkv.shape[0]):
+        slot, pos = int(row_slot[r]), int(positions[r])
+        if slot < 0:
+            continue
+        qk = prepared(qkv[r, :(H + G) * dim].view(H + G, dim), pos).to(qkv.dtype)
+        qkv[r, :H * dim] = qk[:H].reshape(-1)
+        if G:
+            page, at = int(block_table[slot, pos // page_size]), pos % page_size
+            k_pages[page, :, at] = qk[H:].to(k_pages.dtype)
+            v_pages[page, :, at] = qkv[r, (H + G) * dim:(H + G) * dim + G * v_dim].view(G, v_dim).to(v_pages.dtype)
+
+
 def scaled_sum(a, scale_a, b, scale_b):
     return (a.to(torch.float32) * scale_a + b.to(torch.float32) * scale_b).to(a.dtype)
 
@@ -532,7 +583,7 @@ def moe_down(hidden, chosen, weights, w_down, shared, shared_gate):
     y = torch.einsum("ntdf,ntf->ntd", w_down.to(torch.float32)[chosen.long()], h)
     out = (y * weights[:, :, None]).sum(1)
     if shared is not None:
-        out = out + shared_gate[:, None] * shared.to(torch.float32)
+        out = out + (shared_gate[:, None] if shared_gate is not None else 1.0) * shared.to(torch.float32)
     return out.to(hidden.dtype)
 
 
@@ -660,19 +711,19 @@ def paged_attention(q, out, plane, block_table, positions, row_slot, num_heads, 
     return out
 
 
-def swiglu(gu, out, block=None):
+def swiglu(gu, out, block=None, form=None):
     f = out.shape[1]
     block = block or f
     both = gu.to(torch.float32).reshape(gu.shape[0], f // block, 2, block)
     g = both[:, :, 0, :].reshape(-1, f)
     u = both[:, :, 1, :].reshape(-1, f)
-    out.copy_((g / (1 + torch.exp(-g)) * u).to(out.dtype))
+    out.copy_(gated(g, u, form).to(out.dtype))
     return out
 
 
-def gemm_swiglu(a, w_gu, hidden, block):
+def gemm_swiglu(a, w_gu, hidden, block, form=None):
     gu = gemm(a, w_gu)
-    return swiglu(gu, torch.empty((a.shape[0], hidden), dtype=a.dtype), block)
+    return swiglu(gu, torch.empty((a.shape[0], hidden), dtype=a.dtype), block, form)
 
 
 def mtp_input(h_prev, state, row_slot, row_last, tokens, table, scale, eps, out):
@@ -781,7 +832,8 @@ _NAMES = ["rotary_fusable", "gemm", "gemm_f32_out", "gemm_swiglu", "embed_rows",
           "softcap_f32", "activation", "gemm_act", "forget_gate_recurrence", "head_norm_store", "diff_combine",
           "norm_mix_store", "window_attention", "delta_rule", "linear_attention", "latent_prepare", "gemm_heads", "moe_route",
           "moe_gate_up", "moe_down", "moe_experts", "gated_linear_attention", "state_space_scan", "skip_gate_group_norm",
-          "embed_pairs", "group_norm", "rotate_tie_store", "scaled_sum"]
+          "embed_pairs", "group_norm", "rotate_tie_store", "scaled_sum", "add_layer_norm",
+          "rotate_norm_store"]
 
 
 def install(monkeypatch) -> None:

@@ -347,6 +347,10 @@ def _positive_int(v) -> bool:
     return isinstance(v, int) and not isinstance(v, bool) and v > 0
 
 
+def _number(v) -> bool:
+    return isinstance(v, (int, float)) and not isinstance(v, bool)
+
+
 @dataclass
 class MizidraConfig:
     """Configuration of the Mizidra decoder: a normed embedding, pre-norm layers whose mixer is one of three kinds
@@ -811,6 +815,158 @@ class KubolornConfig:
             d["canon"] = {"taps": self.canon_taps}
         if self.loop is not None:
             d["loop"] = dict(self.loop)
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+
+@dataclass
+class LomutarConfig:
+    """Configuration of the Lomutar decoder: layers with one layer norm whose output the attention and the feed-forward both
+    read, an output matrix of its own.
+
+    ``config.json`` is nested: ``vocab``, ``width``, ``norm.eps`` and ``layers``, a list with, per layer, ``type``
+    (``attention``), ``mixer`` and ``mlp`` (null: none).
+
+    * ``mixer`` — ``heads, kv_heads, dim, vdim, scale``, ``rot`` = ``base, dims`` and optionally ``scaling.factor`` (divides every
+      frequency), ``mask.size`` (the keys a token sees, itself among them; no ``mask``: all earlier ones) and ``kv_from`` (an
+      earlier layer with keys and values of the same heads and widths, which this layer reads instead of making its own);
+    * ``mlp`` — ``kind`` ``dense`` with ``ff``, or ``moe`` with ``expert`` = ``ff, limit``, ``router`` = ``experts, top`` and
+      optionally ``groups`` = ``count, keep``, and optionally ``shared`` = ``ff, limit``.
+
+    The design has no context limit of its own: ``max_context`` (optional) bounds what the engine lays out (block tables,
+    rotation tables)."""
+
+    architecture: ClassVar[str] = "Lomutar"
+    MIXERS: ClassVar[tuple] = ("attention",)
+
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float = 1e-5
+    max_context: int = 1 << 16
+    eos_token_id: Optional[int] = None
+    torch_dtype: str = "bfloat16"
+
+    def __post_init__(self):
+        errs = []
+        for name in ("vocab_size", "hidden_size", "max_context"):
+            if not _positive_int(getattr(self, name)):
+                errs.append(f"{name} must be a positive integer, got {getattr(self, name)!r}")
+        if not isinstance(self.layers, list) or not self.layers:
+            errs.append("layers must be a non-empty list")
+            raise ConfigError("; ".join(errs))
+        if not (self.norm_eps >= 0):
+            errs.append(f"norm.eps must be >= 0, got {self.norm_eps}")
+        for i, layer in enumerate(self.layers):
+            kind = layer.get("type") if isinstance(layer, dict) else None
+            if kind not in self.MIXERS:
+                errs.append(f"layers[{i}].type must be one of {self.MIXERS}, got {kind!r}")
+            elif not isinstance(layer.get("mixer"), dict):
+                errs.append(f"layers[{i}].mixer is missing")
+            else:
+                errs += self._mixer_errors(i, layer["mixer"])
+                if layer.get("mlp") is not None:
+                    errs += self._mlp_errors(i, layer["mlp"])
+        if self.torch_dtype not in ("bfloat16", "float32"):
+            errs.append(f"torch_dtype must be bfloat16 or float32, got {self.torch_dtype!r}")
+        if errs:
+            raise ConfigError("; ".join(errs))
+
+    def _mixer_errors(self, i: int, m: dict) -> list:
+        at, errs = f"layers[{i}].mixer", []
+        bad = [k for k in ("heads", "kv_heads", "dim", "vdim") if not _positive_int(m.get(k))]
+        if bad:
+            return [f"{at}: {', '.join(bad)} must be positive integers"]
+        if m["heads"] % m["kv_heads"]:
+            errs.append(f"{at}: {m['heads']} heads are not a multiple of {m['kv_heads']} kv heads")
+        if not _number(m.get("scale")):
+            errs.append(f"{at}.scale is missing")
+        mask = m.get("mask")
+        if mask is not None and not (isinstance(mask, dict) and _positive_int(mask.get("size"))):
+            errs.append(f"{at}.mask.size must be a positive integer")
+        rot = m.get("rot")
+        if rot is not None:
+            if not isinstance(rot, dict) or not _number(rot.get("base")) or not rot["base"] > 0:
+                errs.append(f"{at}.rot.base is missing")
+            elif not _positive_int(rot.setdefault("dims", m["dim"])) or rot["dims"] % 2 or rot["dims"] > m["dim"]:
+                errs.append(f"{at}: rot.dims must be even and at most dim ({m['dim']})")
+            elif rot.get("scaling") and not (_number(rot["scaling"].get("factor")) and rot["scaling"]["factor"] > 0):
+                errs.append(f"{at}.rot.scaling.factor must be a positive number")
+        j = m.get("kv_from")
+        if j is not None:
+            if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < i:
+                errs.append(f"{at}.kv_from must name an earlier layer, got {j!r}")
+            else:
+                src = self.layers[j].get("mixer") if isinstance(self.layers[j], dict) else None
+                if not isinstance(src, dict) or src.get("kv_from") is not None:
+                    errs.append(f"{at}.kv_from: layer {j} has no keys and values of its own")
+                elif any(src.get(k) != m[k] for k in ("kv_heads", "dim", "vdim")):
+                    errs.append(f"{at}.kv_from: kv_heads, dim and vdim of layer {j} differ from this layer's")
+        return errs
+
+    @staticmethod
+    def _mlp_errors(i: int, f: dict) -> list:
+        at, errs = f"layers[{i}].mlp", []
+        if not isinstance(f, dict) or f.get("kind") not in ("dense", "moe"):
+            return [f"{at}.kind must be 'dense' or 'moe', got {f.get('kind') if isinstance(f, dict) else f!r}"]
+        if f["kind"] == "dense":
+            return [] if _positive_int(f.get("ff")) else [f"{at}.ff must be a positive integer"]
+        for key in ("expert", "shared"):
+            u = f.get(key)
+            if u is None and key == "shared":
+                continue
+            if not isinstance(u, dict) or not _positive_int(u.get("ff")):
+                errs.append(f"{at}.{key}.ff must be a positive integer")
+            elif not _number(u.get("limit")) or not u["limit"] > 0:
+                errs.append(f"{at}.{key}.limit must be a positive number")
+        r = f.get("router")
+        if not isinstance(r, dict) or not _positive_int(r.get("experts")) or not _positive_int(r.get("top")):
+            return errs + [f"{at}.router needs experts and top"]
+        allowed, g = r["experts"], r.get("groups")
+        if g:
+            if not _positive_int(g.get("count")) or not _positive_int(g.get("keep")) or r["experts"] % g["count"] \
+                    or g["keep"] > g["count"]:
+                return errs + [f"{at}.router.groups: count must divide the experts and keep <= count"]
+            allowed = r["experts"] // g["count"] * g["keep"]
+        if r["top"] > allowed:
+            errs.append(f"{at}.router.top {r['top']} exceeds the {allowed} experts that can be chosen")
+        return errs
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def window_of(self, i: int) -> Optional[int]:
+        """The keys a token of layer i sees (None: all earlier ones)."""
+        mask = self.layers[i]["mixer"].get("mask")
+        return mask["size"] if mask else None
+
+    def cache_window(self, i: int) -> Optional[int]:
+        """The keys that the plane which layer i uses must keep: as many as the widest window of its owner and of all layers
+        that read it (None: all)."""
+        owner = self.layers[i]["mixer"].get("kv_from")
+        owner = i if owner is None else owner
+        users = [self.window_of(j) for j, layer in enumerate(self.layers) if j == owner or layer["mixer"].get("kv_from") == owner]
+        return None if any(w is None for w in users) else max(users)
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "LomutarConfig":
+        missing = [k for k in ("vocab", "width", "layers") if k not in raw]
+        if missing:
+            raise ConfigError(f"config for architecture {cls.architecture!r}: missing keys: " + ", ".join(missing))
+        d = dict(vocab_size=raw["vocab"], hidden_size=raw["width"], layers=copy.deepcopy(raw["layers"]))
+        if isinstance(raw.get("norm"), dict) and "eps" in raw["norm"]:
+            d["norm_eps"] = float(raw["norm"]["eps"])
+        for k in ("max_context", "eos_token_id", "torch_dtype"):
+            if k in raw:
+                d[k] = raw[k]
+        return cls(**d)
+
+    def to_dict(self) -> dict:
+        d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+             "norm": {"eps": self.norm_eps}, "layers": copy.deepcopy(self.layers), "max_context": self.max_context,
+             "torch_dtype": self.torch_dtype}
         if self.eos_token_id is not None:
             d["eos_token_id"] = self.eos_token_id
         return d

@@ -33,6 +33,7 @@ struct Epilogue {
     bf16* out; int ldo;
     int M, N;
     int epi;
+    GateForm gate;           // EPI_SWIGLU: the form of the gating
     // rows that still lack their norm's factor: partial sums of squares [M][in_parts] (null: none)
     const float* in_ss; int in_parts; NormFactor in_factor;
     // EPI_RESIDUAL: the stream [M][ldr] (read and written), the next norm's weight [N], partial sums out [M][strips]
@@ -217,12 +218,12 @@ __device__ __forceinline__ void push_reduce_store(const float (&acc)[MT][2][4], 
             if (valid && strip * STRIP + col < e.N)
                 e.out[(size_t)row * e.ldo + strip * STRIP + col] = __float2bfloat16_rn(epilogue_act(sum, e.epi));
         } else {
-            // the strip is [32 gate | 32 up]: out column strip*32 + j = silu(gate_j) * up_j
+            // the strip is [32 gate | 32 up]: out column strip*32 + j = gated(gate_j, up_j)
             pair[half][col] = sum;
             asm volatile("bar.sync 1, 128;\n" ::: "memory");
             if (valid && col < 32) {
                 const float gt = pair[half][col], up = pair[half][col + 32];
-                e.out[(size_t)row * e.ldo + strip * 32 + col] = __float2bfloat16_rn(gt / (1.f + expf(-gt)) * up);
+                e.out[(size_t)row * e.ldo + strip * 32 + col] = __float2bfloat16_rn(gated_unit(gt, up, e.gate));
             }
             asm volatile("bar.sync 1, 128;\n" ::: "memory");
         }

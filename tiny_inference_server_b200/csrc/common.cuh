@@ -6,6 +6,7 @@
 #include <cuda_runtime.h>
 #include <cuda_bf16.h>
 #include <stdint.h>
+#include <math.h>
 
 #define TIS_API extern "C" __attribute__((visibility("default")))
 
@@ -100,6 +101,25 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
+}
+
+// ---- gated units -----------------------------------------------------------------------------
+// What a gated feed-forward does with a gate g and an up value u:
+//   g' = min(g, limit), u' = min(max(u, -limit), limit), out = g' * sigmoid(g' * (c1 + c3 * g'^2)) * (u' + shift).
+// limit = inf, c1 = 1, c3 = 0, shift = 0: silu(g) * u.  c1 = 2 sqrt(2/pi), c3 = 0.044715 c1: gelu in its tanh form times u
+// (0.5 (1 + tanh(y)) = sigmoid(2 y)).  A finite limit with c1 = alpha, shift = 1: the clamped unit.
+struct GateForm { float limit, c1, c3, shift; };
+inline GateForm gate_silu() { GateForm f; f.limit = INFINITY; f.c1 = 1.f; f.c3 = 0.f; f.shift = 0.f; return f; }
+__device__ __forceinline__ float gated_unit(float g, float u, const GateForm& f) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit);
+    return g / (1.f + expf(-g * fmaf(f.c3 * g, g, f.c1))) * (u + f.shift);
+}
+// the same with the faster exponential, for epilogues whose result is rounded to bfloat16
+__device__ __forceinline__ float gated_unit_fast(float g, float u, const GateForm& f) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit);
+    return g / (1.f + __expf(-g * fmaf(f.c3 * g, g, f.c1))) * (u + f.shift);
 }
 
 // Block-wide sum / max for blockDim.x a multiple of 32 (<= 1024); `red` holds 33 floats.

@@ -245,7 +245,7 @@ __global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams p) {
 // out_ss [M][ceil(N / 64)] = sums of squares of the new res by strip of 64 columns.
 // fault (may be null): set to 8 when the wait for the cluster's partial sums runs out.
 TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int N, int K,
-                                  int ksplit, int epi, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
+                                  int ksplit, int epi, GateForm gate, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
                                   float* res, int ldr, const float* norm_w, float* out_ss, int* fault,
                                   cudaStream_t stream) {
     if (M <= 0 || N <= 0 || K <= 0) return TIS_OK;
@@ -283,7 +283,7 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
     }
     GemmParams p;
     p.x = (const bf16*)x; p.ldx = ldx; p.w = (const bf16*)w; p.ldw = ldw; p.K = K;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
     p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss; p.e.fault = fault;
     TIS_TIMELINE_TAKE(p);
@@ -332,6 +332,6 @@ TIS_API int tis_gemm_skinny(const void* x, int ldx, const void* w, int ldw, void
         tis_set_error("gemm_skinny: the residual epilogue goes through tis_gemm_skinny_fused");
         return TIS_BAD_SIZE;
     }
-    return tis_gemm_skinny_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
+    return tis_gemm_skinny_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, gate_silu(), nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
                                  nullptr, nullptr, stream);
 }

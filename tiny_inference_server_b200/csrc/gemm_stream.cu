@@ -217,7 +217,7 @@ __global__ void __launch_bounds__(NTH + 32) gemm_stream_kernel(const __grid_cons
 // Refuses what the TMA engine cannot address: K, N and the strides must be multiples of 8 elements and
 // the pointers 16-byte aligned.  in_ss .. out_ss: as in tis_gemm_skinny_fused.
 TIS_API int tis_gemm_stream_fused(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int N, int K,
-                                  int ksplit, int epi, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
+                                  int ksplit, int epi, GateForm gate, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
                                   float* res, int ldr, const float* norm_w, float* out_ss, int* fault,
                                   cudaStream_t stream) {
     if (M <= 0 || N <= 0 || K <= 0) return TIS_OK;
@@ -258,7 +258,7 @@ TIS_API int tis_gemm_stream_fused(const void* x, int ldx, const void* w, int ldw
     if (!tensor_map(w, N, K, ldw, BK, true, &wm)) return TIS_CUDA_ERROR;
     StreamParams p;
     p.x = (const bf16*)x; p.ldx = ldx; p.K = K;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.fault = fault;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate; p.e.fault = fault;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
     p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss;
     TIS_TIMELINE_TAKE(p);
@@ -311,6 +311,6 @@ TIS_API int tis_gemm_stream(const void* x, int ldx, const void* w, int ldw, void
         tis_set_error("gemm_stream: the residual epilogue goes through tis_gemm_stream_fused");
         return TIS_BAD_SIZE;
     }
-    return tis_gemm_stream_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
+    return tis_gemm_stream_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, gate_silu(), nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
                                  nullptr, fault, stream);
 }

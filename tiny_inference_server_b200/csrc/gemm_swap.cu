@@ -267,10 +267,10 @@ gemm_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 if (n < p.e.N) {
                     const int oc = (n0 >> 1) + (c4 >> 4) * 32 + (c4 & 7) * 4;
                     bf16* o = p.e.out + (size_t)row * p.e.ldo + oc;
-                    o[0] = __float2bfloat16_rn(g.x / (1.f + expf(-g.x)) * u.x);
-                    o[1] = __float2bfloat16_rn(g.y / (1.f + expf(-g.y)) * u.y);
-                    o[2] = __float2bfloat16_rn(g.z / (1.f + expf(-g.z)) * u.z);
-                    o[3] = __float2bfloat16_rn(g.w / (1.f + expf(-g.w)) * u.w);
+                    o[0] = __float2bfloat16_rn(gated_unit(g.x, u.x, p.e.gate));
+                    o[1] = __float2bfloat16_rn(gated_unit(g.y, u.y, p.e.gate));
+                    o[2] = __float2bfloat16_rn(gated_unit(g.z, u.z, p.e.gate));
+                    o[3] = __float2bfloat16_rn(gated_unit(g.w, u.w, p.e.gate));
                 }
             }
         }
@@ -330,7 +330,7 @@ int launch_swap(const CUtensorMap& mw, const CUtensorMap& mx, SwapParams p, int 
 // Refuses what the TMA engine cannot address: K, N and the strides must be multiples of 8 elements and the pointers
 // 16-byte aligned.  in_ss .. out_ss: as in tis_gemm_skinny_fused (epi 2 = the residual epilogue).
 TIS_API int tis_gemm_swap_fused(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int N, int K,
-                                int ksplit, int epi, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
+                                int ksplit, int epi, GateForm gate, const float* in_ss, int in_parts, float in_eps, int in_width, int in_kind,
                                 float* res, int ldr, const float* norm_w, float* out_ss, int* fault, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || K <= 0) return TIS_OK;
     if (M > 64) {
@@ -370,7 +370,7 @@ TIS_API int tis_gemm_swap_fused(const void* x, int ldx, const void* w, int ldw, 
     if (!tensor_map(w, N, K, ldw, BK, true, &mw) || !tensor_map(x, K, M, ldx, nb, true, &mx)) return TIS_CUDA_ERROR;
     SwapParams p;
     p.K = K; p.stages = 0;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.fault = fault;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate; p.e.fault = fault;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
     p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss;
     p.kc = ((K + ksplit - 1) / ksplit + BK - 1) / BK * BK;
@@ -385,6 +385,6 @@ TIS_API int tis_gemm_swap(const void* x, int ldx, const void* w, int ldw, void* 
         tis_set_error("gemm_swap: the residual epilogue goes through tis_gemm_swap_fused");
         return TIS_BAD_SIZE;
     }
-    return tis_gemm_swap_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
+    return tis_gemm_swap_fused(x, ldx, w, ldw, out, ldo, M, N, K, ksplit, epi, gate_silu(), nullptr, 0, 0.f, 0, 0, nullptr, 0, nullptr,
                                nullptr, fault, stream);
 }

@@ -37,6 +37,7 @@ struct TcParams {
     int M, N, K;
     int tiles_m, tiles_n;
     int* fault;
+    GateForm gate;              // EPI_SWIGLU: the form of the gating
 };
 
 template <int BN, int STAGES, int EPI>
@@ -152,7 +153,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     tmem_ld32(taddr + c * 64 + 32, u);
                     if (row < p.M && n0 + c * 64 < p.N) {
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) g[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
+                        for (int i = 0; i < 32; ++i) g[i] = gated_unit_fast(g[i], u[i], p.gate);
                         bf16* o = p.out + (size_t)row * p.ldo + (n0 >> 1) + c * 32;
 #pragma unroll
                         for (int q = 0; q < 4; ++q) store8(o + q * 8, g + q * 8);
@@ -205,7 +206,7 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, TcParams p, cudaStream_
 // TMA engine cannot address: K, N and the strides must be multiples of 8 elements and the
 // pointers 16-byte aligned; with epi = 1, N must be a multiple of 64.
 TIS_API int tis_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int N, int K,
-                        int epi, int* fault, cudaStream_t stream) {
+                        int epi, GateForm gate, int* fault, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return TIS_OK;
     if (K <= 0 || (K % 8) || (N % 8) || (ldx % 8) || (ldw % 8) || (ldo % 8) ||
         (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) % 16) {
@@ -229,6 +230,7 @@ TIS_API int tis_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* ou
     p.M = M; p.N = N; p.K = K;
     p.tiles_m = p.tiles_n = 0;
     p.fault = fault;
+    p.gate = gate;
     // The tile width that needs the least time by a simple count: rounds of tiles over the SMs
     // times the width of a tile plus its fixed cost.
     const int tm = (M + BM - 1) / BM, sms = sm_count();

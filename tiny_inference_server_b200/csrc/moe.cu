@@ -80,13 +80,16 @@ __device__ __forceinline__ void fill_f32(float* dst, const T* __restrict__ src, 
 // largest picks, and only the experts of the `keep` strongest groups stay in the race;  the `top` largest picks
 // win (the lower index on a tie);  weights: their s over the sum of those (+ weight_eps).  Also sigmoid(w_sg . x)
 // if w_sg is given.  score_kind 1: the logits themselves are the picks (correction added if given) and the weights are
-// the softmax over the chosen experts' logits only.
+// the softmax over the chosen experts' logits only.  score_kind 2: s = softmax(W x) over all E experts; without a
+// correction the logits themselves are the picks (the order is the same and nothing underflows).  group_best: a group's
+// strength is its largest pick.  renorm 0 (score kinds 0 and 2): the weights are the chosen s as they are.
 // ------------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(2 * MOE_THREADS)
 moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ wr, const float* __restrict__ corr,
                  const float* __restrict__ w_sg, int d, int E, int groups, int keep, int top, float weight_eps,
-                 int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_gate, int score_kind) {
+                 int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_gate, int score_kind, int group_best,
+                 int renorm) {
     extern __shared__ __align__(16) float smem[];
     float* xs = smem;                  // [d]
     float* sc = xs + d;                // [E]  sigmoid scores
@@ -108,14 +111,29 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ wr,
         if (lane == 0) {
             for (int j = 0; j < (e1 != e0 ? 2 : 1); ++j) {
                 const int e = j == 0 ? e0 : e1;
-                const float s = (score_kind == 1 && e < E) ? z[j] : 1.f / (1.f + expf(-z[j]));
+                const float s = (score_kind != 0 && e < E) ? z[j] : 1.f / (1.f + expf(-z[j]));
                 if (e < E) { sc[e] = s; pick[e] = s + (corr != nullptr ? corr[e] : 0.f); }
                 else shared_gate[r] = s;
             }
         }
     }
     __syncthreads();
-    if (tid != 0) return;
+    if (warp != 0) return;
+    if (score_kind == 2) {                                 // the softmax over all experts, by one warp
+        float big = -INFINITY;
+        for (int e = lane; e < E; e += 32) big = fmaxf(big, sc[e]);
+        big = warp_max(big);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(sc[e] - big);
+        const float inv = 1.f / warp_sum(sum);
+        for (int e = lane; e < E; e += 32) {
+            const float s = expf(sc[e] - big) * inv;
+            if (corr != nullptr) pick[e] = s + corr[e];    // (else the picks are the logits)
+            sc[e] = s;
+        }
+        __syncwarp();
+    }
+    if (lane != 0) return;
     if (groups > 0) {
         const int per = E / groups;
         for (int g = 0; g < groups; ++g) {
@@ -124,7 +142,7 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ wr,
                 const float v = pick[g * per + i];
                 if (v > a) { b = a; a = v; } else if (v > b) b = v;
             }
-            strength[g] = per > 1 ? a + b : a;
+            strength[g] = per > 1 && !group_best ? a + b : a;
         }
         // the `keep` strongest groups stay; a kept group's strength is set to +inf as its mark
         for (int k = 0; k < keep; ++k) {
@@ -162,12 +180,14 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ wr,
         for (int k = 0; k < top; ++k) weights[(size_t)r * top + k] /= total;
         return;
     }
+    if (!renorm) return;
     const float inv = 1.f / (total + weight_eps);
     for (int k = 0; k < top; ++k) weights[(size_t)r * top + k] *= inv;
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// hidden[r * top + k][j] = silu(Wg[e][j] . x[r]) * (Wu[e][j] . x[r]),  e = chosen[r][k];  w_gu (E, 2, F, d).
+// hidden[r * top + k][j] = gated(Wg[e][j] . x[r], Wu[e][j] . x[r]) in the form `gate` (GateForm in common.cuh),
+// e = chosen[r][k];  w_gu (E, 2, F, d).
 // act >= 0: units without a gate, hidden = act(Wu[e][j] . x[r]) with w_gu (E, F, d) and act 0 relu^2, 1 gelu (tanh), 2 silu.
 // A CTA per (row and choice, block of COLS hidden columns); a warp a column at a time.
 // ------------------------------------------------------------------------------------------------------------
@@ -182,7 +202,7 @@ __device__ __forceinline__ float unit_act(float x, int kind) {
 template <typename T>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ chosen, const T* __restrict__ w_gu,
-                   T* __restrict__ hidden, int d, int top, int E, int F, int act) {
+                   T* __restrict__ hidden, int d, int top, int E, int F, int act, GateForm gate) {
     extern __shared__ __align__(16) float smem[];
     pdl_launch_dependents();
     const int pair = blockIdx.x, r = pair / top;
@@ -218,8 +238,8 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
         float r[4];
         warp_dots<T, 4>(w, x4, d, lane, vec, r);
         if (lane == 0) {
-            hidden[(size_t)pair * F + j] = from_f32<T>(r[0] / (1.f + expf(-r[0])) * r[1]);
-            if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(r[2] / (1.f + expf(-r[2])) * r[3]);
+            hidden[(size_t)pair * F + j] = from_f32<T>(gated_unit(r[0], r[1], gate));
+            if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(gated_unit(r[2], r[3], gate));
         }
     }
 }
@@ -286,10 +306,10 @@ int set_smem(K kernel, size_t bytes, const char* what) {
 
 TIS_API int tis_moe_route(int dtype, const void* x, int ldx, const float* wr, const float* corr, const float* w_sg,
                           int n, int d, int E, int groups, int keep, int top, float weight_eps, int* chosen,
-                          float* weights, float* shared_gate, int score_kind, cudaStream_t stream) {
+                          float* weights, float* shared_gate, int score_kind, int group_best, int renorm, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || E <= 0 || top <= 0 || top > E || groups < 0 || (groups > 0 && (E % groups || keep <= 0 || keep > groups ||
-        top > E / groups * keep)) || (w_sg != nullptr && shared_gate == nullptr)) {
+        top > E / groups * keep)) || score_kind < 0 || score_kind > 2 || (w_sg != nullptr && shared_gate == nullptr)) {
         tis_set_error("moe_route: %d experts, top %d, %d groups of which %d kept", E, top, groups, keep);
         return TIS_BAD_SIZE;
     }
@@ -298,13 +318,13 @@ TIS_API int tis_moe_route(int dtype, const void* x, int ldx, const float* wr, co
         const int st = set_smem(moe_route_kernel<T>, smem, "moe_route");
         if (st != TIS_OK) return st;
         tis_launch(moe_route_kernel<T>, dim3(n), dim3(2 * MOE_THREADS), smem, stream, (const T*)x, ldx, wr, corr, w_sg, d, E,
-                   groups, keep, top, weight_eps, chosen, weights, shared_gate, score_kind);
+                   groups, keep, top, weight_eps, chosen, weights, shared_gate, score_kind, group_best, renorm);
     });
     return tis_check_launch("moe_route");
 }
 
 TIS_API int tis_moe_gate_up(int dtype, const void* x, int ldx, const int* chosen, const void* w_gu, void* hidden, int n,
-                            int d, int top, int E, int F, int act, cudaStream_t stream) {
+                            int d, int top, int E, int F, int act, GateForm gate, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || top <= 0 || E <= 0 || F <= 0) {
         tis_set_error("moe_gate_up: width %d, top %d, %d experts of %d hidden", d, top, E, F);
@@ -315,7 +335,7 @@ TIS_API int tis_moe_gate_up(int dtype, const void* x, int ldx, const int* chosen
         const int st = set_smem(moe_gate_up_kernel<T>, smem, "moe_gate_up");
         if (st != TIS_OK) return st;
         tis_launch(moe_gate_up_kernel<T>, dim3(n * top, (F + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
-                   (const T*)x, ldx, chosen, (const T*)w_gu, (T*)hidden, d, top, E, F, act);
+                   (const T*)x, ldx, chosen, (const T*)w_gu, (T*)hidden, d, top, E, F, act, gate);
     });
     return tis_check_launch("moe_gate_up");
 }
@@ -405,15 +425,15 @@ __device__ __forceinline__ void g_cp_async16(void* smem, const void* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(a), "l"(gmem));
 }
 
-// C[tile rows][n0 .. n0 + 64) = A . W[e]^T over K.  GATED: W[e] holds N gate rows and then N up rows, and C = silu(gate) *
-// up; else W[e] holds N rows.  GATHER: row i of the tile is row sorted_pair[.] / top of A (a token's input; places
+// C[tile rows][n0 .. n0 + 64) = A . W[e]^T over K.  GATED: W[e] holds N gate rows and then N up rows, and C = gated(gate,
+// up) in the form `gate`; else W[e] holds N rows.  GATHER: row i of the tile is row sorted_pair[.] / top of A (a token's input; places
 // without a pair: zeros); else row i of the tile is row tile * 64 + i of A (the sorted hidden rows).  act >= 0 (not GATED):
 // C = act(A . W[e]^T), the first product of units without a gate.
 template <bool GATED, bool GATHER>
 __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ sorted_pair, int top,
                    const int* __restrict__ tile_expert, const bf16* __restrict__ W, size_t expert_stride,
-                   bf16* __restrict__ C, int ldc, int N, int K, int act) {
+                   bf16* __restrict__ C, int ldc, int N, int K, int act, GateForm gate) {
     constexpr int BROWS = GATED ? 2 * GT_COLS : GT_COLS;
     __shared__ __align__(16) bf16 As[GT_STAGES][GT_ROWS][GT_LD];
     __shared__ __align__(16) bf16 Bs[GT_STAGES][BROWS][GT_LD];
@@ -505,8 +525,8 @@ moe_grouped_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ 
                 const int col = n0 + wn * 32 + n * 8 + 2 * t4;
                 float v0 = acc[0][mi][n][2 * half], v1 = acc[0][mi][n][2 * half + 1];
                 if (GATED) {
-                    v0 = v0 / (1.f + __expf(-v0)) * acc[GATED ? 1 : 0][mi][n][2 * half];
-                    v1 = v1 / (1.f + __expf(-v1)) * acc[GATED ? 1 : 0][mi][n][2 * half + 1];
+                    v0 = gated_unit_fast(v0, acc[GATED ? 1 : 0][mi][n][2 * half], gate);
+                    v1 = gated_unit_fast(v1, acc[GATED ? 1 : 0][mi][n][2 * half + 1], gate);
                 } else if (act >= 0) {
                     v0 = unit_act(v0, act);
                     v1 = unit_act(v1, act);
@@ -573,7 +593,7 @@ TIS_API int tis_moe_grouped_tiles(int pairs, int E) { return (pairs + GT_ROWS - 
 TIS_API int tis_moe_grouped(const void* x, int ldx, const int* chosen, const float* weights, const void* w_gu,
                             const void* w_down, const void* shared, int lds, const float* shared_gate, void* out,
                             int* sorted_pair, int* pair_place, int* tile_expert, void* hidden, void* y, int n, int d,
-                            int top, int E, int F, int act, cudaStream_t stream) {
+                            int top, int E, int F, int act, GateForm gate, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || F <= 0 || d % GT_BK || F % GT_BK || ldx % 8 || lds % 2 || E <= 0 || E > 4096 || top <= 0 ||
         ((uintptr_t)x | (uintptr_t)w_gu | (uintptr_t)w_down | (uintptr_t)hidden | (uintptr_t)y) % 16 ||
@@ -588,16 +608,16 @@ TIS_API int tis_moe_grouped(const void* x, int ldx, const int* chosen, const flo
     if (act >= 0)
         tis_launch(moe_grouped_kernel<false, true>, dim3(tiles, (F + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                    (const bf16*)x, ldx, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_gu, (size_t)F * d,
-                   (bf16*)hidden, F, F, d, act);
+                   (bf16*)hidden, F, F, d, act, gate);
     else
         tis_launch(moe_grouped_kernel<true, true>, dim3(tiles, (F + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                    (const bf16*)x, ldx, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_gu,
-                   (size_t)2 * F * d, (bf16*)hidden, F, F, d, -1);
+                   (size_t)2 * F * d, (bf16*)hidden, F, F, d, -1, gate);
     st = tis_check_launch("moe_grouped_gate_up");
     if (st != TIS_OK) return st;
     tis_launch(moe_grouped_kernel<false, false>, dim3(tiles, (d + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                (const bf16*)hidden, F, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_down, (size_t)d * F,
-               (bf16*)y, d, d, F, -1);
+               (bf16*)y, d, d, F, -1, gate);
     st = tis_check_launch("moe_grouped_down");
     if (st != TIS_OK) return st;
     return tis_moe_combine_launch(y, d, pair_place, weights, shared, lds, shared_gate, out, n, d, top, stream);

@@ -5,7 +5,7 @@
 // names.  The experts' matrices lie stacked and stored (out, in): for the tensor cores that is the K-major second
 // operand, as the keys of attention are, so a TMA box of BN weight rows x 64 elements of K lands as the operand tile
 // it is, and a tile's expert only moves the box's row coordinate.
-//   gated   C[rows][h] = silu(x . Wg[e][h]) * (x . Wu[e][h]): the box of a tile's gate rows and the box of its up rows
+//   gated   C[rows][h] = gated(x . Wg[e][h], x . Wu[e][h]) (GateForm in common.cuh): the box of a tile's gate rows and the box of its up rows
 //           form one operand of BN = 2 x BH rows; the accumulator's first BH columns are the gates, the others the ups.
 //   plain   C[rows][c] = x . Wd[e][c].
 // Roles, hand-offs, bounded waits and the double-buffered accumulator are those of gemm_tc.cu; tiles whose table entry
@@ -30,6 +30,7 @@ struct MoeTcParams {
     int tiles_m, tiles_n;
     const int* tile_expert;
     int* fault;
+    GateForm gate;          // gated: the form of the gating
     int act;                // not gated: -1 none, else the activation of the output (0 relu^2, 1 gelu (tanh), 2 silu)
 };
 
@@ -145,7 +146,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
                     float u[32];
                     tmem_ld32(taddr + BH + c * 32, u);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) g[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
+                    for (int i = 0; i < 32; ++i) g[i] = gated_unit_fast(g[i], u[i], p.gate);
                 } else if (p.act >= 0) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) g[i] = tile_act(g[i], p.act);
@@ -221,7 +222,7 @@ TIS_API int tis_moe_tc_tiles(int pairs, int E) { return (pairs + BM - 1) / BM + 
 TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const float* weights, const void* w_gu,
                                const void* w_down, const void* shared, int lds, const float* shared_gate, void* out,
                                int* sorted_pair, int* pair_place, int* tile_expert, void* xs, void* hidden, void* y, int n,
-                               int d, int top, int E, int F, int act, int* fault, cudaStream_t stream) {
+                               int d, int top, int E, int F, int act, GateForm gate, int* fault, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || F <= 0 || d % BK || F % BK || ldx % 8 || lds % 2 || E <= 0 || E > 4096 || top <= 0 ||
         ((uintptr_t)x | (uintptr_t)w_gu | (uintptr_t)w_down | (uintptr_t)xs | (uintptr_t)hidden | (uintptr_t)y) % 16 ||
@@ -240,6 +241,7 @@ TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const 
     CUtensorMap ma, mb;
     MoeTcParams p;
     p.fault = fault;
+    p.gate = gate;
     p.tile_expert = tile_expert;
     p.tiles_m = tiles_m;
     p.tiles_n = 0;

@@ -495,15 +495,17 @@ TIS_API int tis_rope_kv_write(int dtype, void* qkv, int row_stride, const int* p
 }
 
 // ----------------------------------------------------------------------------------
-// SwiGLU gating: out[r, j] = silu(gate_j) * up_j   (main_models_new.py:51).  The input row
+// Gating: out[r, j] = gated(gate_j, up_j) in the given form (GateForm in common.cuh; silu(gate_j) * up_j:
+// main_models_new.py:51).  The input row
 // holds gate and up in alternating blocks of `block` columns: [gate 0..b-1 | up 0..b-1 |
 // gate b..2b-1 | ...]; block = F is the plain layout [all gates | all ups].
 // ----------------------------------------------------------------------------------
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, int block, size_t total) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, int block, size_t total, GateForm form) {
     pdl_launch_dependents();
     pdl_wait();
     constexpr int N = Vec16<T>::N;
+    constexpr bool FAST = N == 8;              // bfloat16
     if (block % N == 0) {
         // two 16-byte items per thread and trip, all four loads ordered before the first use
         const unsigned nvec = (unsigned)(total / N);
@@ -523,11 +525,11 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
             Vec16<T>::load(s2, g2);
             Vec16<T>::load(s2 + block, u2);
 #pragma unroll
-            for (int k = 0; k < N; ++k) o[k] = g1[k] / (1.f + __expf(-g1[k])) * u1[k];
+            for (int k = 0; k < N; ++k) o[k] = FAST ? gated_unit_fast(g1[k], u1[k], form) : gated_unit(g1[k], u1[k], form);
             Vec16<T>::store(out + (size_t)r1 * F + j1, o);
             if (two) {
 #pragma unroll
-                for (int k = 0; k < N; ++k) o[k] = g2[k] / (1.f + __expf(-g2[k])) * u2[k];
+                for (int k = 0; k < N; ++k) o[k] = FAST ? gated_unit_fast(g2[k], u2[k], form) : gated_unit(g2[k], u2[k], form);
                 Vec16<T>::store(out + (size_t)r2 * F + j2, o);
             }
         }
@@ -541,11 +543,11 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const T* src = gu + r * 2 * F + (size_t)b * 2 * block + (j - b * block);
         const float g = to_f32(src[0]);
         const float u = to_f32(src[block]);
-        out[idx] = from_f32<T>(g / (1.f + expf(-g)) * u);
+        out[idx] = from_f32<T>(gated_unit(g, u, form));
     }
 }
 
-TIS_API int tis_swiglu(int dtype, const void* gu, void* out, int n, int F, int block, cudaStream_t stream) {
+TIS_API int tis_swiglu(int dtype, const void* gu, void* out, int n, int F, int block, GateForm form, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (block <= 0 || F % block) {
         tis_set_error("swiglu: block %d does not divide the hidden size %d", block, F);
@@ -561,7 +563,7 @@ TIS_API int tis_swiglu(int dtype, const void* gu, void* out, int n, int F, int b
     if (blocks > 148 * 16) blocks = 148 * 16;
     TIS_DISPATCH_DTYPE(dtype, T,
         tis_launch(swiglu_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)gu, (T*)out, F, block,
-                   total));
+                   total, form));
     return tis_check_launch("swiglu");
 }
 

@@ -19,7 +19,7 @@ import torch
 from . import build as _build
 
 _lib = None
-ABI_VERSION = 11
+ABI_VERSION = 12
 #: launches of this library's kernels so far (library matrix products are not counted)
 launches = 0
 #: calls by kind, for tests that must know which kernel a product or an attention went to
@@ -121,6 +121,31 @@ EPI_ACT = {"relu2": 3, "gelu_tanh": 4, "silu": 5}
 #: TIS_FUSED_NORM=0 keeps the norm kernel
 FUSED_NORM = os.environ.get("TIS_FUSED_NORM", "1") != "0"
 
+
+class GateForm(ctypes.Structure):
+    """What a gated unit does with a gate g and an up value u: ``g' * sigmoid(g' * (c1 + c3 * g'^2)) * (u' + shift)`` with
+    ``g' = min(g, limit)`` and ``u' = min(max(u, -limit), limit)`` (``csrc/common.cuh``)."""
+
+    _fields_ = [("limit", ctypes.c_float), ("c1", ctypes.c_float), ("c3", ctypes.c_float), ("shift", ctypes.c_float)]
+
+
+def gate_silu() -> GateForm:
+    """``silu(g) * u``"""
+    return GateForm(math.inf, 1.0, 0.0, 0.0)
+
+
+def gate_gelu_tanh() -> GateForm:
+    """``gelu(g) * u`` with gelu in its tanh form (``0.5 (1 + tanh(y)) = sigmoid(2 y)``)"""
+    c = 2.0 * math.sqrt(2.0 / math.pi)
+    return GateForm(math.inf, c, 0.044715 * c, 0.0)
+
+
+def gate_clamped(limit: float, alpha: float = 1.702, shift: float = 1.0) -> GateForm:
+    """``g' * sigmoid(alpha * g') * (u' + shift)``, the gate bounded above by ``limit``, the up value on both sides"""
+    return GateForm(limit, alpha, 0.0, shift)
+
+
+SILU = gate_silu()
 
 #: the factor a norm multiplies a row with, as a function of the row's sum of squares s over a width d:
 #: "l2_eps": sqrt(d) / (sqrt(s) + eps) (eps added to the L2 norm); "mean_eps": rsqrt(s / d + eps)
@@ -247,11 +272,11 @@ def _ksplit_swap(n_cols: int, k: int) -> int:
 
 
 def gemm_swap(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bool = False,
-              ksplit: Optional[int] = None, sink: Optional["ResidualSink"] = None):
+              ksplit: Optional[int] = None, sink: Optional["ResidualSink"] = None, form: GateForm = SILU):
     """``a (n <= 64, K) @ w (K, N)`` in bfloat16 on the tcgen05 tensor cores with the operands swapped (128
     columns of ``w`` are the rows of the tile, the rows of ``a`` its narrow side); with ``swiglu`` the columns of
-    ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2).  ``a`` may be ``ScaledRows``; with ``sink`` the
-    result is added to the residual stream and comes back as ``ScaledRows``."""
+    ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2), gated in ``form``.  ``a`` may be ``ScaledRows``; with
+    ``sink`` the result is added to the residual stream and comes back as ``ScaledRows``."""
     lib = library()
     scaled = a if isinstance(a, ScaledRows) else None
     if scaled is not None:
@@ -268,7 +293,7 @@ def gemm_swap(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bo
     calls["gemm_swap"] += 1
     epi = EPI_RESIDUAL if sink is not None else (EPI_SWIGLU if swiglu else EPI_STORE)
     _check(lib.tis_gemm_swap_fused(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), n, cols, k,
-                                   ksplit or _ksplit_swap(cols, k), epi, *head, *tail, _p(tc_fault()), _stream()), lib)
+                                   ksplit or _ksplit_swap(cols, k), epi, form, *head, *tail, _p(tc_fault()), _stream()), lib)
     return result if sink is not None else out
 
 
@@ -305,10 +330,11 @@ def _sink_fits(sink: Optional[ResidualSink], n: int, cols: int, out) -> bool:
 
 
 def gemm_stream(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bool = False,
-                ksplit: Optional[int] = None, sink: Optional[ResidualSink] = None, act: Optional[str] = None):
+                ksplit: Optional[int] = None, sink: Optional[ResidualSink] = None, act: Optional[str] = None,
+                form: GateForm = SILU):
     """``a (n <= 64, K) @ w (K, N)`` in bfloat16 by the TMA-fed weight-streaming kernel; with ``swiglu``
-    the columns of ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2).  ``a`` may be ``ScaledRows``;
-    with ``sink`` the result is added to the residual stream and comes back as ``ScaledRows``; with ``act`` (a key of
+    the columns of ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2), gated in ``form``.  ``a`` may be
+    ``ScaledRows``; with ``sink`` the result is added to the residual stream and comes back as ``ScaledRows``; with ``act`` (a key of
     ``EPI_ACT``; not with ``swiglu`` or ``sink``) the 32-bit sums pass that activation on their way out."""
     lib = library()
     scaled = a if isinstance(a, ScaledRows) else None
@@ -326,7 +352,7 @@ def gemm_stream(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: 
     calls["gemm_stream"] += 1
     epi = _epilogue(sink, swiglu, act)
     _check(lib.tis_gemm_stream_fused(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), n, cols, k,
-                                     ksplit or _ksplit(cols, k), epi, *head, *tail, _p(tc_fault()), _stream()), lib)
+                                     ksplit or _ksplit(cols, k), epi, form, *head, *tail, _p(tc_fault()), _stream()), lib)
     return result if sink is not None else out
 
 
@@ -339,15 +365,16 @@ def _epilogue(sink, swiglu: bool, act: Optional[str]) -> int:
 
 
 def gemm_skinny(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bool = False,
-                ksplit: Optional[int] = None, sink: Optional[ResidualSink] = None, act: Optional[str] = None):
+                ksplit: Optional[int] = None, sink: Optional[ResidualSink] = None, act: Optional[str] = None,
+                form: GateForm = SILU):
     """``a (n <= 64, K) @ w (K, N)`` in bfloat16 by a weight-streaming kernel; with ``swiglu``
-    the columns of ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2).  ``a`` may be ``ScaledRows``;
-    with ``sink`` the result is added to the residual stream and comes back as ``ScaledRows``; ``act`` as in
+    the columns of ``w`` are [32 gate | 32 up] blocks and the result is (n, N/2), gated in ``form``.  ``a`` may be
+    ``ScaledRows``; with ``sink`` the result is added to the residual stream and comes back as ``ScaledRows``; ``act`` as in
     ``gemm_stream``."""
     rows = a.rows if isinstance(a, ScaledRows) else a
     if (_stream_pays(rows.shape[0], rows.shape[1], w.shape[1], ksplit) and rows.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
             and _stream_fits(rows.shape[0], rows.shape[1], ksplit or _ksplit(w.shape[1], rows.shape[1]))):
-        return gemm_stream(a, w, out, swiglu, ksplit, sink, act)
+        return gemm_stream(a, w, out, swiglu, ksplit, sink, act, form)
     lib = library()
     scaled = a if isinstance(a, ScaledRows) else None
     a = rows
@@ -363,7 +390,7 @@ def gemm_skinny(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: 
     calls["gemm_skinny"] += 1
     epi = _epilogue(sink, swiglu, act)
     _check(lib.tis_gemm_skinny_fused(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), n, cols, k,
-                                     ksplit or _ksplit(cols, k), epi, *head, *tail, _p(tc_fault()), _stream()), lib)
+                                     ksplit or _ksplit(cols, k), epi, form, *head, *tail, _p(tc_fault()), _stream()), lib)
     return result if sink is not None else out
 
 
@@ -395,7 +422,8 @@ def _tc_ok(a: torch.Tensor, w: torch.Tensor, min_rows: int) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bool = False) -> torch.Tensor:
+def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, swiglu: bool = False,
+            form: GateForm = SILU) -> torch.Tensor:
     """``a (n, K) @ w (K, N)`` in bfloat16 on the tcgen05 tensor cores (TMA-fed, accumulator in
     tensor memory); with ``swiglu`` the columns of ``w`` are [32 gate | 32 up] blocks and the
     result is (n, N/2)."""
@@ -406,7 +434,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None
         out = torch.empty((n, cols // 2 if swiglu else cols), dtype=a.dtype, device=a.device)
     calls["gemm_tc"] += 1
     _check(lib.tis_gemm_tc(_p(a), a.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), n, cols, k,
-                           EPI_SWIGLU if swiglu else EPI_STORE, _p(tc_fault()), _stream()), lib)
+                           EPI_SWIGLU if swiglu else EPI_STORE, form, _p(tc_fault()), _stream()), lib)
     return out
 
 
@@ -503,8 +531,8 @@ def gemm(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, sink: Optional[
     return torch.mm(a, w, out=out)
 
 
-def gemm_swiglu(a, w_gu: torch.Tensor, hidden: int, block: int) -> torch.Tensor:
-    """``swiglu(a @ w_gu)``: (n, hidden).  ``w_gu`` (K, 2*hidden) holds gate and up columns in
+def gemm_swiglu(a, w_gu: torch.Tensor, hidden: int, block: int, form: GateForm = SILU) -> torch.Tensor:
+    """``gated(a @ w_gu)`` in the form ``form``: (n, hidden).  ``w_gu`` (K, 2*hidden) holds gate and up columns in
     alternating blocks of ``block``.  Few bfloat16 rows with block 32: one kernel with the
     gating in its epilogue; else the product and the gating kernel.  ``a`` may be ``ScaledRows``."""
     scaled = a if isinstance(a, ScaledRows) else None
@@ -512,17 +540,17 @@ def gemm_swiglu(a, w_gu: torch.Tensor, hidden: int, block: int) -> torch.Tensor:
         a = scaled.rows
     if block == 32 and _skinny_ok(a, w_gu, SKINNY_SWIGLU_MAX_ROWS) and (
             _ring_tiles(w_gu.shape[1], a.shape[1]) <= RING_MAX_TILES or not _swap_ok(a, w_gu, swiglu=True)):
-        return gemm_skinny(scaled if scaled is not None else a, w_gu, swiglu=True)
+        return gemm_skinny(scaled if scaled is not None else a, w_gu, swiglu=True, form=form)
     if (block == 32 and _skinny_ok(a, w_gu, SWAP_SWIGLU_MAX_ROWS) and w_gu.shape[1] % 64 == 0
             and a.data_ptr() % 16 == 0 and w_gu.data_ptr() % 16 == 0):
-        return gemm_swap(scaled if scaled is not None else a, w_gu, swiglu=True)
+        return gemm_swap(scaled if scaled is not None else a, w_gu, swiglu=True, form=form)
     if scaled is not None:
         a = scaled.dense()
     if block == 32 and _tc_ok(a, w_gu, TC_MIN_ROWS) and w_gu.shape[1] % 64 == 0:
-        return gemm_tc(a, w_gu, swiglu=True)
+        return gemm_tc(a, w_gu, swiglu=True, form=form)
     gu = gemm(a, w_gu)
     out = torch.empty((a.shape[0], hidden), dtype=a.dtype, device=a.device)
-    return swiglu(gu, out, block)
+    return swiglu(gu, out, block, form)
 
 
 def gemm_f32_out(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -791,12 +819,12 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
     return out
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor, block: Optional[int] = None) -> torch.Tensor:
-    """out[r, j] = silu(gate_j) * up_j where a row of ``gu`` holds gate and up columns in
+def swiglu(gu: torch.Tensor, out: torch.Tensor, block: Optional[int] = None, form: GateForm = SILU) -> torch.Tensor:
+    """out[r, j] = gated(gate_j, up_j) in the form ``form`` (silu(gate_j) * up_j unless given) where a row of ``gu`` holds gate and up columns in
     alternating blocks of ``block`` (default: the hidden size, i.e. [all gates | all ups])."""
     lib = library()
     n, f = out.shape
-    _check(lib.tis_swiglu(_dt(gu), _p(gu), _p(out), n, f, block or f, _stream()), lib)
+    _check(lib.tis_swiglu(_dt(gu), _p(gu), _p(out), n, f, block or f, form, _stream()), lib)
     return out
 
 
@@ -1263,6 +1291,49 @@ def group_norm(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b:
     return out1, out2
 
 
+def add_layer_norm(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b: Optional[torch.Tensor], w: torch.Tensor,
+                   b: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``residual += delta_a + delta_b`` (each None: nothing), then ``out = (residual - mean) / sqrt(variance + eps) * w + b``
+    row by row in 32-bit (the variance is the mean of the squared deviations)."""
+    lib = library()
+    n, d = residual.shape
+    for t in (delta_a, delta_b):
+        if t is not None and (t.dtype != out.dtype or not t.is_contiguous()):
+            raise KernelError("add_layer_norm: the updates are contiguous and of the output's type")
+    _check(lib.tis_add_layer_norm(_dt(out), _p(residual), _p(delta_a), _p(delta_b), _p(w), _p(b), _f(eps), _p(out), n, d,
+                                  _stream()), lib)
+    return out
+
+
+def rotate_norm_store(qkv: torch.Tensor, num_heads: int, kv_heads: int, dim: int, v_dim: int, cos: Optional[torch.Tensor],
+                      sin: Optional[torch.Tensor], interleaved: bool, norm: bool, eps: float, k_pages: Optional[torch.Tensor],
+                      v_pages: Optional[torch.Tensor], block_table: torch.Tensor, positions: torch.Tensor,
+                      row_slot: torch.Tensor, page_size: int, fault: torch.Tensor) -> None:
+    """Between the projections and the cache of an attention whose queries and keys are rotated and then normed head by
+    head.  A row of ``qkv``: H query heads and G key heads of ``dim`` elements, G value heads of ``v_dim``.  The first
+    elements of every query and key head, twice as many as ``cos`` and ``sin`` (positions, rot / 2; None: none) have columns,
+    are rotated by the row's position (``interleaved``: element 2i with 2i + 1, else i with i + rot / 2); with ``norm`` the
+    head is then divided by its root mean square (eps inside the root).  Queries in place; keys and values into the row's
+    page.  ``kv_heads`` 0: the rows hold queries only and nothing is stored.  Everything is computed in 32-bit."""
+    lib = library()
+    n = qkv.shape[0]
+    rot = 0 if cos is None else 2 * cos.shape[1]
+    kps = khs = vps = vhs = ctypes.c_size_t(0)
+    if kv_heads:
+        kps, khs = _page_strides(k_pages, dim)
+        vps, vhs = _page_strides(v_pages, v_dim)
+        if k_pages.shape[1] != kv_heads or v_pages.shape[1] != kv_heads:
+            raise KernelError("rotate_norm_store: the pages do not fit the key/value heads")
+    else:
+        k_pages = v_pages = None
+    if qkv.stride(1) != 1:
+        raise KernelError("rotate_norm_store: the rows are not dense")
+    _check(lib.tis_rotate_norm_store(_dt(qkv), _p(qkv), qkv.stride(0), num_heads, kv_heads, dim, v_dim, rot, int(interleaved),
+                                     _p(cos), _p(sin), int(norm), _f(eps), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
+                                     page_size, k_pages.shape[0] if k_pages is not None else 0, _p(block_table),
+                                     block_table.stride(0), _p(positions), _p(row_slot), _p(fault), n, _stream()), lib)
+
+
 def scaled_sum(a: torch.Tensor, scale_a: float, b: torch.Tensor, scale_b: float) -> torch.Tensor:
     """``a * scale_a + b * scale_b`` (n, d), the sum formed in 32-bit; row strides free."""
     lib = library()
@@ -1295,17 +1366,21 @@ def rotate_tie_store(qk: torch.Tensor, num_heads: int, kv_heads: int, dim: int, 
 # ---------------------------------------------------------------------------------------
 
 #: how a router turns logits into choices and weights
-ROUTER_SCORES = {"sigmoid": 0, "softmax_chosen": 1}
+ROUTER_SCORES = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
+#: the strength of a group of experts: the sum of its two largest choosing scores, or its largest
+GROUP_SCORES = {"two_best": 0, "best": 1}
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor],
               w_shared_gate: Optional[torch.Tensor], groups: int, keep: int, top: int, weight_eps: float = 1e-20,
-              scores: str = "sigmoid"):
+              scores: str = "sigmoid", group_score: str = "two_best", renorm: bool = True):
     """The router of a mixture of experts, a row at a time, in 32-bit: ``s = sigmoid(w_router x)`` (E experts);
     choosing scores ``s + correction``; with ``groups`` > 0 only the experts of the ``keep`` groups (of E / groups
     neighbours) with the largest sum of their two best choosing scores can be chosen; the ``top`` largest choosing
     scores win (the lower index on a tie); weights ``s`` of the chosen over their sum (+ ``weight_eps``).  ``scores``
-    ``"softmax_chosen"``: the logits themselves choose and the weights are the softmax over the chosen logits only.  Returns
+    ``"softmax_chosen"``: the logits themselves choose and the weights are the softmax over the chosen logits only;
+    ``"softmax"``: ``s = softmax(w_router x)`` over all experts.  ``group_score`` (``GROUP_SCORES``) ``"best"``: a group is as
+    strong as its largest choosing score.  ``renorm`` False: the weights are the chosen ``s`` as they are.  Returns
     (chosen (n, top) int32, weights (n, top) float32, sigmoid(w_shared_gate . x) (n,) float32 or None)."""
     lib = library()
     n, d = x.shape
@@ -1315,12 +1390,13 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torc
     shared = torch.empty((n,), dtype=torch.float32, device=x.device) if w_shared_gate is not None else None
     _check(lib.tis_moe_route(_dt(x), _p(x), x.stride(0), _p(w_router), _p(correction), _p(w_shared_gate), n, d, experts,
                              int(groups), int(keep), int(top), _f(weight_eps), _p(chosen), _p(weights), _p(shared),
-                             ROUTER_SCORES[scores], _stream()), lib)
+                             ROUTER_SCORES[scores], GROUP_SCORES[group_score], int(renorm), _stream()), lib)
     return chosen, weights, shared
 
 
-def moe_gate_up(x: torch.Tensor, chosen: torch.Tensor, w_gate_up: torch.Tensor, act: Optional[str] = None) -> torch.Tensor:
-    """``hidden[r * top + k] = silu(Wg[e] x[r]) * (Wu[e] x[r])`` with ``e = chosen[r, k]``: ``w_gate_up`` (E, 2, F, d)
+def moe_gate_up(x: torch.Tensor, chosen: torch.Tensor, w_gate_up: torch.Tensor, act: Optional[str] = None,
+                form: GateForm = SILU) -> torch.Tensor:
+    """``hidden[r * top + k] = gated(Wg[e] x[r], Wu[e] x[r])`` in the form ``form`` with ``e = chosen[r, k]``: ``w_gate_up`` (E, 2, F, d)
     holds every expert's gate and up matrices (out, in); the result is (n * top, F) in the dtype of ``x``.  ``act``
     (``ACTIVATIONS``): units without a gate, ``hidden = act(Wu[e] x[r])`` with ``w_gate_up`` (E, F, d)."""
     lib = library()
@@ -1329,13 +1405,13 @@ def moe_gate_up(x: torch.Tensor, chosen: torch.Tensor, w_gate_up: torch.Tensor, 
     experts, hidden = w_gate_up.shape[0], w_gate_up.shape[-2]
     out = torch.empty((n * top, hidden), dtype=x.dtype, device=x.device)
     _check(lib.tis_moe_gate_up(_dt(x), _p(x), x.stride(0), _p(chosen), _p(w_gate_up), _p(out), n, d, top, experts, hidden,
-                               ACTIVATIONS[act] if act is not None else -1, _stream()), lib)
+                               ACTIVATIONS[act] if act is not None else -1, form, _stream()), lib)
     return out
 
 
 def moe_down(hidden: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_down: torch.Tensor,
              shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor]) -> torch.Tensor:
-    """``out[r] = sum_k weights[r, k] * Wd[chosen[r, k]] hidden[r * top + k] (+ shared_gate[r] * shared[r])``:
+    """``out[r] = sum_k weights[r, k] * Wd[chosen[r, k]] hidden[r * top + k] (+ shared_gate[r] * shared[r]; the gate None: + shared[r])``:
     ``w_down`` (E, d, F) (out, in), ``hidden`` (n * top, F), ``shared`` (n, d) or None; the result is (n, d)."""
     lib = library()
     n, top = chosen.shape
@@ -1398,9 +1474,10 @@ MOE_TC_MIN_PAIRS = int(os.environ.get("TIS_MOE_TC_MIN_PAIRS", "1024"))
 
 
 def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor], act: Optional[str] = None) -> torch.Tensor:
-    """``out[r] = sum_k weights[r, k] * unit(chosen[r, k])(x[r]) (+ shared_gate[r] * shared[r])`` with the gated units
-    ``unit(e)(x) = Wd[e] (silu(Wg[e] x) * (Wu[e] x))``: ``w_gate_up`` (E, 2, F, d), ``w_down`` (E, d, F); or, with ``act``
+                shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor], act: Optional[str] = None,
+                form: GateForm = SILU) -> torch.Tensor:
+    """``out[r] = sum_k weights[r, k] * unit(chosen[r, k])(x[r]) (+ shared_gate[r] * shared[r], or + shared[r])`` with the gated
+    units ``unit(e)(x) = Wd[e] gated(Wg[e] x, Wu[e] x)`` in the form ``form``: ``w_gate_up`` (E, 2, F, d), ``w_down`` (E, d, F); or, with ``act``
     (``ACTIVATIONS``), units without a gate, ``Wd[e] act(Wu[e] x)`` and ``w_gate_up`` (E, F, d).  Few rows, and
     float32: ``moe_gate_up`` and ``moe_down`` (a dot product per output element, the weights read where they lie).  Many
     bfloat16 rows: the rows are sorted by expert on the device and every expert's rows run as tiles on the tensor
@@ -1428,7 +1505,7 @@ def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_
         _check(lib.tis_moe_grouped_tc(_p(x), x.stride(0), _p(chosen), _p(weights), _p(w_gate_up), _p(w_down), _p(shared),
                                       shared.stride(0) if shared is not None else 0, _p(shared_gate), _p(out), _p(sorted_pair),
                                       _p(pair_place), _p(tile_expert), _p(xs), _p(hid), _p(y), n, d, top, experts, hidden,
-                                      act_code, _p(tc_fault()), _stream()), lib)
+                                      act_code, form, _p(tc_fault()), _stream()), lib)
         return out
     if (grouped and n * top >= MOE_GROUPED_MIN_PAIRS and d % 32 == 0
             and hidden % 32 == 0):
@@ -1445,6 +1522,6 @@ def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_
         _check(lib.tis_moe_grouped(_p(x), x.stride(0), _p(chosen), _p(weights), _p(w_gate_up), _p(w_down), _p(shared),
                                    shared.stride(0) if shared is not None else 0, _p(shared_gate), _p(out), _p(sorted_pair),
                                    _p(pair_place), _p(tile_expert), _p(hid), _p(y), n, d, top, experts, hidden, act_code,
-                                   _stream()), lib)
+                                   form, _stream()), lib)
         return out
-    return moe_down(moe_gate_up(x, chosen, w_gate_up, act), chosen, weights, w_down, shared, shared_gate)
+    return moe_down(moe_gate_up(x, chosen, w_gate_up, act, form), chosen, weights, w_down, shared, shared_gate)

@@ -5,5 +5,6 @@ from . import kefisun  # noqa: F401  (registers "Kefisun")
 from . import mizidra  # noqa: F401  (registers "Mizidra")
 from . import biruvik  # noqa: F401  (registers "Biruvik")
 from . import kubolorn  # noqa: F401  (registers "Kubolorn")
+from . import lomutar  # noqa: F401  (registers "Lomutar")
 
 __all__ = ["Model", "ScheduleEntry", "StepOutput"]

@@ -168,7 +168,11 @@ class Norm(Part):
     ``sink(values)``: a norm whose factor per row is a function of the row's sum of squares may return
     a ``kernels.ops.ResidualSink`` for the stream ``values``: the part before the norm then adds its
     update to the stream inside its last product and the part after applies the factor after its first
-    product, so that the norm needs no kernel.  None (the default): the norm runs as a kernel of its own."""
+    product, so that the norm needs no kernel.  None (the default): the norm runs as a kernel of its own.
+
+    ``takes_two_updates``: ``add_norm`` also takes ``delta_b``, a second pending update beside the first."""
+
+    takes_two_updates = False
 
     @classmethod
     def from_config(cls, cfg, prefix: str):

@@ -4,7 +4,8 @@ not have: an *input filter* between the first norm and the mixer (a part with ``
 for instance a short convolution over time, with per-request state of its own), no feed-forward
 at all (the block is its first sublayer only), and a norm *behind* a sublayer as well (``post_mixer_norm``,
 ``post_ffn_norm``): ``x += post(sublayer(norm(x)))``, the update normalised in 32-bit on its way into the stream.  ``parallel``: both sublayers
-read the same stream, ``x += mixer(norm1(x)) + ff(norm2(x))``; the feed-forward may then have an input filter of its own
+read the same stream, ``x += mixer(norm1(x)) + ff(norm2(x))`` — or, without a second norm (``norm_ffn`` None), the same
+norm's output, ``h = norm1(x)``, ``x += mixer(h) + ff(h)``; the feed-forward may then have an input filter of its own
 (``ffn_filter``), whose state follows the mixer filter's in the block's filter state."""
 from __future__ import annotations
 
@@ -24,6 +25,8 @@ class Block(Part):
             raise ValueError("only a block whose sublayers read the same stream filters the feed-forward's input")
         if parallel and (post_mixer_norm is not None or post_ffn_norm is not None):
             raise ValueError("a block whose sublayers read the same stream has no norms behind them")
+        if ffn is not None and norm_ffn is None and not parallel:
+            raise ValueError("only a block whose sublayers read the same stream can share one norm")
         self.parallel = parallel
         self.ffn_filter = ffn_filter
         self.post_mixer_norm = post_mixer_norm
@@ -46,8 +49,8 @@ class Block(Part):
 
     def _forward_parallel(self, stream: ResidualStream, step, binding: LayerBinding) -> None:
         mixer, ffn = self.mixer, self.ffn
-        if ffn is None:
-            a = stream.normed(self.norm_mixer)
+        if ffn is None or self.norm_ffn is None:               # one norm, whose output both sublayers read
+            a = f = stream.normed(self.norm_mixer)
         else:
             a, f = stream.normed_pair(self.norm_mixer, self.norm_ffn)
         first = 0

@@ -12,7 +12,8 @@ from .base import BuildContext, FeedForward, WeightSpec
 
 class SwiGLU(FeedForward):
     """``(silu(x W1) * (x W2)) W3`` (upstream ``swiglu`` and ``ffn_router``,
-    main_models_new.py:44-60); weights ``(in, out)``: W1 gate and W2 up ``(width, hidden)``,
+    main_models_new.py:44-60), or another gating of the two projections (``form``, a ``kernels.ops.GateForm``: gelu, the
+    clamped unit); weights ``(in, out)``: W1 gate and W2 up ``(width, hidden)``,
     W3 ``(hidden, width)``.  On the device gate and up are one matrix ``(width, 2*hidden)``
     whose columns alternate in blocks of 32 gates and 32 ups (when 32 divides the hidden size;
     else all gates, then all ups), so that one 64-column strip of the product holds both
@@ -22,8 +23,9 @@ class SwiGLU(FeedForward):
     fuses_residual = True
 
     def __init__(self, width: int, hidden: int, prefix: str = "", names: Optional[Dict[str, str]] = None,
-                 stored_out_in: bool = False):
+                 stored_out_in: bool = False, form: Optional[ops.GateForm] = None):
         super().__init__(prefix)
+        self.form = ops.gate_silu() if form is None else form
         self.width = width
         self.hidden = hidden
         self.stored_out_in = stored_out_in        # the three matrices are stored (out, in) instead of (in, out)
@@ -58,7 +60,7 @@ class SwiGLU(FeedForward):
         self.w_down = down.to(device=ctx.device, dtype=ctx.dtype).contiguous()
 
     def forward(self, x, step=None, residual=None):
-        h = ops.gemm_swiglu(x, self.w_gate_up, self.hidden, self.block)
+        h = ops.gemm_swiglu(x, self.w_gate_up, self.hidden, self.block, self.form)
         return ops.gemm(h, self.w_down, sink=residual)
 
 
@@ -152,7 +154,11 @@ class RoutedExperts(FeedForward):
 
     Options: ``scores`` ``"softmax_chosen"``: the logits ``z`` themselves choose (the ``top`` largest) and the weights are
     the softmax over the chosen logits only; ``correction`` False: there is no correction tensor; ``unit_act`` (a name of
-    ``kernels.ops.ACTIVATIONS``): the experts have no gate, ``W_down act(W_up h)``, and no ``e<i>.gate`` tensors.
+    ``kernels.ops.ACTIVATIONS``): the experts have no gate, ``W_down act(W_up h)``, and no ``e<i>.gate`` tensors;
+    ``scores`` ``"softmax"``: ``s`` is the softmax over all experts; ``group_score`` ``"best"``: a group is as strong as its
+    largest choosing score; ``renorm`` False: the weights are the chosen ``s`` as they are; ``form``, ``shared_form`` (a
+    ``kernels.ops.GateForm``): the gating of the experts and of the shared unit instead of silu; ``shared_gated`` False: the
+    shared unit is added as it is, and there is no ``shared.sg``.
 
     Tensor names below the prefix: ``e<i>.gate, e<i>.up, e<i>.down``, ``router``, ``correction``, ``shared.gate,
     shared.up, shared.down, shared.sg`` (matrices stored (out, in)).  On the device the experts' matrices are stacked:
@@ -163,8 +169,13 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, width: int, hidden: int, experts: int, top: int, groups: int = 0, keep: int = 0,
                  shared_hidden: int = 0, prefix: str = "", scores: str = "sigmoid", correction: bool = True,
-                 unit_act: Optional[str] = None):
+                 unit_act: Optional[str] = None, group_score: str = "two_best", renorm: bool = True,
+                 form: Optional[ops.GateForm] = None, shared_form: Optional[ops.GateForm] = None, shared_gated: bool = True):
         super().__init__(prefix)
+        if group_score not in ops.GROUP_SCORES:
+            raise ValueError(f"group score {group_score!r}: known are {sorted(ops.GROUP_SCORES)}")
+        self.group_score, self.renorm, self.shared_gated = group_score, renorm, shared_gated
+        self.form = ops.gate_silu() if form is None else form
         if scores not in ops.ROUTER_SCORES:
             raise ValueError(f"router scores {scores!r}: known are {sorted(ops.ROUTER_SCORES)}")
         if unit_act is not None and unit_act not in ops.ACTIVATIONS:
@@ -177,7 +188,7 @@ class RoutedExperts(FeedForward):
         self.width, self.hidden, self.experts, self.top = width, hidden, experts, top
         self.groups, self.keep, self.shared_hidden = groups, keep, shared_hidden
         self.shared = SwiGLU(width, shared_hidden, prefix=prefix + "shared.", stored_out_in=True,
-                             names={"gate": "gate", "up": "up", "down": "down"}) if shared_hidden else None
+                             names={"gate": "gate", "up": "up", "down": "down"}, form=shared_form) if shared_hidden else None
         self.w_gate_up = self.w_down = self.w_router = self.correction = self.w_shared_gate = None
 
     @classmethod
@@ -201,7 +212,7 @@ class RoutedExperts(FeedForward):
                 specs[f"e{e}.gate"] = WeightSpec((self.hidden, self.width))
             specs[f"e{e}.up"] = WeightSpec((self.hidden, self.width))
             specs[f"e{e}.down"] = WeightSpec((self.width, self.hidden))
-        if self.shared is not None:
+        if self.shared is not None and self.shared_gated:
             specs["shared.sg"] = WeightSpec((1, self.width))
         return specs
 
@@ -217,14 +228,16 @@ class RoutedExperts(FeedForward):
         self.w_down = torch.stack([tensors[f"{p}e{e}.down"] for e in range(self.experts)]).to(**dev).contiguous()
         self.w_router = tensors[p + "router"].to(**f32).contiguous()
         self.correction = tensors[p + "correction"].to(**f32).contiguous() if self.has_correction else None
-        if self.shared is not None:
+        if self.shared is not None and self.shared_gated:
             self.w_shared_gate = tensors[p + "shared.sg"].to(**f32).reshape(-1).contiguous()
 
     def forward(self, x, step=None):
         chosen, weights, shared_gate = ops.moe_route(x, self.w_router, self.correction, self.w_shared_gate, self.groups,
-                                                     self.keep, self.top, self.WEIGHT_EPS, scores=self.scores)
+                                                     self.keep, self.top, self.WEIGHT_EPS, scores=self.scores,
+                                                     group_score=self.group_score, renorm=self.renorm)
         shared = self.shared.forward(x, step) if self.shared is not None else None
-        return ops.moe_experts(x, chosen, weights, self.w_gate_up, self.w_down, shared, shared_gate, act=self.unit_act)
+        return ops.moe_experts(x, chosen, weights, self.w_gate_up, self.w_down, shared, shared_gate, act=self.unit_act,
+                               form=self.form)
 
 
 register_part("ffn", "swiglu", SwiGLU)

@@ -1,0 +1,111 @@
+"""Grouped-query attention whose queries and keys are rotated and then divided by their root mean square, in a window, with a
+keyless term in the softmax, over keys and values of its own or of an earlier layer."""
+from __future__ import annotations
+
+from typing import Dict, Optional
+
+import torch
+
+from ..kernels import ops, window_plan
+from ..registry import register_part
+from .base import BuildContext, KVSpec, LayerBinding, Mixer, WeightSpec
+from .window_attention import pad8
+
+#: ``cache_window`` of a layer whose keys every reader sees inside its own window
+OWN_WINDOW = "own"
+
+
+class NormedRotaryAttention(Mixer):
+    """Causal softmax attention with ``num_heads`` query heads over ``kv_heads`` key/value heads (query head h reads key/value
+    head ``h // (num_heads / kv_heads)``):
+
+    * ``q = Wq h``, ``k = Wk h`` (``dim`` elements a head), ``v = Wv h`` (``v_dim``), no biases;
+    * ``position`` (a ``RotaryHalf`` family member, None: none) rotates the first ``position.rotary_dim`` elements of every
+      query and key head by the token's position;
+    * ``qk_norm``: every query and key head is *then* divided by its root mean square over ``dim`` (``eps`` inside the root, no
+      weight);
+    * ``score = (q . k) * scale`` over the keys ``p - window + 1 .. p`` (``window`` None: ``0 .. p``), softmax in 32-bit; with
+      ``has_sink`` its denominator also holds ``exp(sink[h])``, a term without a key or a value behind it;
+    * ``Wo`` on the heads' outputs side by side.
+
+    The cache holds the keys as the scores take them (rotated, normed) and the values.  ``reads_cache``: the layer has no key
+    and value projections and stores nothing; its schedule entry names the entry whose plane it reads
+    (``models.base.ScheduleEntry.source``), which holds keys and values of the same heads and widths.  A layer whose plane
+    is read by layers with wider windows keeps as much as the widest of them sees (``cache_window``).
+
+    Tensor names below the prefix: ``q, k, v, o`` (stored (out, in)) and ``sink``."""
+
+    graph_safe = True
+    fuses_residual = True
+
+    def __init__(self, width: int, num_heads: int, kv_heads: int, dim: int, v_dim: int, scale: float, eps: float, position,
+                 window: Optional[int] = None, has_sink: bool = True, qk_norm: bool = True, reads_cache: bool = False,
+                 cache_window=OWN_WINDOW, prefix: str = ""):
+        super().__init__(prefix)
+        if num_heads % kv_heads:
+            raise ValueError(f"{num_heads} query heads are not a multiple of {kv_heads} kv heads")
+        self.width, self.num_heads, self.kv_heads, self.dim, self.v_dim = width, num_heads, kv_heads, dim, v_dim
+        self.scale, self.eps, self.position, self.window = float(scale), float(eps), position, window
+        self.has_sink, self.qk_norm, self.reads_cache = has_sink, qk_norm, reads_cache
+        self.cache_window = window if cache_window == OWN_WINDOW else cache_window
+        if self.cache_window is not None and (window is None or window > self.cache_window):
+            raise ValueError(f"a window of {window} keys over a plane that keeps {self.cache_window}")
+        self.nq, self.nk, self.nv, self.no = num_heads * dim, kv_heads * dim, kv_heads * v_dim, num_heads * v_dim
+        self.w_in = self.w_o = self.sink = None
+
+    @classmethod
+    def from_config(cls, cfg, prefix: str, layer_index: int, lag: int = 0, position=None, cache_window=OWN_WINDOW):
+        m = cfg.layers[layer_index]["mixer"]
+        mask = m.get("mask")
+        return cls(cfg.hidden_size, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], cfg.norm_eps, position,
+                   window=mask["size"] if mask else None, reads_cache=m.get("kv_from") is not None,
+                   cache_window=cache_window, prefix=prefix)
+
+    def children(self):
+        return (self.position,) if self.position is not None else ()
+
+    def kv_spec(self) -> KVSpec:
+        return KVSpec(self.kv_heads, self.dim, self.cache_window, 0, k_dim=self.dim, v_dim=self.v_dim)
+
+    def step_planners(self):
+        return (window_plan.planner(self.num_heads // self.kv_heads),)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        specs = {"q": WeightSpec((self.nq, self.width))}
+        if not self.reads_cache:
+            specs.update({"k": WeightSpec((self.nk, self.width)), "v": WeightSpec((self.nv, self.width))})
+        specs["o"] = WeightSpec((self.width, self.no))
+        if self.has_sink:
+            specs["sink"] = WeightSpec((self.num_heads,), init="uniform", lo=-1.0, hi=1.0)
+        return specs
+
+    def load(self, tensors, ctx: BuildContext) -> None:
+        p = self.prefix
+        names = ("q",) if self.reads_cache else ("q", "k", "v")
+        w = torch.cat([tensors[p + n] for n in names], dim=0).to(ctx.dtype)
+        cols = w.shape[0]
+        w_in = torch.zeros((self.width, pad8(cols)), dtype=ctx.dtype)        # rows of the product start on 16-byte boundaries
+        w_in[:, :cols] = w.t()
+        self.w_in = w_in.to(ctx.device).contiguous()
+        self.w_o = tensors[p + "o"].to(device=ctx.device, dtype=ctx.dtype).t().contiguous()
+        if self.has_sink:
+            self.sink = tensors[p + "sink"].to(device=ctx.device, dtype=torch.float32).contiguous()
+
+    def forward(self, x, step, binding: LayerBinding, residual=None):
+        n = x.shape[0]
+        g = binding.kv_group
+        table, page_size = step.block_tables[g], step.page_sizes[g]
+        proj = ops.gemm(x, self.w_in)
+        pos = self.position
+        ops.rotate_norm_store(proj, self.num_heads, 0 if self.reads_cache else self.kv_heads, self.dim, self.v_dim,
+                              pos.cos if pos is not None else None, pos.sin if pos is not None else None,
+                              pos.interleaved if pos is not None else True, self.qk_norm, self.eps, binding.k_pages,
+                              binding.v_pages, table, step.positions, step.row_slot, page_size, step.fault)
+        out = torch.empty((n, self.no), dtype=x.dtype, device=x.device)
+        ops.window_attention(proj[:, :self.nq], None, out, binding.k_pages, binding.v_pages, table, step.positions,
+                             step.row_slot, self.num_heads, page_size, self.window, self.scale, None, None, step.fault, step,
+                             sink=self.sink)
+        return ops.gemm(out, self.w_o, sink=residual)
+
+
+register_part("mixer", "normed_rotary_attention", NormedRotaryAttention)

@@ -123,6 +123,8 @@ class RMSNormGrouped(Norm):
     ``add_norm_pair(residual, delta, delta_b, other)`` also writes the output of a second norm of the same groups and eps
     (``other``), whose factors are the same."""
 
+    takes_two_updates = True
+
     def __init__(self, width: int, groups: int, eps: float, prefix: str = "", weight_name: str = "weight"):
         super().__init__(prefix)
         if groups <= 0 or width % groups:
@@ -169,6 +171,44 @@ class RMSNormGrouped(Norm):
         return values
 
 
+class LayerNorm(Norm):
+    """``y = (x - mean) / sqrt(variance + eps) * w + b`` in float32, the variance being the mean of the squared deviations and
+    eps inside the root.  Tensor names: ``weight_name`` and ``weight_name + ".b"``.  ``add_norm(residual, delta, delta_b=...)``
+    adds up to two pending updates before it normalises, in the same kernel."""
+
+    takes_two_updates = True
+
+    def __init__(self, width: int, eps: float, prefix: str = "", weight_name: str = "weight"):
+        super().__init__(prefix)
+        self.width, self.eps, self.weight_name = width, float(eps), weight_name
+        self.scale: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self.out_dtype = torch.float32
+
+    @classmethod
+    def from_config(cls, cfg, prefix: str):
+        return cls(cfg.hidden_size, cfg.norm_eps, prefix=prefix)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.weight_name: WeightSpec((self.width,), init="ones_normal"), self.weight_name + ".b": WeightSpec((self.width,))}
+
+    def load(self, tensors, ctx: BuildContext) -> None:
+        f32 = dict(device=ctx.device, dtype=torch.float32)
+        self.scale = tensors[self.prefix + self.weight_name].to(**f32).contiguous()
+        self.bias = tensors[self.prefix + self.weight_name + ".b"].to(**f32).contiguous()
+        self.out_dtype = ctx.dtype
+
+    def add_norm(self, residual: torch.Tensor, delta: Optional[torch.Tensor], delta_norm=None, delta_b=None) -> torch.Tensor:
+        if delta_norm is not None:
+            raise ValueError("the layer norm takes updates as they are")
+        out = torch.empty(residual.shape, dtype=self.out_dtype, device=residual.device)
+        return ops.add_layer_norm(residual, delta, delta_b, self.scale, self.bias, self.eps, out)
+
+    def forward(self, residual: torch.Tensor) -> torch.Tensor:
+        return self.add_norm(residual, None)
+
+
+register_part("norm", "layer_norm", LayerNorm)
 register_part("norm", "rmsnorm_grouped", RMSNormGrouped)
 register_part("norm", "rmsnorm_l2", RMSNormL2)
 register_part("norm", "rmsnorm_mean_eps", RMSNormMeanEps)

@@ -15,12 +15,15 @@ class RotaryHalf(PositionEncoding):
     (``precompute_rope_fast`` and ``rotate_half``, main_models_new.py:63-80):
     angle[pos, i] = pos * theta^(-2i/rot).  Tables of cos and sin, ``[positions, rot/2]``
     float32; the angles are formed in float64 on the host so that a table entry is the
-    correctly rounded value.  ``rotary_dim`` below the head size leaves the rest of each
+    correctly rounded value.  ``factor`` divides every angle (positions interpolated linearly).  ``rotary_dim`` below the head size leaves the rest of each
     head unrotated; ``interleaved`` pairs (2i, 2i+1) instead."""
 
     def __init__(self, head_dim: int, theta: float, max_positions: int, rotary_dim: Optional[int] = None,
-                 interleaved: bool = False, prefix: str = ""):
+                 interleaved: bool = False, prefix: str = "", factor: float = 1.0):
         super().__init__(prefix)
+        if not factor > 0:
+            raise ValueError(f"a rotation's angles are divided by a positive number, not {factor}")
+        self.factor = float(factor)
         self.head_dim = head_dim
         self.rotary_dim = head_dim if rotary_dim is None else rotary_dim
         if self.rotary_dim % 2 or not (0 < self.rotary_dim <= head_dim):
@@ -37,7 +40,7 @@ class RotaryHalf(PositionEncoding):
 
     def tables(self):
         i = torch.arange(0, self.rotary_dim // 2, dtype=torch.float64)
-        inv = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / self.rotary_dim)
+        inv = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / self.rotary_dim) / self.factor
         ang = torch.outer(torch.arange(self.max_positions, dtype=torch.float64), inv)
         return torch.cos(ang).to(torch.float32), torch.sin(ang).to(torch.float32)
 
@@ -65,8 +68,8 @@ class RotaryInterleaved(RotaryHalf):
     """Pairs (2i, 2i+1) instead of (i, i + rot/2); the same angles."""
 
     def __init__(self, head_dim: int, theta: float, max_positions: int, rotary_dim: Optional[int] = None,
-                 prefix: str = ""):
-        super().__init__(head_dim, theta, max_positions, rotary_dim, interleaved=True, prefix=prefix)
+                 prefix: str = "", factor: float = 1.0):
+        super().__init__(head_dim, theta, max_positions, rotary_dim, interleaved=True, prefix=prefix, factor=factor)
 
 
 class RotaryRescaled(RotaryHalf):

@@ -74,7 +74,7 @@ class ResidualStream:
             if ready.norm is norm:
                 return ready if scaled else ready.dense()
             return norm.add_norm(self.values, None)        # made for another norm: the stream itself is whole
-        if self.pending_b is not None and (self.pending_post is not None or not hasattr(norm, "add_norm_pair")):
+        if self.pending_b is not None and (self.pending_post is not None or not norm.takes_two_updates):
             ops.residual_add(self.values, self.pending_b)
             self.pending_b = None
         delta, self.pending = self.pending, None
