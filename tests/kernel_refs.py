@@ -546,7 +546,7 @@ def add_layer_norm(residual, delta_a, delta_b, w, b, eps, out):
 
 
 def rotate_norm_store(qkv, num_heads, kv_heads, dim, v_dim, cos, sin, interleaved, norm, eps, k_pages, v_pages, block_table,
-                      positions, row_slot, page_size, fault):
+                      positions, row_slot, page_size, fault, permuted=False):
     def prepared(z, pos):               # (heads, dim)
         out = z.to(torch.float32).clone()
         if cos is not None:
@@ -569,8 +569,9 @@ def rotate_norm_store(qkv, num_heads, kv_heads, dim, v_dim, cos, sin, interleave
         qkv[r, :H * dim] = qk[:H].reshape(-1)
         if G:
             page, at = int(block_table[slot, pos // page_size]), pos % page_size
-            k_pages[page, :, at] = qk[H:].to(k_pages.dtype)
-            v_pages[page, :, at] = qkv[r, (H + G) * dim:(H + G) * dim + G * v_dim].view(G, v_dim).to(v_pages.dtype)
+            row = (lambda z: cache_row(z.contiguous(), pos)) if permuted else (lambda z: z)
+            k_pages[page, :, at] = row(qk[H:].to(k_pages.dtype))
+            v_pages[page, :, at] = row(qkv[r, (H + G) * dim:(H + G) * dim + G * v_dim].view(G, v_dim).to(v_pages.dtype))
 
 
 def scaled_sum(a, scale_a, b, scale_b):
@@ -679,15 +680,21 @@ def _unrotate_rows(x, positions):
     return out.permute(0, 2, 1, 3).reshape(L, kvh, hd)
 
 
-def rotary_fusable(q, step, num_heads, kv_heads, head_dim):
+def rotary_fusable(q, step, num_heads, kv_heads, head_dim, pairs=False):
     """On the CPU every decode step takes the path where attention does the rotary encoding and the
     cache write itself, so that its plumbing runs in the CPU tests too."""
     return step is not None and getattr(step, "decode_only", False)
 
 
 def paged_attention(q, out, plane, block_table, positions, row_slot, num_heads, kv_heads, head_dim, page_size,
-                    window, fault, step=None, rotary=None, write_kv=True):
-    if rotary is not None:
+                    window, fault, step=None, rotary=None, write_kv=True, scale=None, sink=None):
+    from tiny_inference_server_b200.kernels import ops
+    scale = 1.0 / math.sqrt(head_dim) if scale is None else scale
+    if isinstance(rotary, ops.PairRotary):
+        rotate_norm_store(q, num_heads, kv_heads if write_kv else 0, head_dim, head_dim, rotary.cos, rotary.sin, True,
+                          rotary.norm_eps is not None, rotary.norm_eps or 0.0, plane[:, 0], plane[:, 1], block_table, positions,
+                          row_slot, page_size, fault, permuted=True)
+    elif rotary is not None:
         rope_kv_write(q, positions, row_slot, rotary[0], rotary[1], plane, block_table, num_heads, kv_heads, head_dim,
                       page_size, fault, write_kv=write_kv)
     n = q.shape[0]
@@ -705,8 +712,10 @@ def paged_attention(q, out, plane, block_table, positions, row_slot, num_heads, 
         k = k.repeat_interleave(g, dim=1)
         v = v.repeat_interleave(g, dim=1)
         qq = q[r, :hq].to(torch.float32).view(num_heads, head_dim)
-        s = torch.einsum("hd,khd->hk", qq, k) / math.sqrt(head_dim)
-        p = torch.softmax(s, dim=-1)
+        s = torch.einsum("hd,khd->hk", qq, k) * scale
+        if sink is not None:
+            s = torch.cat([s, sink.to(torch.float32)[:, None]], dim=1)
+        p = torch.softmax(s, dim=-1)[:, :k.shape[0]]
         out[r] = torch.einsum("hk,khd->hd", p, v).reshape(-1).to(out.dtype)
     return out
 

@@ -54,6 +54,10 @@ constexpr int DTILES = HD / 8;       // n8 tiles of the output
 static_assert(HD % 16 == 0 && HD >= 16 && HD <= 256, "head size must be a multiple of 16 in 16..256");
 
 enum { MODE_ROWS = 0, MODE_KEYS = 1 };
+// What the kernel does with a decode row's queries and key before they meet (FUSED below): nothing; a rotation of the whole
+// head with element i paired with i + HD/2; a rotation of the first elements with 2i paired with 2i + 1 and, if asked, the
+// division of the head by its root mean square.
+enum { FUSED_NONE = 0, FUSED_HALVES = 1, FUSED_PAIRS = 2 };
 
 struct AttnParams {
     const bf16* q; int q_stride;
@@ -72,6 +76,9 @@ struct AttnParams {
     int recv_offset;        // bytes from the start of shared memory to where the cluster's partial results land
     // rotary encoding and cache write done by this kernel (decode rows; see FUSED below)
     const float* rope_cos; const float* rope_sin;   // [positions][HD/2]
+    int rope_rot;           // FUSED_PAIRS: how many elements of a head are rotated (tables [positions][rope_rot / 2]),
+    int rope_norm; float rope_eps;      // and whether the head is then divided by its root mean square
+    const float* sink;      // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     bf16* plane_w;          // the plane, writable: where the row's key and value go (null: another entry fills it)
     TIS_TIMELINE_MEMBER     // (instrumented builds only; the decode kernel's stamps: 0 entry, 1 before and 2 after the
                             //  dependency wait, 3 first tile landed, 4 last tile landed, 5 loop done, 6 partial results
@@ -194,6 +201,78 @@ __device__ __forceinline__ void load_tile(bf16* stage, unsigned long long* bar, 
         atomicExch(p.fault, 3);
     }
     mbar_arrive(bar);
+}
+
+// The keyless term of a row's softmax, added to a finished numerator and denominator whose maximum (in units of log2) is mt.
+__device__ __forceinline__ void add_sink(float& num, float& den, float mt, float sink) {
+    const float s2 = sink * 1.4426950408889634f;
+    const float m = fmaxf(mt, s2);
+    const float f = mt == -INFINITY ? 0.f : fast_exp2(mt - m);
+    num *= f;
+    den = den * f + fast_exp2(s2 - m);
+}
+
+// FUSED_PAIRS: the queries' fragments rotated and normed in registers.  Columns 2t and 2t + 1 of a fragment are a rotation
+// pair; a row's columns lie in the four lanes that share it.  A rotation keeps the sum of squares, so the norm's factor
+// comes from the values as they are.  cs, sn: the position's cosines and sines.
+template <int NR>
+__device__ __forceinline__ void rotate_norm_fragments(unsigned (&qa)[KSTEPS][4], const AttnParams& p, const float* cs,
+                                                      const float* sn, const bool (&valid)[2], int t_lane) {
+    float f[2] = {1.f, 1.f};
+    if (p.rope_norm) {
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            float ss = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < KSTEPS; ++kk)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qa[kk][2 * hf + i]));
+                    ss = fmaf(x.x, x.x, fmaf(x.y, x.y, ss));
+                }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            f[i] = valid[i] ? 1.f / sqrtf(ss / (float)HD + p.rope_eps) : 0.f;
+        }
+    }
+#pragma unroll
+    for (int kk = 0; kk < KSTEPS; ++kk)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            const int pair = kk * 8 + hf * 4 + t_lane;
+            float c = 1.f, s = 0.f;
+            if (2 * pair < p.rope_rot) { c = cs[pair]; s = sn[pair]; }
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qa[kk][2 * hf + i]));
+                qa[kk][2 * hf + i] = pack_bf16((x.x * c - x.y * s) * f[i], (x.y * c + x.x * s) * f[i]);
+            }
+        }
+}
+
+// FUSED_PAIRS: chunk `lane` (of NCH; the other lanes hold nothing) of the row's own key, rotated and normed, by one warp.
+__device__ __forceinline__ void own_key_pairs(float (&o)[8], const bf16* krow, const AttnParams& p, const float* cs,
+                                              const float* sn, int lane) {
+    float x[8];
+    const bool in = lane < NCH;
+    if (in) Vec16<bf16>::load(krow + lane * 8, x);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int pair = lane * 4 + j;
+        float c = 1.f, s = 0.f;
+        if (in && 2 * pair < p.rope_rot) { c = cs[pair]; s = sn[pair]; }
+        const float a = in ? x[2 * j] : 0.f, b = in ? x[2 * j + 1] : 0.f;
+        o[2 * j] = a * c - b * s;
+        o[2 * j + 1] = b * c + a * s;
+        ss = fmaf(a, a, fmaf(b, b, ss));
+    }
+    if (p.rope_norm) {
+        ss = warp_sum(ss);
+        const float f = 1.f / sqrtf(ss / (float)HD + p.rope_eps);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o[j] *= f;
+    }
 }
 
 // NR: packed rows a thread keeps softmax state for.  2: rows g and g+8 of the 16 a warp owns.
@@ -320,17 +399,18 @@ __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, uns
                 acc += from[sp * step_sp + c] * f;
             }
         }
+        if (p.sink != nullptr) add_sink(acc, lsum, mt, p.sink[kvh * G + g]);
         p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
             __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
     }
     TIS_STAMP(p, 8);
 }
 
-template <int MODE, int NR, int NG, bool FUSED = false>
+template <int MODE, int NR, int NG, int FUSED = FUSED_NONE>
 __global__ void __launch_bounds__(NTHREADS * NG)
 attn_mma_kernel(const AttnParams p) {
     static_assert(NG == 1 || MODE == MODE_ROWS, "key groups are for row tiles");
-    static_assert(!FUSED || (MODE == MODE_KEYS && HD % 32 == 0), "the fused rotary path is for decode rows");
+    static_assert(!FUSED || (MODE == MODE_KEYS && (FUSED == FUSED_PAIRS || HD % 32 == 0)), "the fused rotary path is for decode rows");
     constexpr int NT = MODE == MODE_ROWS ? 8 : 2;        // n8 key tiles a warp scores per staged tile
     constexpr int KB = MODE == MODE_ROWS ? 4 : 1;        // k16 key blocks a warp multiplies with V
     constexpr int STAGE_ELEMS = 2 * KT * RS;
@@ -401,8 +481,10 @@ attn_mma_kernel(const AttnParams p) {
         const int pos_first = p.positions[row0 + first], pos_last = p.positions[row0 + rows - 1];
         range_hi = pos_last + 1;
         range_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
-        range_lo = max(range_lo, split * p.keys_per_split);
-        range_hi = min(range_hi, (split + 1) * p.keys_per_split);
+        // the splits share out the keys from the window's first tile on
+        const int base = p.window > 0 ? range_lo / KT * KT : 0;
+        range_lo = max(range_lo, base + split * p.keys_per_split);
+        range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
     const bool empty = first < 0 || range_lo >= range_hi;
 
@@ -460,7 +542,12 @@ attn_mma_kernel(const AttnParams p) {
                 qa[kk][2 + i] = w1;
             }
         }
-        if (FUSED) {
+        if (FUSED == FUSED_PAIRS) {
+            const int pos = p.positions[row0 + rows - 1];
+            rotate_norm_fragments<NR>(qa, p, p.rope_cos + (size_t)pos * (p.rope_rot / 2), p.rope_sin + (size_t)pos * (p.rope_rot / 2),
+                                      valid, t_lane);
+        }
+        if (FUSED == FUSED_HALVES) {
             // rotate the queries: column c of a head pairs with c + HD/2, which the same thread holds KSTEPS/2
             // fragments further on; one position for the whole tile (it has one row)
             const int pos = p.positions[row0 + rows - 1];
@@ -525,7 +612,16 @@ attn_mma_kernel(const AttnParams p) {
                     : p.plane_w + (((size_t)own_page * 2) * p.KVH + kvh) * (size_t)p.page_size * HD +
                       (size_t)(own_pos % p.page_size) * HD;
                 bf16* v_gl = own_page < 0 ? nullptr : k_gl + (size_t)p.KVH * p.page_size * HD;
-                if (warp == 0 && lane < NCH / 2) {
+                if (FUSED == FUSED_PAIRS && warp == 0) {
+                    float o1[8];
+                    own_key_pairs(o1, krow, p, p.rope_cos + (size_t)own_pos * (p.rope_rot / 2),
+                                  p.rope_sin + (size_t)own_pos * (p.rope_rot / 2), lane);
+                    if (lane < NCH) {
+                        const int ch1 = cache_chunk(lane, own_pos, NCH) * 8;
+                        Vec16<bf16>::store(k_sm + ch1, o1);
+                        if (k_gl != nullptr) Vec16<bf16>::store(k_gl + ch1, o1);
+                    }
+                } else if (FUSED == FUSED_HALVES && warp == 0 && lane < NCH / 2) {
                     const int c = lane;
                     float x1[8], x2[8], o1[8], o2[8];
                     Vec16<bf16>::load(krow + c * 8, x1);
@@ -733,6 +829,7 @@ attn_mma_kernel(const AttnParams p) {
                     acc += mo[(w * 16 + m) * HD + d] * f;
                 }
             }
+            if (p.num_splits == 1 && p.sink != nullptr) add_sink(acc, lt, mt, p.sink[hq]);
             const float val = lt > 0.f ? acc / lt : 0.f;
             if (p.num_splits == 1) {
                 p.out[(size_t)row * p.out_stride + (size_t)hq * HD + d] = __float2bfloat16_rn(val);
@@ -750,8 +847,13 @@ attn_mma_kernel(const AttnParams p) {
             const int r = m / G, g = m - r * G;
             if (r >= rows) continue;
             const int row = row0 + r, hq = kvh * G + g;
-            const float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
+            float inv = l_run[i] > 0.f ? 1.f / l_run[i] : 0.f;
             if (p.num_splits == 1) {
+                if (p.sink != nullptr) {
+                    float num = 1.f, den = l_run[i];
+                    add_sink(num, den, m_run[i], p.sink[hq]);
+                    inv = den > 0.f ? num / den : 0.f;
+                }
                 bf16* dst = p.out + (size_t)row * p.out_stride + (size_t)hq * HD;
 #pragma unroll
                 for (int d = 0; d < DTILES; ++d)
@@ -800,6 +902,7 @@ attn_mma_kernel(const AttnParams p) {
                         acc += w * cluster.map_shared_rank(cm_o, sp)[m * HD + d];
                     }
                 }
+                if (p.sink != nullptr) add_sink(acc, wsum, mt, p.sink[kvh * G + g]);
                 p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
                     __float2bfloat16_rn(wsum > 0.f ? acc / wsum : 0.f);
             }
@@ -868,10 +971,10 @@ __device__ __forceinline__ void load_tile_warp(bf16* stage, unsigned long long* 
     mbar_arrive(bar);
 }
 
-template <int NR, bool FUSED>
+template <int NR, int FUSED>
 __global__ void __launch_bounds__(DEC_THREADS, HD <= 128 ? 2 : 1)
 attn_decode_kernel(const AttnParams p) {
-    static_assert(!FUSED || HD % 32 == 0, "the fused rotary path rotates pairs of k16 fragments");
+    static_assert(FUSED != FUSED_HALVES || HD % 32 == 0, "the fused rotary path rotates pairs of k16 fragments");
     constexpr int NT = 2;                                // n8 key tiles a warp scores per staged tile
     constexpr int STAGE_ELEMS = 2 * KT * RS;
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -932,8 +1035,10 @@ attn_decode_kernel(const AttnParams p) {
         const int pos_first = first == rows - 1 ? pos_last : p.positions[row0 + first];
         range_hi = pos_last + 1;
         range_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
-        range_lo = max(range_lo, split * p.keys_per_split);
-        range_hi = min(range_hi, (split + 1) * p.keys_per_split);
+        // the splits share out the keys from the window's first tile on
+        const int base = p.window > 0 ? range_lo / KT * KT : 0;
+        range_lo = max(range_lo, base + split * p.keys_per_split);
+        range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
     const bool none = first < 0 || range_lo >= range_hi;
     const int* bt = p.block_table + (size_t)(slot >= 0 ? slot : 0) * p.bt_stride;
@@ -980,6 +1085,11 @@ attn_decode_kernel(const AttnParams p) {
         // shared memory while they would only wait (in registers they would not fit beside the queries)
         if (FUSED && ntiles > 0) {
             const int pos = p.positions[row0 + rows - 1];
+            if (FUSED == FUSED_PAIRS) {
+                const int half = p.rope_rot / 2;
+                for (int i = tid; i < 2 * half; i += NTHREADS)
+                    rope_sh[i] = i < half ? p.rope_cos[(size_t)pos * half + i] : p.rope_sin[(size_t)pos * half + i - half];
+            } else
             for (int i = tid; i < HD / 4; i += NTHREADS) {              // HD / 2 cosines and as many sines, four a thread
                 const float* src = i < HD / 8 ? p.rope_cos + (size_t)pos * (HD / 2) + 4 * i
                                               : p.rope_sin + (size_t)pos * (HD / 2) + 4 * (i - HD / 8);
@@ -1006,7 +1116,8 @@ attn_decode_kernel(const AttnParams p) {
                     qa[kk][2 + i] = w1;
                 }
             }
-            if (FUSED) {
+            if (FUSED == FUSED_PAIRS) rotate_norm_fragments<NR>(qa, p, rope_sh, rope_sh + p.rope_rot / 2, valid, t_lane);
+            if (FUSED == FUSED_HALVES) {
                 const float* cs = rope_sh;
                 const float* sn = rope_sh + HD / 2;
 #pragma unroll
@@ -1043,7 +1154,15 @@ attn_decode_kernel(const AttnParams p) {
                         : p.plane_w + (((size_t)own_page * 2) * p.KVH + kvh) * (size_t)p.page_size * HD +
                           (size_t)(own_pos % p.page_size) * HD;
                     bf16* v_gl = own_page < 0 ? nullptr : k_gl + (size_t)p.KVH * p.page_size * HD;
-                    if (warp == 0 && lane < NCH / 2) {
+                    if (FUSED == FUSED_PAIRS && warp == 0) {
+                        float o1[8];
+                        own_key_pairs(o1, krow, p, rope_sh, rope_sh + p.rope_rot / 2, lane);
+                        if (lane < NCH) {
+                            const int ch1 = cache_chunk(lane, own_pos, NCH) * 8;
+                            Vec16<bf16>::store(k_sm + ch1, o1);
+                            if (k_gl != nullptr) Vec16<bf16>::store(k_gl + ch1, o1);
+                        }
+                    } else if (FUSED == FUSED_HALVES && warp == 0 && lane < NCH / 2) {
                         const int c = lane;
                         float x1[8], x2[8], o1[8], o2[8];
                         Vec16<bf16>::load(krow + c * 8, x1);
@@ -1173,7 +1292,8 @@ attn_decode_kernel(const AttnParams p) {
 // out[row, head] = sum_s w_s * part_o[row, head, s],  w_s = 2^(lse_s - max) / sum, for the rows of one tile
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                   bf16* __restrict__ out, int out_stride, const int* __restrict__ tile_row0,
-                                  const int* __restrict__ tile_rows, int H, int num_splits) {
+                                  const int* __restrict__ tile_rows, int H, int num_splits,
+                                  const float* __restrict__ sink) {
     const int tile = blockIdx.y, hq = blockIdx.x;
     const int row0 = tile_row0 != nullptr ? tile_row0[tile] : tile, rows = tile_rows != nullptr ? tile_rows[tile] : 1;
     for (int r = 0; r < rows; ++r) {
@@ -1192,6 +1312,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
                     acc += w * part_o[(pr + s) * HD + d];
                 }
             }
+            if (sink != nullptr) add_sink(acc, wsum, mt, sink[hq]);
             out[(size_t)row * out_stride + (size_t)hq * HD + d] = __float2bfloat16_rn(wsum > 0.f ? acc / wsum : 0.f);
         }
     }
@@ -1245,10 +1366,13 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
                        const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
                        int max_tile_rows, int n_rows, int H, int KVH, int page_size, int window, float scale,
                        int keys_per_split, int num_splits, float* scratch, int* fault, cudaStream_t stream,
-                       const float* rope_cos, const float* rope_sin, int write_kv) {
+                       const float* rope_cos, const float* rope_sin, int write_kv, int rope_kind = FUSED_NONE,
+                       int rope_rot = 0, int rope_norm = 0, float rope_eps = 0.f, const float* sink = nullptr) {
     if (num_tiles <= 0) return TIS_OK;
-    const bool fused = rope_cos != nullptr;
-    if (fused && (mode != MODE_KEYS || max_tile_rows != 1 || HD % 32 != 0 || rope_sin == nullptr)) {
+    const bool fused = rope_kind != FUSED_NONE, pairs_kind = rope_kind == FUSED_PAIRS;
+    if (fused && (mode != MODE_KEYS || max_tile_rows != 1 || (!pairs_kind && HD % 32 != 0) ||
+                  ((rope_rot > 0 || !pairs_kind) && (rope_cos == nullptr || rope_sin == nullptr)) || rope_rot < 0 || rope_rot % 2 ||
+                  rope_rot > HD)) {
         tis_set_error("attention: the rotary encoding is done inside the kernel only for tiles of one row (got %d) in "
                       "keys mode and head sizes that are multiples of 32 (this library: %d)", max_tile_rows, HD);
         return TIS_BAD_SIZE;
@@ -1286,7 +1410,8 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
     p.part_lse = scratch ? scratch + (size_t)n_rows * H * num_splits * HD : nullptr;
     p.cluster_merge = (num_splits > 1 && num_splits <= (mode == MODE_KEYS && scratch == nullptr ? MAX_CLUSTER : 8)) ? 1 : 0;
     p.fault = fault;
-    p.rope_cos = rope_cos; p.rope_sin = rope_sin;
+    p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.rope_rot = rope_rot; p.rope_norm = rope_norm; p.rope_eps = rope_eps;
+    p.sink = sink;
     p.plane_w = (fused && write_kv) ? (bf16*)plane : nullptr;
     TIS_TIMELINE_TAKE(p);
     // decode tiles go to the kernel with a producer warp where its layout allows (page segments: two lanes each)
@@ -1351,20 +1476,28 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
         cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
 #if TIS_HD % 32 == 0
-        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_HALVES>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_HALVES>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
 #endif
-        cudaFuncSetAttribute(attn_decode_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_decode_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_decode_kernel<1, false>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        cudaFuncSetAttribute(attn_decode_kernel<2, false>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_PAIRS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_PAIRS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_PAIRS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_PAIRS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_PAIRS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_PAIRS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_PAIRS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_PAIRS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_NONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_NONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_NONE>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_NONE>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
 #if TIS_HD % 32 == 0
-        cudaFuncSetAttribute(attn_decode_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_decode_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(attn_decode_kernel<1, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        cudaFuncSetAttribute(attn_decode_kernel<2, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(attn_decode_kernel<1, FUSED_HALVES>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_decode_kernel<2, FUSED_HALVES>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
 #endif
         cudaGetLastError();
         if (3 * smem_bytes(MODE_ROWS) <= 227 * 1024)
@@ -1413,17 +1546,22 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
                 cfg.numAttrs = ++na;
             }
             const bool nr1 = max_tile_rows > 0 && max_tile_rows * G <= 8;
+            if (pairs_kind && nr1) cudaLaunchKernelEx(&cfg, attn_decode_kernel<1, FUSED_PAIRS>, p);
+            else if (pairs_kind) cudaLaunchKernelEx(&cfg, attn_decode_kernel<2, FUSED_PAIRS>, p);
+            else
 #if TIS_HD % 32 == 0
-            if (fused && nr1) cudaLaunchKernelEx(&cfg, attn_decode_kernel<1, true>, p);
-            else if (fused) cudaLaunchKernelEx(&cfg, attn_decode_kernel<2, true>, p);
+            if (fused && nr1) cudaLaunchKernelEx(&cfg, attn_decode_kernel<1, FUSED_HALVES>, p);
+            else if (fused) cudaLaunchKernelEx(&cfg, attn_decode_kernel<2, FUSED_HALVES>, p);
             else
 #endif
-            if (nr1) cudaLaunchKernelEx(&cfg, attn_decode_kernel<1, false>, p);
-            else cudaLaunchKernelEx(&cfg, attn_decode_kernel<2, false>, p);
+            if (nr1) cudaLaunchKernelEx(&cfg, attn_decode_kernel<1, FUSED_NONE>, p);
+            else cudaLaunchKernelEx(&cfg, attn_decode_kernel<2, FUSED_NONE>, p);
         }
+        else if (pairs_kind && G <= 8) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_PAIRS>, p);
+        else if (pairs_kind) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_PAIRS>, p);
 #if TIS_HD % 32 == 0
-        else if (fused && G <= 8) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 1, 1, true>, p);
-        else if (fused) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 2, 1, true>, p);
+        else if (fused && G <= 8) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 1, 1, FUSED_HALVES>, p);
+        else if (fused) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 2, 1, FUSED_HALVES>, p);
 #endif
         else if (max_tile_rows > 0 && max_tile_rows * G <= 8) cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 1, 1>, p);
         else cudaLaunchKernelEx(&cfg, attn_mma_kernel<MODE_KEYS, 2, 1>, p);
@@ -1433,7 +1571,7 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
     if (num_splits > 1 && !p.cluster_merge) {
         dim3 mg(H, num_tiles);
         attn_merge_kernel<<<mg, HD < 128 ? (HD < 32 ? 32 : HD) : 128, 0, stream>>>(p.part_o, p.part_lse, (bf16*)out, out_stride,
-                                                                                  tile_row0, tile_rows, H, num_splits);
+                                                                                  tile_row0, tile_rows, H, num_splits, p.sink);
         st = tis_check_launch("attn_merge");
     }
     return st;
@@ -1449,18 +1587,33 @@ TIS_API int tis_attn_mma(int mode, const void* q, int q_stride, void* out, int o
                        keys_per_split, num_splits, scratch, fault, stream, nullptr, nullptr, 0);
 }
 
+// The same with `sink` (null: none): exp(sink[h]) is one more term of head h's softmax denominator.
+TIS_API int tis_attn_mma_sink(int mode, const void* q, int q_stride, void* out, int out_stride, const void* plane,
+                              const int* block_table, int bt_stride, int num_pages, const int* positions,
+                              const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
+                              int max_tile_rows, int n_rows, int H, int KVH, int page_size, int window, float scale,
+                              int keys_per_split, int num_splits, float* scratch, const float* sink, int* fault,
+                              cudaStream_t stream) {
+    return attn_launch(mode, q, q_stride, out, out_stride, plane, block_table, bt_stride, num_pages, positions, row_slot,
+                       tile_row0, tile_rows, num_tiles, max_tile_rows, n_rows, H, KVH, page_size, window, scale,
+                       keys_per_split, num_splits, scratch, fault, stream, nullptr, nullptr, 0, FUSED_NONE, 0, 0, 0.f, sink);
+}
+
 // Decode rows (tiles of one row, keys mode) whose rotary encoding and cache write this kernel does itself:
 // `qkv` rows are [H*HD queries | KVH*HD keys | KVH*HD values] as the projection left them (only the queries
 // when write_kv is 0: another entry of the schedule fills the plane); cos/sin [positions][HD/2] float32,
-// half-split pairs, the whole head rotated.  At most eight key splits (they merge inside a cluster).
+// half-split pairs, the whole head rotated (kind 1); or kind 2: neighbouring elements paired, the first `rot` of a head rotated
+// (tables [positions][rot/2], may be null for rot 0) and, with `norm`, the head then divided by its root mean square (`eps`
+// inside the root).  `sink`: as in tis_attn_mma_sink.  At most 16 key splits (they merge inside a cluster).
 TIS_API int tis_attn_decode_rope(const void* qkv, int q_stride, void* out, int out_stride, void* plane,
                                  const int* block_table, int bt_stride, int num_pages, const int* positions,
                                  const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
                                  int n_rows, int H, int KVH, int page_size, int window, float scale,
                                  int keys_per_split, int num_splits, const float* rope_cos, const float* rope_sin,
-                                 int write_kv, int* fault, cudaStream_t stream) {
-    if (rope_cos == nullptr || rope_sin == nullptr) {
-        tis_set_error("attn_decode_rope: no rotary tables");
+                                 int write_kv, int kind, int rot, int norm, float eps, const float* sink, int* fault,
+                                 cudaStream_t stream) {
+    if (kind != FUSED_HALVES && kind != FUSED_PAIRS) {
+        tis_set_error("attn_decode_rope: rotation kind %d", kind);
         return TIS_BAD_SIZE;
     }
     if (num_splits > MAX_CLUSTER) {
@@ -1469,7 +1622,7 @@ TIS_API int tis_attn_decode_rope(const void* qkv, int q_stride, void* out, int o
     }
     return attn_launch(MODE_KEYS, qkv, q_stride, out, out_stride, plane, block_table, bt_stride, num_pages, positions,
                        row_slot, tile_row0, tile_rows, num_tiles, 1, n_rows, H, KVH, page_size, window, scale,
-                       keys_per_split, num_splits, nullptr, fault, stream, rope_cos, rope_sin, write_kv);
+                       keys_per_split, num_splits, nullptr, fault, stream, rope_cos, rope_sin, write_kv, kind, rot, norm, eps, sink);
 }
 
 

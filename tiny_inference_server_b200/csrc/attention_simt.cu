@@ -35,7 +35,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
                             const T* __restrict__ plane, const int* __restrict__ block_table, int bt_stride,
                             int num_pages, const int* __restrict__ positions, const int* __restrict__ row_slot,
                             int H, int KVH, int hd, int page_size, int window, float scale,
-                            int* __restrict__ fault) {
+                            const float* __restrict__ sink, int* __restrict__ fault) {
     extern __shared__ float smem[];
     float* qs = smem;                      // hd
     float* ps = smem + hd;                 // SIMT_KEYS
@@ -62,7 +62,8 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
     const size_t v_shift = (size_t)KVH * page_size * hd;
 
     float acc0 = 0.f, acc1 = 0.f;          // dims tid and tid + 128 of the output (hd <= 256)
-    float m = -INFINITY, l = 0.f;
+    // a sink is one more term of the denominator, exp(sink[head]), without a value: maximum and sum start there
+    float m = sink != nullptr ? sink[h] : -INFINITY, l = sink != nullptr ? 1.f : 0.f;
     for (int t0 = lo; t0 < hi; t0 += SIMT_KEYS) {
         const int j = t0 + tid;
         float s = -INFINITY;
@@ -112,7 +113,8 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
 TIS_API int tis_paged_attention_simt(int dtype, const void* q, int q_stride, void* out, int out_stride,
                                      const void* plane, const int* block_table, int bt_stride, int num_pages,
                                      const int* positions, const int* row_slot, int n, int H, int KVH, int hd,
-                                     int page_size, int window, float scale, int* fault, cudaStream_t stream) {
+                                     int page_size, int window, float scale, const float* sink, int* fault,
+                                     cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (hd % 16 || hd <= 0 || hd > 256) {
         tis_set_error("paged_attention: head size %d is not a multiple of 16 in 16..256", hd);
@@ -131,6 +133,6 @@ TIS_API int tis_paged_attention_simt(int dtype, const void* q, int q_stride, voi
     TIS_DISPATCH_DTYPE(dtype, T,
         paged_attention_simt_kernel<T><<<grid, SIMT_KEYS, smem, stream>>>(
             (const T*)q, q_stride, (T*)out, out_stride, (const T*)plane, block_table, bt_stride, num_pages,
-            positions, row_slot, H, KVH, hd, page_size, window, scale, fault));
+            positions, row_slot, H, KVH, hd, page_size, window, scale, sink, fault));
     return tis_check_launch("paged_attention_simt");
 }

@@ -59,6 +59,7 @@ struct TcAttnParams {
     const int* tile_row0; const int* tile_rows; int num_tiles;
     int H, KVH, page_size, window;
     float scale_log2;
+    const float* sink;      // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     int* fault;
 };
 
@@ -332,10 +333,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             const float* mg0 = reinterpret_cast<const float*>(p_smem);
             const float* mg1 = reinterpret_cast<const float*>(p_smem + P_BYTES);
             const float m0 = mg0[r], m1 = mg1[r], l0 = mg0[BM + r], l1 = mg1[BM + r];
-            const float m = fmaxf(m0, m1);
+            const float sink2 = p.sink != nullptr ? p.sink[head] * 1.4426950408889634f : -INFINITY;
+            const float m = fmaxf(fmaxf(m0, m1), sink2);
             const float w0 = m0 == -INFINITY ? 0.f : fast_exp2(m0 - m);
             const float w1 = (T < 2 || m1 == -INFINITY) ? 0.f : fast_exp2(m1 - m);
-            const float l = l0 * w0 + l1 * w1;
+            const float l = l0 * w0 + l1 * w1 + (sink2 == -INFINITY ? 0.f : fast_exp2(sink2 - m));
             const float inv = l > 0.f ? 1.f / l : 0.f;
             constexpr int COLS = HD / 2;                  // this group's share of the columns
 #pragma unroll 1
@@ -378,11 +380,12 @@ TIS_API int tis_attn_tc_supported() { return 1; }
 
 // Attention of `num_tiles` tiles of up to 128 consecutive rows of one request each.  q is
 // (n, >= H*hd) with row stride q_stride, out (n, H*hd); plane is [pages, 2, KVH, page_size, hd];
-// page_size 16, 32, 64 or 128.
+// page_size 16, 32, 64 or 128.  `sink` (null: none): exp(sink[h]) is one more term of head h's softmax denominator.
 TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int out_stride, const void* plane,
                         const int* block_table, int bt_stride, int num_pages, const int* positions,
                         const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles, int H,
-                        int KVH, int page_size, int window, float scale, int* fault, cudaStream_t stream) {
+                        int KVH, int page_size, int window, float scale, const float* sink, int* fault,
+                        cudaStream_t stream) {
     if (num_tiles <= 0) return TIS_OK;
     if (page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) {
         tis_set_error("attn_tc: page size %d; this kernel takes 16, 32, 64 or 128", page_size);
@@ -411,6 +414,7 @@ TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int 
     p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.num_tiles = num_tiles;
     p.H = H; p.KVH = KVH; p.page_size = page_size; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f;
+    p.sink = sink;
     p.fault = fault;
     tis_launch(attn_tc_kernel, dim3(num_tiles * H), dim3(NTH), (size_t)smem, stream, mq, mkv, p);
     return tis_check_launch("attn_tc");
@@ -421,7 +425,7 @@ TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int 
 TIS_API int tis_attn_tc_supported() { return 0; }
 
 TIS_API int tis_attn_tc(const void*, int, int, void*, int, const void*, const int*, int, int, const int*, const int*,
-                        const int*, const int*, int, int, int, int, int, float, int*, cudaStream_t) {
+                        const int*, const int*, int, int, int, int, int, float, const float*, int*, cudaStream_t) {
     tis_set_error("attn_tc: built for a head size it does not take (64 and 128 only)");
     return TIS_BAD_SIZE;
 }

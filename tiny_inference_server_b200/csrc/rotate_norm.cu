@@ -6,13 +6,14 @@
 //   queries stay where they are, keys and values go into the row's page.
 // `G` 0: a row holds queries only and nothing is written into the cache (a layer that reads another layer's keys).
 // Pages: element (page, kv head, position in the page, i) at pages + page * page_stride + head * head_stride +
-// position * width + i.  Everything is computed in 32-bit; T is the storage type.
+// position * width + i; with `permuted` the 16-byte chunks of a row are permuted by the position (cache_chunk in common.cuh:
+// the row format of the attention kernels whose keys and values have one width).  Everything is computed in 32-bit; T is the storage type.
 #include "common.cuh"
 
 namespace {
 
 struct RotateNorm {
-    int ld, H, G, dim, v_dim, rot, interleaved, norm;
+    int ld, H, G, dim, v_dim, rot, interleaved, norm, permuted;
     float eps;
     const float* cos_t;
     const float* sin_t;
@@ -73,8 +74,9 @@ rotate_norm_vec_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restri
             const int g = hh - p.H - p.G;
             const T* src = row + (size_t)(p.H + p.G) * p.dim + (size_t)g * p.v_dim;
             T* dst = v_pages + (size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim;
+            const int nch = p.v_dim / N;
             for (int i = lane * N; i < p.v_dim; i += LPH * N)
-                *reinterpret_cast<uint4*>(dst + i) = *reinterpret_cast<const uint4*>(src + i);
+                *reinterpret_cast<uint4*>(dst + (p.permuted ? cache_chunk(i / N, pos, nch) * N : i)) = *reinterpret_cast<const uint4*>(src + i);
         }
     }
     const bool works = live && !is_v && (is_q || page >= 0);
@@ -107,7 +109,7 @@ rotate_norm_vec_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restri
         if (e < p.dim) {
 #pragma unroll
             for (int j = 0; j < N; ++j) v[k][j] *= f;
-            Vec16<T>::store(dst + e, v[k]);
+            Vec16<T>::store(dst + (p.permuted && !is_q ? cache_chunk(e / N, pos, p.dim / N) * N : e), v[k]);
         }
     }
 }
@@ -130,9 +132,14 @@ rotate_norm_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__
     const int in_page = pos % p.page_size;
     pdl_wait();
     T* row = qkv + (size_t)r * p.ld;
+    constexpr int N = Vec16<T>::N;
+    auto place = [&](int i, int width, bool permuted) {
+        return permuted ? cache_chunk(i / N, pos, width / N) * N + i % N : i;
+    };
     const int heads = p.H + (page >= 0 ? p.G : 0);
     for (int hh = warp; hh < heads; hh += nw) {
         T* src = row + (size_t)hh * p.dim;
+        const bool perm = p.permuted && hh >= p.H;
         T* dst = hh < p.H ? src : k_pages + (size_t)page * p.k_page_stride + (size_t)(hh - p.H) * p.k_head_stride + (size_t)in_page * p.dim;
         float ss = 0.f;
         for (int i = lane; i < half; i += 32) {
@@ -147,16 +154,16 @@ rotate_norm_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__
         for (int i = lane; i < half; i += 32) {
             const int ia = p.interleaved ? 2 * i : i, ib = p.interleaved ? 2 * i + 1 : i + half;
             const float a = to_f32(src[ia]), b = to_f32(src[ib]);
-            dst[ia] = from_f32<T>((a * ct[i] - b * st[i]) * f);
-            dst[ib] = from_f32<T>((b * ct[i] + a * st[i]) * f);
+            dst[place(ia, p.dim, perm)] = from_f32<T>((a * ct[i] - b * st[i]) * f);
+            dst[place(ib, p.dim, perm)] = from_f32<T>((b * ct[i] + a * st[i]) * f);
         }
-        for (int i = p.rot + lane; i < p.dim; i += 32) dst[i] = from_f32<T>(to_f32(src[i]) * f);
+        for (int i = p.rot + lane; i < p.dim; i += 32) dst[place(i, p.dim, perm)] = from_f32<T>(to_f32(src[i]) * f);
     }
     if (page < 0) return;
     const T* vals = row + (size_t)(p.H + p.G) * p.dim;
     for (int idx = threadIdx.x; idx < p.G * p.v_dim; idx += blockDim.x) {
         const int g = idx / p.v_dim, e = idx - g * p.v_dim;
-        v_pages[(size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim + e] = vals[idx];
+        v_pages[(size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim + place(e, p.v_dim, p.permuted)] = vals[idx];
     }
 }
 
@@ -183,7 +190,7 @@ void launch_any(T* qkv, T* k_pages, T* v_pages, const RotateNorm& p, bool vec, c
 }  // namespace
 
 TIS_API int tis_rotate_norm_store(int dtype, void* qkv, int ld, int H, int G, int dim, int v_dim, int rot, int interleaved,
-                                  const float* cos_t, const float* sin_t, int norm, float eps, void* k_pages,
+                                  int permuted, const float* cos_t, const float* sin_t, int norm, float eps, void* k_pages,
                                   size_t k_page_stride, size_t k_head_stride, void* v_pages, size_t v_page_stride,
                                   size_t v_head_stride, int page_size, int num_pages, const int* block_table, int bt_stride,
                                   const int* positions, const int* row_slot, int* fault, int n, cudaStream_t stream) {
@@ -195,12 +202,16 @@ TIS_API int tis_rotate_norm_store(int dtype, void* qkv, int ld, int H, int G, in
         return TIS_BAD_SIZE;
     }
     RotateNorm p;
-    p.ld = ld; p.H = H; p.G = G; p.dim = dim; p.v_dim = v_dim; p.rot = rot; p.interleaved = interleaved; p.norm = norm; p.eps = eps;
+    p.ld = ld; p.H = H; p.G = G; p.dim = dim; p.v_dim = v_dim; p.rot = rot; p.interleaved = interleaved; p.permuted = permuted; p.norm = norm; p.eps = eps;
     p.cos_t = cos_t; p.sin_t = sin_t;
     p.k_page_stride = k_page_stride; p.k_head_stride = k_head_stride; p.v_page_stride = v_page_stride; p.v_head_stride = v_head_stride;
     p.page_size = page_size; p.num_pages = num_pages; p.block_table = block_table; p.bt_stride = bt_stride;
     p.positions = positions; p.row_slot = row_slot; p.fault = fault; p.n = n;
     const size_t N = dtype == TIS_BF16 ? 8 : 4;
+    if (permuted && G > 0 && (dim % N || v_dim % N)) {
+        tis_set_error("rotate_norm_store: rows of %d and %d elements are not whole 16-byte chunks", dim, v_dim);
+        return TIS_BAD_SIZE;
+    }
     const bool vec = (interleaved || rot == 0) && dim % N == 0 && ld % N == 0 && (uintptr_t)qkv % 16 == 0 &&
                      (G == 0 || (v_dim % N == 0 && ((k_page_stride | k_head_stride | v_page_stride | v_head_stride) % N) == 0 &&
                                  ((uintptr_t)k_pages | (uintptr_t)v_pages) % 16 == 0));

@@ -713,18 +713,29 @@ def plan_splits(num_tiles: int, kv_heads: int, max_kv: int, mode_keys: bool, res
 ATTN_ROTARY = os.environ.get("TIS_ATTN_ROTARY", "1") != "0"
 
 
-def rotary_fusable(q: torch.Tensor, step, num_heads: int, kv_heads: int, head_dim: int) -> bool:
+class PairRotary:
+    """A rotation of the first elements of every head, twice as many as ``cos`` and ``sin`` (positions, rot / 2; None: none)
+    have columns, element 2i with 2i + 1, and (``norm_eps`` not None) the division of the head by its root mean square
+    behind it: what ``paged_attention`` can do to a decode row's queries and key itself (``rotary=``)."""
+
+    def __init__(self, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], norm_eps: Optional[float] = None):
+        self.cos, self.sin, self.norm_eps = cos, sin, norm_eps
+
+
+def rotary_fusable(q: torch.Tensor, step, num_heads: int, kv_heads: int, head_dim: int, pairs: bool = False) -> bool:
     """Whether ``paged_attention`` can take rows whose queries are not rotated yet and whose keys and
     values are not in the cache yet (``rotary=``): a decode step (one row per request) in bfloat16, a head
-    size the kernel rotates in registers, at most 16 query heads per kv head."""
+    size the kernel rotates in registers, at most 16 query heads per kv head.  ``pairs``: the rotation is a
+    ``PairRotary``, whose pairs lie in one register at any head size."""
     return (ATTN_ROTARY and q.dtype == torch.bfloat16 and step is not None and getattr(step, "decode_only", False)
-            and head_dim % 32 == 0 and kv_heads > 0 and num_heads % kv_heads == 0 and num_heads // kv_heads <= 16)
+            and (head_dim % 32 == 0 or pairs) and kv_heads > 0 and num_heads % kv_heads == 0 and num_heads // kv_heads <= 16)
 
 
 def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, block_table: torch.Tensor,
                     positions: torch.Tensor, row_slot: torch.Tensor, num_heads: int, kv_heads: int,
                     head_dim: int, page_size: int, window: Optional[int], fault: torch.Tensor,
-                    step=None, rotary=None, write_kv: bool = True) -> torch.Tensor:
+                    step=None, rotary=None, write_kv: bool = True, scale: Optional[float] = None,
+                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the step's rows over the cache.  ``q`` is (n, >= H*hd) with the
     queries first in each row (row stride free); ``out`` is (n, H*hd).  The row at position
     p of slot s sees keys max(0, p-window+1)..p of ``plane`` through ``block_table[s]``.
@@ -735,17 +746,24 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
     ``rotary=(cos, sin)`` (only where ``rotary_fusable``): the rows of ``q`` are the projection's output
     as it is, [queries | keys | values]; the kernel rotates queries and keys itself (half-split pairs,
     tables [positions, hd/2] float32) and, with ``write_kv``, writes the rows' keys and values into
-    their pages — what ``rope_kv_write`` does in a launch of its own everywhere else."""
+    their pages — what ``rope_kv_write`` does in a launch of its own everywhere else.  Or ``rotary`` a ``PairRotary``:
+    neighbouring elements paired, and the norm of every head (``rotate_norm_store`` everywhere else).
+
+    ``scale`` (positive; 1 / sqrt(head_dim) unless given) multiplies the scores.  ``sink`` (H,) float32: head h's softmax
+    denominator also holds ``exp(sink[h])`` (unscaled; it has no key and no value)."""
     lib = library()
     n = q.shape[0]
-    scale = 1.0 / math.sqrt(head_dim)
-    if rotary is not None and not rotary_fusable(q, step, num_heads, kv_heads, head_dim):
+    scale = 1.0 / math.sqrt(head_dim) if scale is None else float(scale)
+    if not scale > 0:
+        raise KernelError(f"paged_attention: the scores are multiplied by a positive number, not {scale}")
+    pairs = isinstance(rotary, PairRotary)
+    if rotary is not None and not rotary_fusable(q, step, num_heads, kv_heads, head_dim, pairs):
         raise KernelError("paged_attention: rotary encoding inside the kernel is for decode steps in bfloat16")
     if q.dtype == torch.float32:
         _check(lib.tis_paged_attention_simt(
             _dt(q), _p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table), block_table.stride(0),
             plane.shape[0], _p(positions), _p(row_slot), n, num_heads, kv_heads, head_dim, page_size,
-            int(window or 0), _f(scale), _p(fault), _stream()), lib)
+            int(window or 0), _f(scale), _p(sink), _p(fault), _stream()), lib)
         return out
     if kv_heads <= 0 or num_heads % kv_heads:
         raise KernelError(f"paged_attention: {num_heads} query heads are not a multiple of {kv_heads} kv heads")
@@ -764,6 +782,9 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         tiles = attention_plan.infer_tiles(positions, row_slot, g)
         max_kv = int(positions.max().item()) + 1 if n else 1
     rows_tiles = tiles.rows
+    # keys that the key splits share out: with a window those from the tile's first one on (a tile's rows see at most
+    # 63 keys more than one of them does, and the share starts at a multiple of 64)
+    split_kv = max_kv if not window else min(max_kv, int(window) + 128)
     w0, wn, wide_count = getattr(tiles, "wide", (None, None, 0))
     # One CTA of the tcgen05 kernel walks all keys of its 128 rows (no key splits yet).  Measured at the
     # 0.9B sizes: with two or more such tiles in the step it wins (256 rows ending at 4096: 51 against
@@ -775,8 +796,8 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         calls["attn_tc"] += 1
         _check(alib.tis_attn_tc(_p(q), q.stride(0), n, _p(out), out.stride(0), _p(plane), _p(block_table),
                                 block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(w0), _p(wn),
-                                wide_count, num_heads, kv_heads, page_size, int(window or 0), _f(scale), _p(fault),
-                                _stream()), alib)
+                                wide_count, num_heads, kv_heads, page_size, int(window or 0), _f(scale), _p(sink),
+                                _p(fault), _stream()), alib)
         skip = tiles.rows_in_wide
         if skip == tiles.rows[2]:
             rows_tiles = (None, None, 0)
@@ -790,16 +811,21 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         resident = alib.resident.get((1, half))
         if resident is None:
             resident = alib.resident[(1, half)] = alib.tis_attn_resident_ctas(1, half)
-        per, splits = plan_splits(count, kv_heads, max_kv, True, resident, None)
+        per, splits = plan_splits(count, kv_heads, split_kv, True, resident, None)
         calls["attn_keys_rotary"] += 1
-        cos, sin = rotary
+        if pairs:
+            cos, sin = rotary.cos, rotary.sin
+            how = (2, 2 * cos.shape[1] if cos is not None else 0, int(rotary.norm_eps is not None), _f(rotary.norm_eps or 0.0))
+        else:
+            cos, sin = rotary
+            how = (1, head_dim, 0, _f(0.0))
         if getattr(tiles, "keys_identity", False) and count == n:
             row0 = rows = None          # tile i is row i: the kernel reads no tile arrays
         _check(alib.tis_attn_decode_rope(_p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table),
                                          block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(row0),
                                          _p(rows), count, n, num_heads, kv_heads, page_size, int(window or 0),
-                                         _f(scale), per, splits, _p(cos), _p(sin), int(bool(write_kv)), _p(fault),
-                                         _stream()), alib)
+                                         _f(scale), per, splits, _p(cos), _p(sin), int(bool(write_kv)), *how, _p(sink),
+                                         _p(fault), _stream()), alib)
         return out
     for mode, (row0, rows, count) in ((1, tiles.keys), (0, rows_tiles)):
         if count == 0:
@@ -809,19 +835,20 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         resident = alib.resident.get((mode, half))
         if resident is None:
             resident = alib.resident[(mode, half)] = alib.tis_attn_resident_ctas(mode, half)
-        per, splits = plan_splits(count, kv_heads, max_kv, mode == 1, resident, None if mode == 1 else min_kv)
+        per, splits = plan_splits(count, kv_heads, split_kv, mode == 1, resident,
+                                  None if mode == 1 or min_kv is None else min(min_kv, split_kv))
         calls["attn_keys" if mode == 1 else "attn_rows"] += 1
         # at most eight splits (plan_splits): they merge inside a thread-block cluster, without scratch
-        _check(alib.tis_attn_mma(mode, _p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table),
+        _check(alib.tis_attn_mma_sink(mode, _p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table),
                                  block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(row0),
                                  _p(rows), count, max_rows, n, num_heads, kv_heads, page_size, int(window or 0), _f(scale),
-                                 per, splits, _p(None), _p(fault), _stream()), alib)
+                                 per, splits, _p(None), _p(sink), _p(fault), _stream()), alib)
     return out
 
 
 def swiglu(gu: torch.Tensor, out: torch.Tensor, block: Optional[int] = None, form: GateForm = SILU) -> torch.Tensor:
-    """out[r, j] = gated(gate_j, up_j) in the form ``form`` (silu(gate_j) * up_j unless given) where a row of ``gu`` holds gate and up columns in
-    alternating blocks of ``block`` (default: the hidden size, i.e. [all gates | all ups])."""
+    """out[r, j] = gated(gate_j, up_j) in the form ``form`` (silu(gate_j) * up_j unless given) where a row of ``gu`` holds
+    gate and up columns in alternating blocks of ``block`` (default: the hidden size, i.e. [all gates | all ups])."""
     lib = library()
     n, f = out.shape
     _check(lib.tis_swiglu(_dt(gu), _p(gu), _p(out), n, f, block or f, form, _stream()), lib)
@@ -1308,13 +1335,14 @@ def add_layer_norm(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delt
 def rotate_norm_store(qkv: torch.Tensor, num_heads: int, kv_heads: int, dim: int, v_dim: int, cos: Optional[torch.Tensor],
                       sin: Optional[torch.Tensor], interleaved: bool, norm: bool, eps: float, k_pages: Optional[torch.Tensor],
                       v_pages: Optional[torch.Tensor], block_table: torch.Tensor, positions: torch.Tensor,
-                      row_slot: torch.Tensor, page_size: int, fault: torch.Tensor) -> None:
+                      row_slot: torch.Tensor, page_size: int, fault: torch.Tensor, permuted: bool = False) -> None:
     """Between the projections and the cache of an attention whose queries and keys are rotated and then normed head by
     head.  A row of ``qkv``: H query heads and G key heads of ``dim`` elements, G value heads of ``v_dim``.  The first
     elements of every query and key head, twice as many as ``cos`` and ``sin`` (positions, rot / 2; None: none) have columns,
     are rotated by the row's position (``interleaved``: element 2i with 2i + 1, else i with i + rot / 2); with ``norm`` the
     head is then divided by its root mean square (eps inside the root).  Queries in place; keys and values into the row's
-    page.  ``kv_heads`` 0: the rows hold queries only and nothing is stored.  Everything is computed in 32-bit."""
+    page, in the row format of ``paged_attention`` if ``permuted`` (16-byte chunks permuted by the position), else as they
+    are.  ``kv_heads`` 0: the rows hold queries only and nothing is stored.  Everything is computed in 32-bit."""
     lib = library()
     n = qkv.shape[0]
     rot = 0 if cos is None else 2 * cos.shape[1]
@@ -1329,7 +1357,7 @@ def rotate_norm_store(qkv: torch.Tensor, num_heads: int, kv_heads: int, dim: int
     if qkv.stride(1) != 1:
         raise KernelError("rotate_norm_store: the rows are not dense")
     _check(lib.tis_rotate_norm_store(_dt(qkv), _p(qkv), qkv.stride(0), num_heads, kv_heads, dim, v_dim, rot, int(interleaved),
-                                     _p(cos), _p(sin), int(norm), _f(eps), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
+                                     int(permuted), _p(cos), _p(sin), int(norm), _f(eps), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
                                      page_size, k_pages.shape[0] if k_pages is not None else 0, _p(block_table),
                                      block_table.stride(0), _p(positions), _p(row_slot), _p(fault), n, _stream()), lib)
 

@@ -6,7 +6,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..kernels import ops, window_plan
+from ..kernels import attention_plan, ops, window_plan
 from ..registry import register_part
 from .base import BuildContext, KVSpec, LayerBinding, Mixer, WeightSpec
 from .window_attention import pad8
@@ -27,6 +27,12 @@ class NormedRotaryAttention(Mixer):
     * ``score = (q . k) * scale`` over the keys ``p - window + 1 .. p`` (``window`` None: ``0 .. p``), softmax in 32-bit; with
       ``has_sink`` its denominator also holds ``exp(sink[h])``, a term without a key or a value behind it;
     * ``Wo`` on the heads' outputs side by side.
+
+    How it runs: keys and values of one width that is a multiple of 16 (16..256), at most 64 query heads a kv head: the paged
+    attention kernels of the rotary GQA model (tcgen05 tiles for long portions, key splits over a cluster for decode rows,
+    which also rotate, norm and store the row's own key); any other widths: the kernels of windowed attention, behind a
+    launch that rotates, norms and stores.  The choice depends on the layer's sizes only, so all layers that use a plane
+    agree on its row format.
 
     The cache holds the keys as the scores take them (rotated, normed) and the values.  ``reads_cache``: the layer has no key
     and value projections and stores nothing; its schedule entry names the entry whose plane it reads
@@ -50,6 +56,7 @@ class NormedRotaryAttention(Mixer):
         self.cache_window = window if cache_window == OWN_WINDOW else cache_window
         if self.cache_window is not None and (window is None or window > self.cache_window):
             raise ValueError(f"a window of {window} keys over a plane that keeps {self.cache_window}")
+        self.paged = (dim == v_dim and dim % 16 == 0 and 16 <= dim <= 256 and num_heads // kv_heads <= 64 and self.scale > 0)
         self.nq, self.nk, self.nv, self.no = num_heads * dim, kv_heads * dim, kv_heads * v_dim, num_heads * v_dim
         self.w_in = self.w_o = self.sink = None
 
@@ -68,7 +75,8 @@ class NormedRotaryAttention(Mixer):
         return KVSpec(self.kv_heads, self.dim, self.cache_window, 0, k_dim=self.dim, v_dim=self.v_dim)
 
     def step_planners(self):
-        return (window_plan.planner(self.num_heads // self.kv_heads),)
+        plan = attention_plan if self.paged else window_plan
+        return (plan.planner(self.num_heads // self.kv_heads),)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         specs = {"q": WeightSpec((self.nq, self.width))}
@@ -97,14 +105,22 @@ class NormedRotaryAttention(Mixer):
         table, page_size = step.block_tables[g], step.page_sizes[g]
         proj = ops.gemm(x, self.w_in)
         pos = self.position
-        ops.rotate_norm_store(proj, self.num_heads, 0 if self.reads_cache else self.kv_heads, self.dim, self.v_dim,
-                              pos.cos if pos is not None else None, pos.sin if pos is not None else None,
-                              pos.interleaved if pos is not None else True, self.qk_norm, self.eps, binding.k_pages,
-                              binding.v_pages, table, step.positions, step.row_slot, page_size, step.fault)
+        cos, sin, interleaved = (pos.cos, pos.sin, pos.interleaved) if pos is not None else (None, None, True)
         out = torch.empty((n, self.no), dtype=x.dtype, device=x.device)
-        ops.window_attention(proj[:, :self.nq], None, out, binding.k_pages, binding.v_pages, table, step.positions,
-                             step.row_slot, self.num_heads, page_size, self.window, self.scale, None, None, step.fault, step,
-                             sink=self.sink)
+        in_kernel = self.paged and interleaved and ops.rotary_fusable(proj, step, self.num_heads, self.kv_heads, self.dim, pairs=True)
+        if not in_kernel:
+            ops.rotate_norm_store(proj, self.num_heads, 0 if self.reads_cache else self.kv_heads, self.dim, self.v_dim, cos, sin,
+                                  interleaved, self.qk_norm, self.eps, binding.k_pages, binding.v_pages, table, step.positions,
+                                  step.row_slot, page_size, step.fault, permuted=self.paged)
+        if self.paged:
+            rotary = ops.PairRotary(cos, sin, self.eps if self.qk_norm else None) if in_kernel else None
+            ops.paged_attention(proj, out, binding.kv_plane, table, step.positions, step.row_slot, self.num_heads, self.kv_heads,
+                                self.dim, page_size, self.window, step.fault, step, rotary=rotary,
+                                write_kv=not self.reads_cache, scale=self.scale, sink=self.sink)
+        else:
+            ops.window_attention(proj[:, :self.nq], None, out, binding.k_pages, binding.v_pages, table, step.positions,
+                                 step.row_slot, self.num_heads, page_size, self.window, self.scale, None, None, step.fault,
+                                 step, sink=self.sink)
         return ops.gemm(out, self.w_o, sink=residual)
 
 
