@@ -518,6 +518,78 @@ def compare_kubolorn(args):
     return 0
 
 
+def lomutar_config(width, heads, kv_heads, ffn, vocab, layers, window=1024, experts=16, top=3):
+    """A Lomutar model with the layer sizes of a member of the GQA family: attention in a window with heads of 128, half of
+    each rotated, every fourth layer reading the keys and values of the layer before it; feed-forwards in turn dense (gelu
+    gating, ffn hidden elements) and routed (``top`` of ``experts`` clamped units of ffn / (top + 1) hidden elements and a
+    shared one of the same size, so that a token meets as many weights as in the dense one)."""
+    fe = max(64, ffn // (top + 1) // 64 * 64)
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+            "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 4.0}}}
+    moe = {"kind": "moe", "expert": {"ff": fe, "limit": 7.0}, "shared": {"ff": fe, "limit": 7.0},
+           "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    made = []
+    for i in range(layers):
+        mixer = json.loads(json.dumps(attn))
+        if i % 4 == 3:
+            mixer["kv_from"] = i - 1
+        made.append({"type": "attention", "mixer": mixer,
+                     "mlp": {"kind": "dense", "ff": ffn} if i % 2 == 0 else json.loads(json.dumps(moe))})
+    return dict(architecture="Lomutar", vocab=vocab, width=width, norm={"eps": 1e-5}, max_context=8192, layers=made)
+
+
+def compare_lomutar(args):
+    """``--compare lomutar``: prefill and decode of the Lomutar architecture beside the rotary GQA model with the same window
+    (the closest for its attention and dense layers) and the Mizidra architecture (the closest for its routed layers) at
+    equal layer sizes, and its kernels beside the like kernels of those.  One JSON line; the default run is untouched."""
+    import gc
+    import types
+    import torch
+    from tiny_inference_server_b200.kernels import microbench, ops
+    from tiny_inference_server_b200.sampling import Sampler
+    pk = peaks()
+    count_ops = lambda: ops.launches  # noqa: E731
+    window, ctx, layers = 1024, 4096, 8
+    result = {"compare": "lomutar", "dtype": "bf16", "data": "synthetic", "layers": layers, "context": ctx, "window": window,
+              "peaks": pk, "sizes": {}}
+    for name in [x for x in args.compare_sizes.split(",") if x]:
+        base = SIZES[name][0]
+        twin = dict(base, num_layers=layers, num_mtp_heads=0, sliding_window=window, max_context=8192, tie_word_embeddings=False)
+        size = (base["hidden_size"], base["num_heads"], base["num_kv_heads"], base["ffn_hidden"], base["vocab_size"], layers)
+        point = {}
+        for label, cfg_dict in (("lomutar", lomutar_config(*size, window=window)), ("gqa", twin), ("mizidra", mizidra_config(*size))):
+            runner = None
+            try:
+                _, runner = build_runner(cfg_dict, ctx, 8, mtp=False)
+                steps = max(8, args.steps // 2)
+                r = {}
+                for b in (1, 8):
+                    ms, launches = decode_run(runner, b, ctx - steps - args.warmup - 2, steps, args.warmup, Sampler, count_ops)
+                    r[f"decode_b{b}_tok_s"] = round(b / (ms * 1e-3), 1)
+                    r[f"decode_b{b}_ms"] = round(ms, 4)
+                    r[f"decode_b{b}_launches"] = round(launches, 1)
+                best, first = prefill_run(runner, PREFILL_TOKENS, reps=2)
+                r["prefill_tok_s"] = round(PREFILL_TOKENS / (best * 1e-3), 1)
+                r["prefill_ms"] = round(best, 3)
+                r["prefill_first_run_ms"] = round(first, 3)
+                point[label] = r
+            except Exception as e:                       # noqa: BLE001
+                point[label] = {"error": f"{type(e).__name__}: {e}"[:300]}
+            del runner
+            gc.collect()
+            torch.cuda.empty_cache()
+        margs = types.SimpleNamespace(width=base["hidden_size"], ffn=base["ffn_hidden"], heads=base["num_heads"],
+                                      kv_heads=base["num_kv_heads"], head_dim=128, page_size=PAGE, tokens=PREFILL_TOKENS, batch=8,
+                                      context=ctx, window=window, experts=16, top=3)
+        try:
+            point["kernels"] = microbench.normed_shared_clamped(margs)
+        except Exception as e:                           # noqa: BLE001
+            point["kernels"] = {"error": f"{type(e).__name__}: {e}"[:300]}
+        result["sizes"][name] = point
+    print(json.dumps(result))
+    return 0
+
+
 def compare_kefisun(args):
     """``--compare kefisun``: prefill and decode of the Kefisun architecture beside the rotary GQA model at equal
     layer sizes (same width, heads, feed-forward, vocabulary, number of layers, and the same window of keys), and
@@ -663,7 +735,7 @@ def main(argv=None):
     ap.add_argument("--impl", default="engine", choices=["engine", "reference"])
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64, other contexts, MTP heads and prefill")
     ap.add_argument("--sizes", default="3b,8b", help="larger members of the family to measure too (3b, 8b; '' = none)")
-    ap.add_argument("--compare", default=None, choices=["kefisun", "mizidra", "biruvik", "kubolorn"],
+    ap.add_argument("--compare", default=None, choices=["kefisun", "mizidra", "biruvik", "kubolorn", "lomutar"],
                     help="instead of the default run: another architecture beside the GQA model at equal layer sizes")
     ap.add_argument("--compare-sizes", default="0.9b,3b", help="with --compare: whose layer sizes (0.9b, 3b, 8b)")
     args = ap.parse_args(argv)
@@ -675,6 +747,9 @@ def main(argv=None):
     if args.compare == "mizidra":
         args.warmup = max(args.warmup, 3)
         return compare_mizidra(args)
+    if args.compare == "lomutar":
+        args.warmup = max(args.warmup, 3)
+        return compare_lomutar(args)
     if args.compare == "kubolorn":
         return compare_kubolorn(args)
     if args.compare == "biruvik":

@@ -14,6 +14,8 @@
     python -m tiny_inference_server_b200.kernels.microbench differential-latent-forget   (two score maps a head,
         windowed attention over compressed rows with head gates, the recurrence whose forget gate writes, a norm behind a
         sublayer, each beside the like kernel of an earlier model)
+    python -m tiny_inference_server_b200.kernels.microbench normed-shared-clamped   (attention with normed heads and a
+        sink, layer norm with two updates, gelu gating, clamped experts, each beside the like kernel of an earlier model)
     python -m tiny_inference_server_b200.kernels.microbench all
 
 ``--reps N --no-timing`` launches the kernel N times and exits (a profiler attaches to that);
@@ -749,6 +751,109 @@ def gated_space_tied(args):
     return out
 
 
+def normed_shared_clamped(args):
+    """The kernels of attention with rotated and normed heads, a window and a keyless softmax term, of the layer norm with two
+    updates, of gated products in their gelu form and of the mixture of clamped units with a softmax router, each beside the
+    kernel of an earlier architecture of this engine that does the like work at equal sizes: the rotary GQA model's attention
+    (same window), rotation, fused norm and gated product, Mizidra's routed experts.  Returns {name: {us, rate, unit, like_us,
+    like_rate}}."""
+    from .attention_plan import infer_tiles
+    dev = "cuda"
+    d, F, H, G, hd, page = args.width, args.ffn, args.heads, args.kv_heads, args.head_dim, args.page_size
+    n, B, ctx, W, E, top = args.tokens, args.batch, args.context, args.window, args.experts, args.top
+    bf, i32 = dict(device=dev, dtype=torch.bfloat16), dict(device=dev, dtype=torch.int32)
+    fault, out, bufs = torch.zeros(4, **i32), {}, 6
+
+    def put(name, us, work, unit, like_us, like_work=None):
+        div, digits = (1e3, 1) if unit == "GB/s" else (1e6, 1)
+        like_work = work if like_work is None else like_work
+        out[name] = {"us": round(us, 2), "rate": round(work / us / div, digits), "unit": unit, "like_us": round(like_us, 2),
+                     "like_rate": round(like_work / like_us / div, digits)}
+        e = out[name]
+        print(f"{name:52s} {e['us']:9.2f} us {e['rate']:9.1f} {unit}   like kernel {e['like_us']:9.2f} us {e['like_rate']:9.1f} {unit}")
+
+    # ---- attention of a prompt portion (n rows from position 0) and of B decode rows, window W, beside the same without a sink
+    num_pages = (n + page - 1) // page
+    nq, nk = H * hd, G * hd
+    planes = [torch.randn(num_pages, 2, G, page, hd, **bf) for _ in range(2)]
+    table = torch.arange(num_pages, **i32).reshape(1, num_pages).contiguous()
+    pos, slot = torch.arange(n, **i32), torch.zeros(n, **i32)
+    qkv = [torch.randn(n, nq + 2 * nk, **bf) for _ in range(bufs)]
+    o, sink = torch.empty(n, nq, **bf), torch.zeros(H, device=dev)
+    step = _Step(infer_tiles(pos, slot, H // G), n - 1)
+    step.decode_only, step.min_position = False, 0
+    flops = 4.0 * nq * sum(min(p + 1, W) for p in range(n))
+    t_new = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs], o, planes[i % 2], table, pos, slot, H, G, hd, page, W, fault, step,
+                                                      sink=sink), 10)
+    t_like = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs], o, planes[i % 2], table, pos, slot, H, G, hd, page, W, fault,
+                                                       step), 10)
+    put(f"attention with a sink, {n} rows, window {W}", t_new, flops, "TFLOP/s", t_like)
+    half = hd // 4                                             # half of every head rotated
+    cos, sin = torch.ones(ctx + n, hd // 2, device=dev), torch.zeros(ctx + n, hd // 2, device=dev)
+    cos_p, sin_p = cos[:, :half].contiguous(), sin[:, :half].contiguous()
+    plane = torch.zeros(num_pages, 2, G, page, hd, **bf)
+    t_new = _graph_time(lambda i: ops.rotate_norm_store(qkv[i % bufs], H, G, hd, hd, cos_p, sin_p, True, True, 1e-5, plane[:, 0],
+                                                        plane[:, 1], table, pos, slot, page, fault, permuted=True), 12)
+    t_like = _graph_time(lambda i: ops.rope_kv_write(qkv[i % bufs], pos, slot, cos, sin, plane, table, H, G, hd, page, fault), 12)
+    put(f"rotation, head norms, cache write, {n} rows", t_new, n * (nq + 2 * nk) * 4, "GB/s", t_like)
+    pages_per = (ctx + page - 1) // page
+    n_planes = max(2, min(12, (300 << 20) // max(1, B * ctx * 2 * nk * 2)))
+    planes = [torch.randn(B * pages_per, 2, G, page, hd, **bf) for _ in range(n_planes)]
+    dtable = torch.arange(B * pages_per, **i32).reshape(B, pages_per).contiguous()
+    pos_b, slot_b = torch.full((B,), ctx - 1, **i32), torch.arange(B, **i32)
+    dstep = _Step(infer_tiles(pos_b, slot_b, H // G), ctx - 1)
+    for win in (W, None):
+        kv_bytes = B * min(win or ctx, ctx) * 2 * nk * 2
+        rot = ops.PairRotary(cos_p, sin_p, 1e-5)
+        t_new = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs][:B], o[:B], planes[i % n_planes], dtable, pos_b, slot_b, H, G, hd,
+                                                          page, win, fault, dstep, rotary=rot, sink=sink))
+        t_like = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs][:B], o[:B], planes[i % n_planes], dtable, pos_b, slot_b, H, G, hd,
+                                                           page, win, fault, dstep, rotary=(cos, sin)))
+        put(f"rotate, norm, store, attend, {B} decode rows, " + (f"window {win}" if win else f"all of {ctx}"), t_new, kv_bytes,
+            "GB/s", t_like)
+    del planes
+    # ---- the layer norm with two updates beside the fused RMS norm with one
+    res = [torch.randn(n, d, device=dev) for _ in range(bufs)]
+    da, db = [torch.randn(n, d, **bf) for _ in range(bufs)], [torch.randn(n, d, **bf) for _ in range(bufs)]
+    y, w, b = torch.empty(n, d, **bf), torch.ones(d, device=dev), torch.zeros(d, device=dev)
+    for rows in (n, B):
+        t_new = _graph_time(lambda i: ops.add_layer_norm(res[i % bufs][:rows], da[i % bufs][:rows], db[i % bufs][:rows], w, b, 1e-5,
+                                                         y[:rows]), 12)
+        t_like = _graph_time(lambda i: ops.add_rmsnorm(res[i % bufs][:rows], da[i % bufs][:rows], w, 1e-5, y[:rows], kind="mean_eps"), 12)
+        put(f"two updates, layer norm, {rows} rows", t_new, rows * d * 14, "GB/s", t_like, rows * d * 12)
+    # ---- gate and up with the gelu gating beside the same with silu
+    x = torch.randn(n, d, **bf)
+    wgu = [torch.randn(d, 2 * F, **bf) * 0.02 for _ in range(4)]
+    gelu = ops.gate_gelu_tanh()
+    for rows in (B, n):
+        work, unit = (2 * d * F * 2, "GB/s") if rows == B else (4.0 * rows * d * F, "TFLOP/s")
+        t_new = _graph_time(lambda i: ops.gemm_swiglu(x[:rows], wgu[i % 4], F, 32, gelu), 8)
+        t_like = _graph_time(lambda i: ops.gemm_swiglu(x[:rows], wgu[i % 4], F, 32), 8)
+        put(f"gate, up, gelu gating, {rows} rows", t_new, work, unit, t_like)
+    del wgu
+    # ---- router and experts beside Mizidra's
+    fe = max(64, F // (top + 1) // 64 * 64)
+    wr, corr = torch.randn(E, d, device=dev) * d ** -0.5, torch.zeros(E, device=dev)
+    for rows in (n, B):
+        t_new = _graph_time(lambda i: ops.moe_route(x[:rows], wr, None, None, 4, 2, top, scores="softmax", group_score="best",
+                                                    renorm=False), 12)
+        t_like = _graph_time(lambda i: ops.moe_route(x[:rows], wr, corr, None, 4, 2, top), 12)
+        put(f"router, softmax, best of groups, {rows} rows", t_new, rows * d * 2 + E * d * 4, "GB/s", t_like)
+    gu = [torch.randn(E, 2, fe, d, **bf) * 0.02 for _ in range(2)]
+    dn = [torch.randn(E, d, fe, **bf) * 0.02 for _ in range(2)]
+    chosen, weights, _ = ops.moe_route(x, wr, None, None, 4, 2, top, scores="softmax", group_score="best", renorm=False)
+    shared, form = torch.randn(n, d, **bf), ops.gate_clamped(7.0)
+    used = len(set(chosen[:B].flatten().tolist()))
+    for rows in (n, B):
+        work, unit = (6.0 * rows * top * d * fe, "TFLOP/s") if rows == n else (used * 3 * d * fe * 2, "GB/s")
+        ones = torch.ones(rows, device=dev)
+        t_new = _graph_time(lambda i: ops.moe_experts(x[:rows], chosen[:rows], weights[:rows], gu[i % 2], dn[i % 2], shared[:rows], None,
+                                                      form=form), 8)
+        t_like = _graph_time(lambda i: ops.moe_experts(x[:rows], chosen[:rows], weights[:rows], gu[i % 2], dn[i % 2], shared[:rows], ones), 8)
+        put(f"clamped experts and their sum, {rows} rows", t_new, work, unit, t_like)
+    return out
+
+
 def sampling(args):
     """The sampling kernel at ``--rows`` rows of ``--vocab`` logits, for the kinds of setting a row can have."""
     dev = "cuda"
@@ -952,7 +1057,7 @@ def timeline(args):
 def main(argv=None):
     ap = argparse.ArgumentParser(prog="microbench", description=__doc__.split("\n\n")[0])
     ap.add_argument("what", choices=["attention", "attention-prefill", "rowwise", "gemm", "prefill", "sampling", "timeline",
-                                     "seqmix", "latent-linear-routed", "differential-latent-forget", "gated-space-tied", "all"])
+                                     "seqmix", "latent-linear-routed", "differential-latent-forget", "gated-space-tied", "normed-shared-clamped", "all"])
     ap.add_argument("--rank", type=int, default=128, help="latent-linear-routed: compressed elements a token")
     ap.add_argument("--rot", type=int, default=64, help="latent-linear-routed: rotated elements a token")
     ap.add_argument("--experts", type=int, default=16)
@@ -1005,6 +1110,8 @@ def main(argv=None):
         differential_latent_forget(args)
     if args.what in ("gated-space-tied", "all"):
         gated_space_tied(args)
+    if args.what in ("normed-shared-clamped", "all"):
+        normed_shared_clamped(args)
     return 0
 
 
