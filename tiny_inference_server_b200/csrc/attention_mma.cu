@@ -76,10 +76,10 @@ struct AttnParams {
     int recv_offset;        // bytes from the start of shared memory to where the cluster's partial results land
     // rotary encoding and cache write done by this kernel (decode rows; see FUSED below)
     const float* rope_cos; const float* rope_sin;   // [positions][HD/2]
+    bf16* plane_w;          // the plane, writable: where the row's key and value go (null: another entry fills it)
     int rope_rot;           // FUSED_PAIRS: how many elements of a head are rotated (tables [positions][rope_rot / 2]),
     int rope_norm; float rope_eps;      // and whether the head is then divided by its root mean square
     const float* sink;      // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
-    bf16* plane_w;          // the plane, writable: where the row's key and value go (null: another entry fills it)
     TIS_TIMELINE_MEMBER     // (instrumented builds only; the decode kernel's stamps: 0 entry, 1 before and 2 after the
                             //  dependency wait, 3 first tile landed, 4 last tile landed, 5 loop done, 6 partial results
                             //  pushed, 7 partials of the cluster arrived, 8 stored)
@@ -321,7 +321,8 @@ __device__ __forceinline__ void merge_barrier_init(unsigned long long* merge_bar
     mbar_arrive_expect_tx(merge_bar, ms.own_blocks ? (int)ms.ns * ms.pairs * (ms.own_blocks * 8 + 2) * 4 : 0);
 }
 
-template <int NR>
+// SINK: the row's softmax may hold a keyless term (p.sink).
+template <int NR, bool SINK>
 __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, unsigned char* smem_raw, float* recv,
                                                         unsigned long long* merge_bar, const MergeShape& ms,
                                                         const float (&o)[DTILES][4], const float (&m_run)[2],
@@ -399,7 +400,7 @@ __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, uns
                 acc += from[sp * step_sp + c] * f;
             }
         }
-        if (p.sink != nullptr) add_sink(acc, lsum, mt, p.sink[kvh * G + g]);
+        if (SINK && p.sink != nullptr) add_sink(acc, lsum, mt, p.sink[kvh * G + g]);
         p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
             __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
     }
@@ -793,7 +794,7 @@ attn_mma_kernel(const AttnParams p) {
     }
 
     if (pushed_merge) {
-        merge_splits_by_pushing<NR>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
+        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
     } else if (MODE == MODE_KEYS) {
         // merge the four warps (each saw a quarter of the keys) through shared memory
         __syncthreads();
@@ -829,7 +830,7 @@ attn_mma_kernel(const AttnParams p) {
                     acc += mo[(w * 16 + m) * HD + d] * f;
                 }
             }
-            if (p.num_splits == 1 && p.sink != nullptr) add_sink(acc, lt, mt, p.sink[hq]);
+            if (FUSED != FUSED_HALVES && p.num_splits == 1 && p.sink != nullptr) add_sink(acc, lt, mt, p.sink[hq]);
             const float val = lt > 0.f ? acc / lt : 0.f;
             if (p.num_splits == 1) {
                 p.out[(size_t)row * p.out_stride + (size_t)hq * HD + d] = __float2bfloat16_rn(val);
@@ -1285,7 +1286,7 @@ attn_decode_kernel(const AttnParams p) {
             l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 1);
             l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 2);
         }
-        merge_splits_by_pushing<NR>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
+        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
     }
 }
 
@@ -1604,7 +1605,7 @@ TIS_API int tis_attn_mma_sink(int mode, const void* q, int q_stride, void* out, 
 // when write_kv is 0: another entry of the schedule fills the plane); cos/sin [positions][HD/2] float32,
 // half-split pairs, the whole head rotated (kind 1); or kind 2: neighbouring elements paired, the first `rot` of a head rotated
 // (tables [positions][rot/2], may be null for rot 0) and, with `norm`, the head then divided by its root mean square (`eps`
-// inside the root).  `sink`: as in tis_attn_mma_sink.  At most 16 key splits (they merge inside a cluster).
+// inside the root).  `sink` (kind 2): as in tis_attn_mma_sink.  At most 16 key splits (they merge inside a cluster).
 TIS_API int tis_attn_decode_rope(const void* qkv, int q_stride, void* out, int out_stride, void* plane,
                                  const int* block_table, int bt_stride, int num_pages, const int* positions,
                                  const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
@@ -1612,8 +1613,8 @@ TIS_API int tis_attn_decode_rope(const void* qkv, int q_stride, void* out, int o
                                  int keys_per_split, int num_splits, const float* rope_cos, const float* rope_sin,
                                  int write_kv, int kind, int rot, int norm, float eps, const float* sink, int* fault,
                                  cudaStream_t stream) {
-    if (kind != FUSED_HALVES && kind != FUSED_PAIRS) {
-        tis_set_error("attn_decode_rope: rotation kind %d", kind);
+    if ((kind != FUSED_HALVES && kind != FUSED_PAIRS) || (kind == FUSED_HALVES && sink != nullptr)) {
+        tis_set_error("attn_decode_rope: rotation kind %d%s", kind, sink != nullptr ? " with a sink" : "");
         return TIS_BAD_SIZE;
     }
     if (num_splits > MAX_CLUSTER) {

@@ -33,11 +33,14 @@ struct Epilogue {
     bf16* out; int ldo;
     int M, N;
     int epi;
-    GateForm gate;           // EPI_SWIGLU: the form of the gating
     // rows that still lack their norm's factor: partial sums of squares [M][in_parts] (null: none)
     const float* in_ss; int in_parts; NormFactor in_factor;
     // EPI_RESIDUAL: the stream [M][ldr] (read and written), the next norm's weight [N], partial sums out [M][strips]
-    float* res; int ldr; const float* norm_w; float* out_ss;
+    float* res; int ldr;
+    union {                  // (one kernel has one epilogue: what the two of them need shares its place)
+        struct { const float* norm_w; float* out_ss; };
+        GateForm gate;       // EPI_SWIGLU: the form of the gating
+    };
     int* fault;
 };
 
@@ -126,7 +129,8 @@ struct RowFactorLoads {
 //   recv: this CTA's receive buffer (recv_floats(MT * 16, ksplit) floats); recv_bar: its barrier;
 //   pair: [2][64] floats of shared memory; row_factor: [MT * 16] floats (read when e.in_ss is set);
 //   strip: index of the strip (its first column is strip * 64), strips: strips of the product.
-template <int MT>
+// FORM: the gating of EPI_SWIGLU is the epilogue's `gate`; else silu, with nothing of the other forms in the kernel.
+template <int MT, bool FORM>
 __device__ __forceinline__ void push_reduce_store(const float (&acc)[MT][2][4], const Epilogue& e, float* recv,
                                                   unsigned long long* recv_bar, float (*pair)[STRIP],
                                                   const float* row_factor, unsigned rank, unsigned ksplit, int strip,
@@ -223,7 +227,7 @@ __device__ __forceinline__ void push_reduce_store(const float (&acc)[MT][2][4], 
             asm volatile("bar.sync 1, 128;\n" ::: "memory");
             if (valid && col < 32) {
                 const float gt = pair[half][col], up = pair[half][col + 32];
-                e.out[(size_t)row * e.ldo + strip * 32 + col] = __float2bfloat16_rn(gated_unit(gt, up, e.gate));
+                e.out[(size_t)row * e.ldo + strip * 32 + col] = __float2bfloat16_rn(FORM ? gated_unit(gt, up, e.gate) : gt / (1.f + expf(-gt)) * up);
             }
             asm volatile("bar.sync 1, 128;\n" ::: "memory");
         }

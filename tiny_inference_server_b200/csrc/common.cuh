@@ -110,6 +110,7 @@ __device__ __forceinline__ float warp_max(float v) {
 // (0.5 (1 + tanh(y)) = sigmoid(2 y)).  A finite limit with c1 = alpha, shift = 1: the clamped unit.
 struct GateForm { float limit, c1, c3, shift; };
 inline GateForm gate_silu() { GateForm f; f.limit = INFINITY; f.c1 = 1.f; f.c3 = 0.f; f.shift = 0.f; return f; }
+inline bool gate_is_silu(const GateForm& f) { return isinf(f.limit) && f.c1 == 1.f && f.c3 == 0.f && f.shift == 0.f; }
 __device__ __forceinline__ float gated_unit(float g, float u, const GateForm& f) {
     g = fminf(g, f.limit);
     u = fminf(fmaxf(u, -f.limit), f.limit);

@@ -98,7 +98,7 @@ __device__ __forceinline__ void load_x(bf16* xs, const GemmParams& p, int k0, in
     }
 }
 
-template <int MT>
+template <int MT, bool FORM>
 __global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams p) {
     namespace cg = cooperative_groups;
     extern __shared__ __align__(16) unsigned char smem[];
@@ -229,7 +229,7 @@ __global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams p) {
     __syncthreads();                    // row_factor is written (also when this CTA had no tile)
     cluster_reduce::cluster_wait();     // every CTA of the cluster has initialised its barrier
     TIS_STAMP(p, 5);
-    cluster_reduce::push_reduce_store<MT>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
+    cluster_reduce::push_reduce_store<MT, FORM>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
                                           gridDim.x, tid);
     TIS_STAMP(p, 6);
 }
@@ -283,9 +283,11 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
     }
     GemmParams p;
     p.x = (const bf16*)x; p.ldx = ldx; p.w = (const bf16*)w; p.ldw = ldw; p.K = K;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
-    p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss; p.e.fault = fault;
+    p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss;
+    p.e.fault = fault;
+    if (epi == EPI_SWIGLU) p.e.gate = gate;
     TIS_TIMELINE_TAKE(p);
     p.kc = ((K + ksplit - 1) / ksplit + BK - 1) / BK * BK;
     const int mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4);
@@ -311,14 +313,23 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
     cudaError_t e;
     static bool configured = false;
     if (!configured) {
-        cudaFuncSetAttribute(gemm_skinny_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
-        cudaFuncSetAttribute(gemm_skinny_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
-        cudaFuncSetAttribute(gemm_skinny_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<4, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
         configured = true;
     }
-    if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<1>, p);
-    else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<2>, p);
-    else e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<4>, p);
+    if (epi == EPI_SWIGLU && !gate_is_silu(gate)) {
+        if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<1, true>, p);
+        else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<2, true>, p);
+        else e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<4, true>, p);
+    } else {
+        if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<1, false>, p);
+        else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<2, false>, p);
+        else e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<4, false>, p);
+    }
     if (e != cudaSuccess) {
         tis_set_error("gemm_skinny: %s", cudaGetErrorString(e));
         return TIS_CUDA_ERROR;

@@ -63,7 +63,7 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const unsigned (&a)[4], 
 // A fifth warp does nothing but order weights (one lane orders the boxes); the four consumer warps never
 // meet inside the loop.  (The same with the producer warp copying 16-byte chunks by cp.async instead was
 // measured too: 9.1 us against 6.3 us for the down projection, one warp cannot issue them fast enough.)
-template <int MT>
+template <int MT, bool FORM>
 __global__ void __launch_bounds__(NTH + 32) gemm_stream_kernel(const __grid_constant__ CUtensorMap wmap, const StreamParams p) {
     namespace cg = cooperative_groups;
     extern __shared__ unsigned char smem_raw[];
@@ -205,7 +205,7 @@ __global__ void __launch_bounds__(NTH + 32) gemm_stream_kernel(const __grid_cons
     cluster_reduce::cluster_wait();         // every CTA of the cluster has initialised its barrier
     TIS_STAMP(p, 5);
     if (!producer)
-        cluster_reduce::push_reduce_store<MT>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
+        cluster_reduce::push_reduce_store<MT, FORM>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
                                               gridDim.x, tid);
     TIS_STAMP(p, 6);
 }
@@ -258,9 +258,10 @@ TIS_API int tis_gemm_stream_fused(const void* x, int ldx, const void* w, int ldw
     if (!tensor_map(w, N, K, ldw, BK, true, &wm)) return TIS_CUDA_ERROR;
     StreamParams p;
     p.x = (const bf16*)x; p.ldx = ldx; p.K = K;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate; p.e.fault = fault;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.fault = fault;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
     p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss;
+    if (epi == EPI_SWIGLU) p.e.gate = gate;
     TIS_TIMELINE_TAKE(p);
     p.kc = ((K + ksplit - 1) / ksplit + BK - 1) / BK * BK;
     const int mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4);
@@ -290,14 +291,23 @@ TIS_API int tis_gemm_stream_fused(const void* x, int ldx, const void* w, int ldw
     cudaError_t e;
     static bool configured = false;
     if (!configured) {
-        cudaFuncSetAttribute(gemm_stream_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
-        cudaFuncSetAttribute(gemm_stream_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
-        cudaFuncSetAttribute(gemm_stream_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<4, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_stream_kernel<4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
         configured = true;
     }
-    if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<1>, wm, p);
-    else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<2>, wm, p);
-    else e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<4>, wm, p);
+    if (epi == EPI_SWIGLU && !gate_is_silu(gate)) {
+        if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<1, true>, wm, p);
+        else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<2, true>, wm, p);
+        else e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<4, true>, wm, p);
+    } else {
+        if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<1, false>, wm, p);
+        else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<2, false>, wm, p);
+        else e = cudaLaunchKernelEx(&cfg, gemm_stream_kernel<4, false>, wm, p);
+    }
     if (e != cudaSuccess) {
         tis_set_error("gemm_stream: %s", cudaGetErrorString(e));
         return TIS_CUDA_ERROR;

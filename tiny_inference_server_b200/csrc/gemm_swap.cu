@@ -370,9 +370,10 @@ TIS_API int tis_gemm_swap_fused(const void* x, int ldx, const void* w, int ldw, 
     if (!tensor_map(w, N, K, ldw, BK, true, &mw) || !tensor_map(x, K, M, ldx, nb, true, &mx)) return TIS_CUDA_ERROR;
     SwapParams p;
     p.K = K; p.stages = 0;
-    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.gate = gate; p.e.fault = fault;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = epi; p.e.fault = fault;
     p.e.in_ss = in_ss; p.e.in_parts = in_parts; p.e.in_factor = norm_factor(in_kind, in_width, in_eps);
     p.e.res = res; p.e.ldr = ldr; p.e.norm_w = norm_w; p.e.out_ss = out_ss;
+    if (epi == EPI_SWIGLU) p.e.gate = gate;
     p.kc = ((K + ksplit - 1) / ksplit + BK - 1) / BK * BK;
     if (nb == 16) return launch_swap<16>(mw, mx, p, ksplit, stream);
     if (nb == 32) return launch_swap<32>(mw, mx, p, ksplit, stream);

@@ -58,6 +58,14 @@ rotate_norm_vec_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restri
 #pragma unroll
         for (int k = 0; k < VPL; ++k) {
             const int e = (lane + LPH * k) * N;
+            if (N == 8 && (p.rot & 7) == 0) {                 // a vector is rotated as a whole or not at all
+                const bool in = e < p.rot;
+                const float4 c4 = in ? *reinterpret_cast<const float4*>(ct + (e >> 1)) : make_float4(1.f, 1.f, 1.f, 1.f);
+                const float4 s4 = in ? *reinterpret_cast<const float4*>(st + (e >> 1)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                cs[k][0] = c4.x; cs[k][1] = c4.y; cs[k][N / 2 - 2] = c4.z; cs[k][N / 2 - 1] = c4.w;
+                sn[k][0] = s4.x; sn[k][1] = s4.y; sn[k][N / 2 - 2] = s4.z; sn[k][N / 2 - 1] = s4.w;
+                continue;
+            }
 #pragma unroll
             for (int j = 0; j < N / 2; ++j) {
                 const bool in = e + 2 * j < p.rot;
