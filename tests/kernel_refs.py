@@ -67,6 +67,8 @@ def embed_rows(table, tokens, out, scale=1.0):
 
 def _norm_factor(x, eps, kind):
     d = x.shape[-1]
+    if kind == "none":
+        return torch.ones_like(x[..., :1])
     if kind == "mean_eps":
         return 1.0 / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
     return math.sqrt(d) / (x.pow(2).sum(-1, keepdim=True).sqrt() + eps)
@@ -82,6 +84,9 @@ def add_rmsnorm(residual, delta, scale, eps, out, kind="l2_eps", delta_norm=None
     if out is None:
         return None
     d = residual.shape[-1]
+    if kind == "none":
+        out.copy_((residual * scale).to(out.dtype))
+        return out
     if kind == "mean_eps":
         out.copy_((residual / torch.sqrt(residual.pow(2).mean(-1, keepdim=True) + eps) * scale).to(out.dtype))
         return out
@@ -123,6 +128,8 @@ def activation(x, out, kind):
         y = torch.clamp(z, min=0.0) ** 2
     elif kind == "gelu_tanh":
         y = 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+    elif kind == "tanh":
+        y = torch.tanh(z)
     else:
         y = z * torch.sigmoid(z)
     out.copy_(y.to(out.dtype))
@@ -195,8 +202,14 @@ def norm_mix_store(qkv, nq, nk, nv, q_weight, k_weight, eps, v_other, mix, k_pag
         v_pages[page, :, pos % page_size, :] = v.view(kv_heads, -1).to(v_pages.dtype)
 
 
+def first_key(pos, window, chunked):
+    if not window:
+        return 0
+    return pos // window * window if chunked else max(0, pos - window + 1)
+
+
 def window_attention(q, gate, out, k_pages, v_pages, block_table, positions, row_slot, num_heads, page_size, window,
-                     scale, bias_slope, bias_rate, fault, step=None, sink=None, gate_per_head=False):
+                     scale, bias_slope, bias_rate, fault, step=None, sink=None, gate_per_head=False, chunked=False, softcap=None):
     kv_heads, k_dim, v_dim = k_pages.shape[1], k_pages.shape[3], v_pages.shape[3]
     g = num_heads // kv_heads
     for r in range(q.shape[0]):
@@ -204,13 +217,15 @@ def window_attention(q, gate, out, k_pages, v_pages, block_table, positions, row
         if slot < 0:
             continue
         pos = int(positions[r])
-        lo = max(0, pos - window + 1) if window else 0
+        lo = first_key(pos, window, chunked)
         idx = torch.arange(lo, pos + 1)
         pages = block_table[slot, idx // page_size].long()
         k = k_pages[pages, :, idx % page_size, :].to(torch.float32).repeat_interleave(g, dim=1)     # (L, H, k_dim)
         v = v_pages[pages, :, idx % page_size, :].to(torch.float32).repeat_interleave(g, dim=1)
         qq = q[r].to(torch.float32).view(num_heads, k_dim)
         s = torch.einsum("hd,khd->hk", qq, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         if bias_slope is not None:
             s = s - bias_slope[:, None] * torch.log(1.0 + bias_rate[:, None] * (pos - idx).to(torch.float32)[None, :])
         if sink is not None:               # one more term in the denominator, without a value
@@ -412,20 +427,23 @@ def gated(g, u, form=None):
     return g * torch.sigmoid(g * (form.c1 + form.c3 * g * g)) * (torch.clamp(u, min=-form.limit, max=form.limit) + form.shift)
 
 
-def moe_gate_up(x, chosen, w_gate_up, act=None, form=None):
+def moe_gate_up(x, chosen, w_gate_up, act=None, form=None, in_weights=None):
     n, top = chosen.shape
-    xf = x.to(torch.float32)
+    xf = x.to(torch.float32)[:, None, :].expand(n, top, x.shape[1])
+    if in_weights is not None:
+        xf = xf * in_weights[:, :, None]
     if act is not None:
-        u = torch.einsum("ntfd,nd->ntf", w_gate_up.to(torch.float32)[chosen.long()], xf)
+        u = torch.einsum("ntfd,ntd->ntf", w_gate_up.to(torch.float32)[chosen.long()], xf)
         return _act(u, act).reshape(n * top, -1).to(x.dtype)
     w = w_gate_up.to(torch.float32)[chosen.long()]                      # (n, top, 2, F, d)
-    g = torch.einsum("ntfd,nd->ntf", w[:, :, 0], xf)
-    u = torch.einsum("ntfd,nd->ntf", w[:, :, 1], xf)
+    g = torch.einsum("ntfd,ntd->ntf", w[:, :, 0], xf)
+    u = torch.einsum("ntfd,ntd->ntf", w[:, :, 1], xf)
     return gated(g, u, form).reshape(n * top, -1).to(x.dtype)
 
 
-def moe_experts(x, chosen, weights, w_gate_up, w_down, shared, shared_gate, act=None, form=None):
-    return moe_down(moe_gate_up(x, chosen, w_gate_up, act, form), chosen, weights, w_down, shared, shared_gate)
+def moe_experts(x, chosen, weights, w_gate_up, w_down, shared, shared_gate, act=None, form=None, weigh_input=False):
+    hid = moe_gate_up(x, chosen, w_gate_up, act, form, weights if weigh_input else None)
+    return moe_down(hid, chosen, None if weigh_input else weights, w_down, shared, shared_gate)
 
 
 def gated_linear_attention(qkv, a_in, power, a_bias, gate, norm_weight, eps, q_scale, state, out, row_slot, row_last,
@@ -478,6 +496,52 @@ def skip_gate_group_norm(o_raw, x, skip, z, weight, groups, eps, out, row_slot, 
     parts = y.view(n, groups, d // groups)
     y = (parts / torch.sqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).reshape(n, d) * weight
     out[:] = y.to(out.dtype)
+    return out
+
+
+def token_shift(x, mu, state, row_slot, row_last):
+    n, d = x.shape
+    out = torch.zeros((n, mu.shape[0], d), dtype=x.dtype)
+    for r0, rows, slot in _segments(row_slot):
+        seq = torch.cat([state[slot, :d][None].to(torch.float32), x[r0:r0 + rows].to(torch.float32)])
+        h, before = seq[1:], seq[:-1]
+        out[r0:r0 + rows] = (h[:, None] + (before - h)[:, None] * mu[None]).to(x.dtype)
+        state[slot, :d] = seq[-1]
+    return out
+
+
+def gemm_side_by_side(a, w, w_last, act=None):
+    out = torch.einsum("ngk,gkj->ngj", a[:, :w.shape[0]].to(torch.float32), w.to(torch.float32)).to(a.dtype)
+    last = gemm(a[:, w.shape[0]], w_last)
+    return out.reshape(a.shape[0], -1), last if act is None else activation(last, last, act)
+
+
+def time_mix(rkvg, w_in, u, w_bias, norm_weight, eps, state, out, row_slot, row_last, num_heads, dim, requests=None, segments=None):
+    H, D = num_heads, dim
+    for r0, rows, slot in _segments(row_slot):
+        S = state[slot, :H * D * D].reshape(H, D, D).to(torch.float32).clone()
+        for t in range(r0, r0 + rows):
+            r, k, v, g = rkvg[t, :4 * H * D].to(torch.float32).view(4, H, D)
+            decay = torch.exp(-torch.exp(w_in[t].to(torch.float32).view(H, D) + w_bias.view(H, D)))
+            kv = k[:, :, None] * v[:, None, :]
+            o = torch.einsum("hkv,hk->hv", S + u.view(H, D)[:, :, None] * kv, r)
+            S = decay[:, :, None] * S + kv
+            o = (o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps)).reshape(-1) * norm_weight
+            out[t] = (o * (g * torch.sigmoid(g)).reshape(-1)).to(out.dtype)
+        state[slot, :H * D * D] = S.reshape(-1)
+    return out
+
+
+def selective_scan(x, dt_in, dt_bias, a_log, b, c, skip, z, state, out, row_slot, row_last, segments=None):
+    I, N = a_log.shape
+    for r0, rows, slot in _segments(row_slot):
+        S = state[slot, :I * N].reshape(I, N).to(torch.float32).clone()
+        for t in range(r0, r0 + rows):
+            dt = torch.nn.functional.softplus(dt_in[t] + dt_bias)
+            xt, zt = x[t].to(torch.float32), z[t].to(torch.float32)
+            S = torch.exp(-dt[:, None] * torch.exp(a_log)) * S + (dt * xt)[:, None] * b[t].to(torch.float32)[None]
+            out[t] = ((S @ c[t].to(torch.float32) + skip * xt) * zt * torch.sigmoid(zt)).to(out.dtype)
+        state[slot, :I * N] = S.reshape(-1)
     return out
 
 
@@ -546,9 +610,13 @@ def add_layer_norm(residual, delta_a, delta_b, w, b, eps, out):
 
 
 def rotate_norm_store(qkv, num_heads, kv_heads, dim, v_dim, cos, sin, interleaved, norm, eps, k_pages, v_pages, block_table,
-                      positions, row_slot, page_size, fault, permuted=False):
+                      positions, row_slot, page_size, fault, permuted=False, whole_weight=None):
     def prepared(z, pos):               # (heads, dim)
         out = z.to(torch.float32).clone()
+        if whole_weight is not None:    # all query heads at once, all key heads at once, before the rotation
+            for part in (out[:num_heads], out[num_heads:]):
+                part /= torch.sqrt(part.pow(2).mean() + eps)
+            out *= whole_weight.view(-1, dim)
         if cos is not None:
             half = cos.shape[1]
             ia = torch.arange(half) * 2 if interleaved else torch.arange(half)
@@ -556,7 +624,7 @@ def rotate_norm_store(qkv, num_heads, kv_heads, dim, v_dim, cos, sin, interleave
             a, b = out[:, ia].clone(), out[:, ib].clone()
             out[:, ia] = a * cos[pos] - b * sin[pos]
             out[:, ib] = b * cos[pos] + a * sin[pos]
-        if norm:
+        if norm and whole_weight is None:
             out = out / torch.sqrt(out.pow(2).mean(-1, keepdim=True) + eps)
         return out
 
@@ -582,7 +650,7 @@ def moe_down(hidden, chosen, weights, w_down, shared, shared_gate):
     n, top = chosen.shape
     h = hidden.to(torch.float32).view(n, top, -1)
     y = torch.einsum("ntdf,ntf->ntd", w_down.to(torch.float32)[chosen.long()], h)
-    out = (y * weights[:, :, None]).sum(1)
+    out = (y * weights[:, :, None]).sum(1) if weights is not None else y.sum(1)
     if shared is not None:
         out = out + (shared_gate[:, None] if shared_gate is not None else 1.0) * shared.to(torch.float32)
     return out.to(hidden.dtype)
@@ -687,7 +755,8 @@ def rotary_fusable(q, step, num_heads, kv_heads, head_dim, pairs=False):
 
 
 def paged_attention(q, out, plane, block_table, positions, row_slot, num_heads, kv_heads, head_dim, page_size,
-                    window, fault, step=None, rotary=None, write_kv=True, scale=None, sink=None):
+                    window, fault, step=None, rotary=None, write_kv=True, scale=None, sink=None, chunked=False, softcap=None,
+                    gate=None):
     from tiny_inference_server_b200.kernels import ops
     scale = 1.0 / math.sqrt(head_dim) if scale is None else scale
     if isinstance(rotary, ops.PairRotary):
@@ -707,16 +776,21 @@ def paged_attention(q, out, plane, block_table, positions, row_slot, num_heads, 
             continue
         pos = int(positions[r])
         hi = pos + 1
-        lo = max(0, hi - window) if window else 0
+        lo = first_key(pos, window, chunked)
         k, v = gather_kv(plane, block_table, slot, lo, hi, page_size)
         k = k.repeat_interleave(g, dim=1)
         v = v.repeat_interleave(g, dim=1)
         qq = q[r, :hq].to(torch.float32).view(num_heads, head_dim)
         s = torch.einsum("hd,khd->hk", qq, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         if sink is not None:
             s = torch.cat([s, sink.to(torch.float32)[:, None]], dim=1)
         p = torch.softmax(s, dim=-1)[:, :k.shape[0]]
-        out[r] = torch.einsum("hk,khd->hd", p, v).reshape(-1).to(out.dtype)
+        o = torch.einsum("hk,khd->hd", p, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[r, :num_heads].to(torch.float32))[:, None]
+        out[r] = o.reshape(-1).to(out.dtype)
     return out
 
 
@@ -842,7 +916,7 @@ _NAMES = ["rotary_fusable", "gemm", "gemm_f32_out", "gemm_swiglu", "embed_rows",
           "norm_mix_store", "window_attention", "delta_rule", "linear_attention", "latent_prepare", "gemm_heads", "moe_route",
           "moe_gate_up", "moe_down", "moe_experts", "gated_linear_attention", "state_space_scan", "skip_gate_group_norm",
           "embed_pairs", "group_norm", "rotate_tie_store", "scaled_sum", "add_layer_norm",
-          "rotate_norm_store"]
+          "rotate_norm_store", "token_shift", "gemm_side_by_side", "time_mix", "selective_scan"]
 
 
 def install(monkeypatch) -> None:

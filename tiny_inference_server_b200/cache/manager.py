@@ -28,7 +28,7 @@ class CacheManager:
         keys, lags, self.plane_refs = group_planes(kv_specs)
         self.groups: List[CacheGroup] = [
             CacheGroup(g, k[0], k[1], k[3], lags[k], page_size, num_pages, max_slots, max_positions, dtype,
-                       self.device, v_dim=k[2], poison=debug_poison)
+                       self.device, v_dim=k[2], poison=debug_poison, chunks=k[4])
             for g, k in enumerate(keys)
         ]
         self.states: Dict[str, torch.Tensor] = {
@@ -94,7 +94,7 @@ class CacheManager:
         need = 0
         for g in self.groups:
             grow = g.pages_to_grow(slot, start + n_new)
-            if g.window is not None:
+            if g.trims:
                 grow -= g.pages_freed_by(slot, start)
             need = max(need, grow)
         return max(0, need)
@@ -116,7 +116,7 @@ class CacheManager:
             if grow and grow - g.pages_freed_by(slot, start) > g.pool.free:
                 raise OutOfPages(f"group {g.gid}: {grow} pages needed, {g.pool.free} free")
         for g in self.groups:
-            if g.window is not None:
+            if g.trims:
                 g.trim(slot, start)
             if new_len > g.end[slot] * g.page_size:
                 g.grow(slot, new_len)

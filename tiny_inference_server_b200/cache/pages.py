@@ -3,7 +3,7 @@
 Upstream keeps one pool tensor for all layers, a deque of free page ids and a python
 list of page ids per request (``block_table.py:31-86``).  Here the planes (one per
 cached layer) are first grouped by what they need — kv heads, the widths of a key and of a
-value row, and whether they keep every key or a window of them — and every group has pages of its own: a pool
+value row, and whether they keep every key, a window of them or the current chunk — and every group has pages of its own: a pool
 tensor ``[planes, pages, 2, kv_heads, page_size, head_dim]``, a free list, and one
 block table per request slot.  A page id addresses the same page in every plane of its
 group, as upstream's does in every layer.
@@ -108,13 +108,16 @@ class CacheGroup:
 
     def __init__(self, gid: int, kv_heads: int, head_dim: int, window: Optional[int], lags: Sequence[int],
                  page_size: int, num_pages: int, max_slots: int, max_positions: int, dtype: torch.dtype,
-                 device: torch.device, v_dim: Optional[int] = None, poison: bool = False):
+                 device: torch.device, v_dim: Optional[int] = None, poison: bool = False, chunks: Sequence[int] = ()):
         self.gid = gid
         self.poison = poison                      # fill pages with POISON when they are given back
         self.kv_heads = kv_heads
         self.head_dim = head_dim                  # elements of a key row
         self.v_dim = head_dim if v_dim is None else v_dim      # elements of a value row
         self.window = window
+        self.chunks = tuple(chunks)               # the readers see keys of their own chunk only (of any of these sizes)
+        if window is not None and self.chunks:
+            raise CacheError("a group keeps a window or chunks")
         self.lags = list(lags)                    # per plane: how far it is filled behind the trunk
         self.max_lag = max(self.lags) if self.lags else 0
         self.page_size = page_size
@@ -162,14 +165,21 @@ class CacheGroup:
         n = self.kv_heads * self.page_size * self.head_dim
         return self.pages[index][:, n:].unflatten(1, (self.kv_heads, self.page_size, self.v_dim))
 
+    @property
+    def trims(self) -> bool:
+        """Whether pages fall out of sight while their request lives."""
+        return self.window is not None or bool(self.chunks)
+
     # ---- planning ---------------------------------------------------------------------
     def dead_before(self, start_pos: int) -> int:
         """First logical page that a step feeding positions from ``start_pos`` on can still
         read.  Without a window every page stays.  With a window W the plane that lags most
-        reads keys from (start_pos - lag) - W + 1 on."""
-        if self.window is None:
+        reads keys from (start_pos - lag) - W + 1 on.  With chunks: from the start of the chunk that the plane which
+        lags most is in, by the chunk size that reaches back furthest."""
+        if not self.trims:
             return 0
-        lowest = start_pos - self.max_lag - self.window + 1
+        at = max(0, start_pos - self.max_lag)
+        lowest = at - self.window + 1 if self.window is not None else min(at - at % c for c in self.chunks)
         return max(0, lowest) // self.page_size
 
     def pages_to_grow(self, slot: int, new_len: int) -> int:
@@ -241,7 +251,7 @@ class CacheGroup:
 
 def group_planes(specs: Sequence[Optional[KVSpec]]):
     """Group the kv specs of the schedule entries: returns ([group key], [PlaneRef or None]).
-    Entries with equal (kv_heads, key width, value width, window) share a group."""
+    Entries with equal (kv_heads, key width, value width, window, chunks) share a group."""
     keys: List[tuple] = []
     lags: Dict[tuple, List[int]] = {}
     refs: List[Optional[PlaneRef]] = []

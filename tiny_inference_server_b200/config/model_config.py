@@ -970,3 +970,177 @@ class LomutarConfig:
         if self.eos_token_id is not None:
             d["eos_token_id"] = self.eos_token_id
         return d
+
+
+@dataclass
+class TazadraConfig:
+    """Configuration of the Tazadra decoder: layers whose sublayers read the stream as it is and whose updates pass a norm and a
+    constant factor; three kinds of mixer; a dense or a routed feed-forward; an output matrix of its own, logits bounded smoothly.
+
+    ``config.json`` is nested: ``vocab``, ``width``, ``norm.eps``, ``residual_mult`` (1 unless given), ``logit_softcap`` (null or
+    absent: none) and ``layers``, a list with, per layer, ``type``, ``mixer`` and ``mlp`` (null: none).  The kinds:
+
+    * ``mamba1`` — ``inner, state, dt_rank, conv``: a selective scan;
+    * ``attention`` — ``heads, kv_heads, dim, vdim, scale``, and optionally ``softcap``, ``rot`` = ``base, dims`` and ``scaling`` =
+      ``factor, low, high, original``, ``mask.size`` (the positions of a chunk; no ``mask``: every earlier key is seen) and
+      ``kv_from`` (an earlier attention layer with keys and values of its own, which this layer reads);
+    * ``wkv`` — ``heads, dim``: a matrix state with a decay per key channel; the rank of the decay's projection is the first
+      dimension of the tensor ``l<i>.mix.w1`` (``complete_from_shapes``).
+
+    ``mlp``: ``kind`` ``dense`` with ``ff, limit``, or ``moe`` with ``expert.ff`` and ``router`` = ``experts, top``.  The design has
+    no context limit of its own: ``max_context`` (optional) bounds what the engine lays out (block tables, rotation tables)."""
+
+    architecture: ClassVar[str] = "Tazadra"
+    MIXERS: ClassVar[dict] = {"mamba1": ("inner", "state", "dt_rank", "conv"), "attention": ("heads", "kv_heads", "dim", "vdim"),
+                              "wkv": ("heads", "dim")}
+
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float = 1e-6
+    residual_mult: float = 1.0
+    logit_softcap: Optional[float] = None
+    max_context: int = 1 << 16
+    eos_token_id: Optional[int] = None
+    torch_dtype: str = "bfloat16"
+
+    def __post_init__(self):
+        errs = []
+        for name in ("vocab_size", "hidden_size", "max_context"):
+            if not _positive_int(getattr(self, name)):
+                errs.append(f"{name} must be a positive integer, got {getattr(self, name)!r}")
+        if not isinstance(self.layers, list) or not self.layers:
+            errs.append("layers must be a non-empty list")
+            raise ConfigError("; ".join(errs))
+        if not (self.norm_eps >= 0):
+            errs.append(f"norm.eps must be >= 0, got {self.norm_eps}")
+        if not _number(self.residual_mult):
+            errs.append(f"residual_mult must be a number, got {self.residual_mult!r}")
+        if self.logit_softcap is not None and not (_number(self.logit_softcap) and self.logit_softcap > 0):
+            errs.append(f"logit_softcap must be positive or null, got {self.logit_softcap!r}")
+        for i, layer in enumerate(self.layers):
+            kind = layer.get("type") if isinstance(layer, dict) else None
+            if kind not in self.MIXERS:
+                errs.append(f"layers[{i}].type must be one of {tuple(self.MIXERS)}, got {kind!r}")
+                continue
+            m = layer.get("mixer")
+            bad = [k for k in self.MIXERS[kind] if not isinstance(m, dict) or not _positive_int(m.get(k))]
+            if bad:
+                errs.append(f"layers[{i}].mixer: {', '.join(bad)} must be positive integers")
+                continue
+            if kind == "attention":
+                errs += self._attention_errors(i, m)
+            elif kind == "mamba1":
+                if m["conv"] > 16:
+                    errs.append(f"layers[{i}].mixer.conv must be 1..16, got {m['conv']}")
+                if m["state"] > 256:
+                    errs.append(f"layers[{i}].mixer.state must be at most 256, got {m['state']}")
+            if layer.get("mlp") is not None:
+                errs += self._mlp_errors(i, layer["mlp"])
+        if self.torch_dtype not in ("bfloat16", "float32"):
+            errs.append(f"torch_dtype must be bfloat16 or float32, got {self.torch_dtype!r}")
+        if errs:
+            raise ConfigError("; ".join(errs))
+
+    def _attention_errors(self, i: int, m: dict) -> list:
+        at, errs = f"layers[{i}].mixer", []
+        if m["heads"] % m["kv_heads"]:
+            errs.append(f"{at}: {m['heads']} heads are not a multiple of {m['kv_heads']} kv heads")
+        if not _number(m.get("scale")):
+            errs.append(f"{at}.scale is missing")
+        cap = m.get("softcap")
+        if cap is not None and not (_number(cap) and cap > 0):
+            errs.append(f"{at}.softcap must be a positive number or null")
+        mask = m.get("mask")
+        if mask is not None and not (isinstance(mask, dict) and _positive_int(mask.get("size"))):
+            errs.append(f"{at}.mask.size must be a positive integer")
+        rot = m.get("rot")
+        if rot is not None:
+            if not isinstance(rot, dict) or not _number(rot.get("base")) or not rot["base"] > 0:
+                errs.append(f"{at}.rot.base is missing")
+            elif not _positive_int(rot.setdefault("dims", m["dim"])) or rot["dims"] % 2 or rot["dims"] > m["dim"]:
+                errs.append(f"{at}: rot.dims must be even and at most dim ({m['dim']})")
+            elif rot.get("scaling"):
+                miss = [k for k in ("factor", "low", "high", "original") if not _number(rot["scaling"].get(k))]
+                if miss:
+                    errs.append(f"{at}.rot.scaling lacks {', '.join(miss)}")
+                elif not rot["scaling"]["factor"] > 0:
+                    errs.append(f"{at}.rot.scaling.factor must be positive")
+        j = m.get("kv_from")
+        if j is not None:
+            if not isinstance(j, int) or isinstance(j, bool) or not 0 <= j < i:
+                errs.append(f"{at}.kv_from must name an earlier layer, got {j!r}")
+            else:
+                src = self.layers[j] if isinstance(self.layers[j], dict) else {}
+                sm = src.get("mixer")
+                if src.get("type") != "attention" or not isinstance(sm, dict) or sm.get("kv_from") is not None:
+                    errs.append(f"{at}.kv_from: layer {j} has no keys and values of its own")
+                elif any(sm.get(k) != m[k] for k in ("kv_heads", "dim", "vdim")):
+                    errs.append(f"{at}.kv_from: kv_heads, dim and vdim of layer {j} differ from this layer's")
+        return errs
+
+    @staticmethod
+    def _mlp_errors(i: int, f: dict) -> list:
+        at = f"layers[{i}].mlp"
+        if not isinstance(f, dict) or f.get("kind") not in ("dense", "moe"):
+            return [f"{at}.kind must be 'dense' or 'moe', got {f.get('kind') if isinstance(f, dict) else f!r}"]
+        errs = []
+        if f["kind"] == "dense":
+            if not _positive_int(f.get("ff")):
+                errs.append(f"{at}.ff must be a positive integer")
+            if not _number(f.get("limit")) or not f["limit"] > 0:
+                errs.append(f"{at}.limit must be a positive number")
+            return errs
+        if not isinstance(f.get("expert"), dict) or not _positive_int(f["expert"].get("ff")):
+            errs.append(f"{at}.expert.ff must be a positive integer")
+        r = f.get("router")
+        if not isinstance(r, dict) or not _positive_int(r.get("experts")) or not _positive_int(r.get("top")):
+            errs.append(f"{at}.router needs experts and top")
+        elif r["top"] > r["experts"]:
+            errs.append(f"{at}.router.top {r['top']} exceeds the {r['experts']} experts")
+        return errs
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def cache_chunks(self, i: int) -> tuple:
+        """The sizes of the chunks that layer i's plane is read by (its owner's and those of the layers that read it); empty:
+        one of them sees every key."""
+        owner = self.layers[i]["mixer"].get("kv_from")
+        owner = i if owner is None else owner
+        masks = [layer["mixer"].get("mask") for j, layer in enumerate(self.layers)
+                 if layer["type"] == "attention" and (j == owner or layer["mixer"].get("kv_from") == owner)]
+        return () if any(not m for m in masks) else tuple(sorted({m["size"] for m in masks}))
+
+    def complete_from_shapes(self, shapes: dict) -> None:
+        """The rank of a ``wkv`` mixer's decay projection is not in config.json: it is the first dimension of the layer's
+        ``mix.w1``."""
+        for i, layer in enumerate(self.layers):
+            if layer["type"] == "wkv" and "decay_rank" not in layer["mixer"]:
+                name = f"l{i}.mix.w1"
+                if name not in shapes or len(shapes[name]) != 2:
+                    raise ConfigError(f"the tensor {name!r} (rank, width) is missing: it gives the rank of layer {i}'s decay "
+                                      f"projection")
+                layer["mixer"]["decay_rank"] = int(shapes[name][0])
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "TazadraConfig":
+        missing = [k for k in ("vocab", "width", "layers") if k not in raw]
+        if missing:
+            raise ConfigError(f"config for architecture {cls.architecture!r}: missing keys: " + ", ".join(missing))
+        d = dict(vocab_size=raw["vocab"], hidden_size=raw["width"], layers=copy.deepcopy(raw["layers"]))
+        if isinstance(raw.get("norm"), dict) and "eps" in raw["norm"]:
+            d["norm_eps"] = float(raw["norm"]["eps"])
+        for k in ("residual_mult", "logit_softcap", "max_context", "eos_token_id", "torch_dtype"):
+            if raw.get(k) is not None:
+                d[k] = raw[k]
+        return cls(**d)
+
+    def to_dict(self) -> dict:
+        d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+             "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult, "logit_softcap": self.logit_softcap,
+             "layers": copy.deepcopy(self.layers), "max_context": self.max_context, "torch_dtype": self.torch_dtype}
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d

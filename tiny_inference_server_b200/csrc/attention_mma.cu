@@ -67,6 +67,8 @@ struct AttnParams {
     const int* tile_row0; const int* tile_rows;
     int H, KVH, G, page_size, window;
     float scale_log2;
+    SoftCap cap;            // bounds the raw scores (k 0: not)
+    const bf16* gate; int ldg;      // (n, H): head h's output times sigmoid(gate[row][h]) (null: none)
     int keys_per_split, num_splits;
     float* part_o; float* part_lse;
     int cluster_merge;      // the splits of a (tile, kv head) are one thread-block cluster and merge through
@@ -210,6 +212,11 @@ __device__ __forceinline__ void add_sink(float& num, float& den, float mt, float
     const float f = mt == -INFINITY ? 0.f : fast_exp2(mt - m);
     num *= f;
     den = den * f + fast_exp2(s2 - m);
+}
+
+// What the gate multiplies head hq's output of a row with.
+__device__ __forceinline__ float head_gate(const AttnParams& p, int row, int hq) {
+    return 1.f / (1.f + __expf(-__bfloat162float(p.gate[(size_t)row * p.ldg + hq])));
 }
 
 // FUSED_PAIRS: the queries' fragments rotated and normed in registers.  Columns 2t and 2t + 1 of a fragment are a rotation
@@ -401,6 +408,7 @@ __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, uns
             }
         }
         if (SINK && p.sink != nullptr) add_sink(acc, lsum, mt, p.sink[kvh * G + g]);
+        if (SINK && p.gate != nullptr) acc *= head_gate(p, row0 + r, kvh * G + g);
         p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
             __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
     }
@@ -472,7 +480,7 @@ attn_mma_kernel(const AttnParams p) {
         head[i] = kvh * G + g;
         const int pos = valid[i] ? p.positions[r_idx[i]] : 0;
         hi_row[i] = valid[i] ? pos + 1 : 0;
-        lo_row[i] = (valid[i] && p.window > 0 && hi_row[i] > p.window) ? hi_row[i] - p.window : 0;
+        lo_row[i] = valid[i] ? first_key(pos, p.window) : 0;
     }
 
     // key range of the tile and of this split
@@ -481,9 +489,9 @@ attn_mma_kernel(const AttnParams p) {
         slot = p.row_slot[row0 + rows - 1];
         const int pos_first = p.positions[row0 + first], pos_last = p.positions[row0 + rows - 1];
         range_hi = pos_last + 1;
-        range_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
+        range_lo = first_key(pos_first, p.window);
         // the splits share out the keys from the window's first tile on
-        const int base = p.window > 0 ? range_lo / KT * KT : 0;
+        const int base = p.window != 0 ? range_lo / KT * KT : 0;
         range_lo = max(range_lo, base + split * p.keys_per_split);
         range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
@@ -671,6 +679,12 @@ attn_mma_kernel(const AttnParams p) {
                     mma_bf16(s[j + 1], qa[kk], b[2], b[3]);
                 }
             }
+            if (p.cap.k != 0.f) {
+#pragma unroll
+                for (int j = 0; j < NT; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2 * NR; ++e) s[j][e] = soft_capped(s[j][e], p.cap);
+            }
             // ---- scale, mask (only where a row's range ends inside this tile), online softmax
             float mx[2] = {-INFINITY, -INFINITY};
             const int t_lo = kt + kofs, t_hi = kt + kofs + NT * 8;
@@ -831,6 +845,7 @@ attn_mma_kernel(const AttnParams p) {
                 }
             }
             if (FUSED != FUSED_HALVES && p.num_splits == 1 && p.sink != nullptr) add_sink(acc, lt, mt, p.sink[hq]);
+            if (FUSED != FUSED_HALVES && p.num_splits == 1 && p.gate != nullptr) acc *= head_gate(p, row, hq);
             const float val = lt > 0.f ? acc / lt : 0.f;
             if (p.num_splits == 1) {
                 p.out[(size_t)row * p.out_stride + (size_t)hq * HD + d] = __float2bfloat16_rn(val);
@@ -855,6 +870,7 @@ attn_mma_kernel(const AttnParams p) {
                     add_sink(num, den, m_run[i], p.sink[hq]);
                     inv = den > 0.f ? num / den : 0.f;
                 }
+                if (p.gate != nullptr) inv *= head_gate(p, row, hq);
                 bf16* dst = p.out + (size_t)row * p.out_stride + (size_t)hq * HD;
 #pragma unroll
                 for (int d = 0; d < DTILES; ++d)
@@ -904,6 +920,7 @@ attn_mma_kernel(const AttnParams p) {
                     }
                 }
                 if (p.sink != nullptr) add_sink(acc, wsum, mt, p.sink[kvh * G + g]);
+                if (p.gate != nullptr) acc *= head_gate(p, row0 + r, kvh * G + g);
                 p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
                     __float2bfloat16_rn(wsum > 0.f ? acc / wsum : 0.f);
             }
@@ -1027,7 +1044,7 @@ attn_decode_kernel(const AttnParams p) {
         head[i] = kvh * G + g;
         const int pos = valid[i] ? p.positions[r_idx[i]] : 0;
         hi_row[i] = valid[i] ? pos + 1 : 0;
-        lo_row[i] = (valid[i] && p.window > 0 && hi_row[i] > p.window) ? hi_row[i] - p.window : 0;
+        lo_row[i] = valid[i] ? first_key(pos, p.window) : 0;
     }
     int range_lo = 0, range_hi = 0, slot = -1;
     if (first >= 0) {
@@ -1035,9 +1052,9 @@ attn_decode_kernel(const AttnParams p) {
         const int pos_last = pos_last_early;
         const int pos_first = first == rows - 1 ? pos_last : p.positions[row0 + first];
         range_hi = pos_last + 1;
-        range_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
+        range_lo = first_key(pos_first, p.window);
         // the splits share out the keys from the window's first tile on
-        const int base = p.window > 0 ? range_lo / KT * KT : 0;
+        const int base = p.window != 0 ? range_lo / KT * KT : 0;
         range_lo = max(range_lo, base + split * p.keys_per_split);
         range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
@@ -1207,6 +1224,12 @@ attn_decode_kernel(const AttnParams p) {
                     mma_bf16(s[0], qa[kk], b[0], b[1]);
                     mma_bf16(s[1], qa[kk], b[2], b[3]);
                 }
+                if (p.cap.k != 0.f) {
+#pragma unroll
+                    for (int j = 0; j < NT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2 * NR; ++e) s[j][e] = soft_capped(s[j][e], p.cap);
+                }
                 float mx[2] = {-INFINITY, -INFINITY};
                 const int t_lo = kt + kofs, t_hi = kt + kofs + NT * 8;
                 const bool interior = t_lo >= range_lo && t_hi <= range_hi && t_lo >= lo_row[0] && t_hi <= hi_row[0] &&
@@ -1368,7 +1391,8 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
                        int max_tile_rows, int n_rows, int H, int KVH, int page_size, int window, float scale,
                        int keys_per_split, int num_splits, float* scratch, int* fault, cudaStream_t stream,
                        const float* rope_cos, const float* rope_sin, int write_kv, int rope_kind = FUSED_NONE,
-                       int rope_rot = 0, int rope_norm = 0, float rope_eps = 0.f, const float* sink = nullptr) {
+                       int rope_rot = 0, int rope_norm = 0, float rope_eps = 0.f, const float* sink = nullptr,
+                       float softcap = 0.f, const void* gate = nullptr, int ldg = 0) {
     if (num_tiles <= 0) return TIS_OK;
     const bool fused = rope_kind != FUSED_NONE, pairs_kind = rope_kind == FUSED_PAIRS;
     if (fused && (mode != MODE_KEYS || max_tile_rows != 1 || (!pairs_kind && HD % 32 != 0) ||
@@ -1386,6 +1410,10 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
     }
     if (G > mpack) {
         tis_set_error("attention: %d query heads per kv head exceed the %d packed rows of this mode", G, mpack);
+        return TIS_BAD_SIZE;
+    }
+    if (gate != nullptr && scratch != nullptr) {
+        tis_set_error("attention: key splits that merge through scratch memory take no gate");
         return TIS_BAD_SIZE;
     }
     if (keys_per_split <= 0 || keys_per_split % KT || num_splits <= 0) {
@@ -1413,6 +1441,8 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
     p.fault = fault;
     p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.rope_rot = rope_rot; p.rope_norm = rope_norm; p.rope_eps = rope_eps;
     p.sink = sink;
+    p.cap = soft_cap(softcap, scale);
+    p.gate = (const bf16*)gate; p.ldg = ldg;
     p.plane_w = (fused && write_kv) ? (bf16*)plane : nullptr;
     TIS_TIMELINE_TAKE(p);
     // decode tiles go to the kernel with a producer warp where its layout allows (page segments: two lanes each)
@@ -1588,16 +1618,17 @@ TIS_API int tis_attn_mma(int mode, const void* q, int q_stride, void* out, int o
                        keys_per_split, num_splits, scratch, fault, stream, nullptr, nullptr, 0);
 }
 
-// The same with `sink` (null: none): exp(sink[h]) is one more term of head h's softmax denominator.
+// The same with `sink` (null: none): exp(sink[h]) is one more term of head h's softmax denominator; `softcap` > 0 bounds the
+// scores, softcap * tanh(score / softcap); `gate` (n, H; null: none) multiplies head h's output by sigmoid(gate[row][h]).
 TIS_API int tis_attn_mma_sink(int mode, const void* q, int q_stride, void* out, int out_stride, const void* plane,
                               const int* block_table, int bt_stride, int num_pages, const int* positions,
                               const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
                               int max_tile_rows, int n_rows, int H, int KVH, int page_size, int window, float scale,
-                              int keys_per_split, int num_splits, float* scratch, const float* sink, int* fault,
-                              cudaStream_t stream) {
+                              int keys_per_split, int num_splits, float* scratch, const float* sink, float softcap,
+                              const void* gate, int ldg, int* fault, cudaStream_t stream) {
     return attn_launch(mode, q, q_stride, out, out_stride, plane, block_table, bt_stride, num_pages, positions, row_slot,
                        tile_row0, tile_rows, num_tiles, max_tile_rows, n_rows, H, KVH, page_size, window, scale,
-                       keys_per_split, num_splits, scratch, fault, stream, nullptr, nullptr, 0, FUSED_NONE, 0, 0, 0.f, sink);
+                       keys_per_split, num_splits, scratch, fault, stream, nullptr, nullptr, 0, FUSED_NONE, 0, 0, 0.f, sink, softcap, gate, ldg);
 }
 
 // Decode rows (tiles of one row, keys mode) whose rotary encoding and cache write this kernel does itself:

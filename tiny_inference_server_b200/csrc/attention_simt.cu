@@ -3,7 +3,8 @@
 // stay float) and works for bfloat16 pages too.
 //
 // One CTA per (query head, row).  The row at position p of the request in slot s reads
-// keys lo..p of the plane through the request's block table, lo = 0 or p-window+1.
+// keys lo..p of the plane through the request's block table, lo = first_key(p, window) (common.cuh).  `softcap` > 0 bounds
+// the scores, `gate` (n, H; null: none) multiplies head h's output by sigmoid(gate[row][h]).
 // Keys are taken 128 at a time: every thread scores one key, the CTA agrees on the new
 // running maximum, then the threads split the head dimension and add the 128 weighted
 // value rows (online softmax, as paged_attention_kernels.py:88-111 upstream, in base e).
@@ -34,8 +35,8 @@ __global__ void __launch_bounds__(SIMT_KEYS)
 paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out, int out_stride,
                             const T* __restrict__ plane, const int* __restrict__ block_table, int bt_stride,
                             int num_pages, const int* __restrict__ positions, const int* __restrict__ row_slot,
-                            int H, int KVH, int hd, int page_size, int window, float scale,
-                            const float* __restrict__ sink, int* __restrict__ fault) {
+                            int H, int KVH, int hd, int page_size, int window, float scale, float softcap,
+                            const T* __restrict__ gate, int ldg, const float* __restrict__ sink, int* __restrict__ fault) {
     extern __shared__ float smem[];
     float* qs = smem;                      // hd
     float* ps = smem + hd;                 // SIMT_KEYS
@@ -51,7 +52,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
     }
     const int pos = positions[r];
     const int hi = pos + 1;
-    const int lo = (window > 0 && hi > window) ? hi - window : 0;
+    const int lo = first_key(pos, window);
     const int kvh = h / (H / KVH);
     const T* qrow = q + (size_t)r * q_stride + (size_t)h * hd;
     for (int i = tid; i < hd; i += SIMT_KEYS) qs[i] = to_f32(qrow[i]);
@@ -75,6 +76,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
             } else {
                 ko = (long long)((size_t)page * page_elems + ((size_t)kvh * page_size + (j % page_size)) * hd);
                 s = dot_row<T>(qs, plane + ko, hd, j) * scale;
+                if (softcap > 0.f) s = softcap * tanhf(s / softcap);
             }
         }
         voff[tid] = ko < 0 ? -1 : ko + (long long)v_shift;
@@ -105,7 +107,8 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
         }
         __syncthreads();                       // ps, voff are rewritten by the next tile
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (gate != nullptr) inv /= 1.f + expf(-to_f32(gate[(size_t)r * ldg + h]));      // one number for the head's elements
     if (tid < hd) o[tid] = from_f32<T>(acc0 * inv);
     if (tid + SIMT_KEYS < hd) o[tid + SIMT_KEYS] = from_f32<T>(acc1 * inv);
 }
@@ -113,8 +116,8 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
 TIS_API int tis_paged_attention_simt(int dtype, const void* q, int q_stride, void* out, int out_stride,
                                      const void* plane, const int* block_table, int bt_stride, int num_pages,
                                      const int* positions, const int* row_slot, int n, int H, int KVH, int hd,
-                                     int page_size, int window, float scale, const float* sink, int* fault,
-                                     cudaStream_t stream) {
+                                     int page_size, int window, float scale, float softcap, const void* gate, int ldg,
+                                     const float* sink, int* fault, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (hd % 16 || hd <= 0 || hd > 256) {
         tis_set_error("paged_attention: head size %d is not a multiple of 16 in 16..256", hd);
@@ -133,6 +136,6 @@ TIS_API int tis_paged_attention_simt(int dtype, const void* q, int q_stride, voi
     TIS_DISPATCH_DTYPE(dtype, T,
         paged_attention_simt_kernel<T><<<grid, SIMT_KEYS, smem, stream>>>(
             (const T*)q, q_stride, (T*)out, out_stride, (const T*)plane, block_table, bt_stride, num_pages,
-            positions, row_slot, H, KVH, hd, page_size, window, scale, sink, fault));
+            positions, row_slot, H, KVH, hd, page_size, window, scale, softcap, (const T*)gate, ldg, sink, fault));
     return tis_check_launch("paged_attention_simt");
 }

@@ -59,6 +59,8 @@ struct TcAttnParams {
     const int* tile_row0; const int* tile_rows; int num_tiles;
     int H, KVH, page_size, window;
     float scale_log2;
+    SoftCap cap;            // bounds the raw scores (k 0: not)
+    const bf16* gate; int ldg;      // (n, H): head h's output times sigmoid(gate[row][h]) (null: none)
     const float* sink;      // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     int* fault;
 };
@@ -97,7 +99,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     if (slot < 0) return;                                 // padding only: the whole CTA leaves together
     const int pos0 = p.positions[row0];                   // the smallest position of the tile
     const int hi = p.positions[row0 + nrows - 1] + 1;     // keys [.., hi) are visible to the last row
-    const int lo_first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    const int lo_first = first_key(pos0, p.window);
     const int tile_begin = lo_first & ~(BN - 1);
     const int T = (hi - tile_begin + BN - 1) / BN;
 
@@ -219,8 +221,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int r = quarter * 32 + lane;
         const bool row_ok = r < nrows && p.row_slot[row0 + r] >= 0;
         const int qpos = row_ok ? p.positions[row0 + r] : 0;
-        const int lo_r = p.window > 0 ? max(0, qpos - p.window + 1) : 0;
-        const int lo_last = p.window > 0 ? max(0, hi - p.window) : 0;      // the last row's first key
+        const int lo_r = first_key(qpos, p.window);
+        const int lo_last = first_key(hi - 1, p.window);                   // the last row's first key
         const unsigned lane_bits = (unsigned)(quarter * 32) << 16;
         const unsigned col_s = COL_S + g * BN, col_o = COL_O + g * 128;
         unsigned char* pg_smem = p_smem + g * P_BYTES;
@@ -249,11 +251,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             // this group hands P over): first the maximum, then the exponentials.
             const bool whole = kt + BN - 1 <= pos0 && kt >= lo_last;      // every row of the tile sees every key
             const bool plain = whole && row_ok;
-            auto load64 = [&](int half, float (&s)[64]) {
+            auto load64 = [&](int half, float (&s)[64], bool bound) {
                 tmem_ld32_issue(tmem_base + lane_bits + col_s + half * 64, s);
                 tmem_ld32_issue(tmem_base + lane_bits + col_s + half * 64 + 32, s + 32);
                 tmem_ld_wait();
                 tmem_ld_arrived(s);
+                if (bound) {
+#pragma unroll
+                    for (int e = 0; e < 64; ++e) s[e] = soft_capped(s[e], p.cap);
+                }
                 if (!plain) {
 #pragma unroll
                     for (int e = 0; e < 64; ++e) {
@@ -267,11 +273,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll 1
             for (int half = 0; half < 2; ++half) {
                 float s[64];
-                load64(half, s);
+                load64(half, s, false);
 #pragma unroll
                 for (int e = 0; e < 64; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], s[e]);
             }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
+            // (the bound never falls: the maximum of the bounded scores is the bounded maximum)
+            const bool capped = p.cap.k != 0.f;
+            float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+            if (capped && mx > -INFINITY) mx = soft_capped(mx, p.cap);
+            mx *= p.scale_log2;
             // raise the reference maximum only when the row's maximum left it far behind
             const bool raise = mx > m_used + RESCALE_STEP || (m_used == -INFINITY && mx > -INFINITY);
             float alpha = 1.f;
@@ -300,7 +310,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 #pragma unroll 1
             for (int half = 0; half < 2; ++half) {
                 float s[64];
-                load64(half, s);
+                load64(half, s, capped);
 #pragma unroll
                 for (int c = 0; c < 8; ++c) {             // eight keys: one 16-byte chunk of the row of P
                     unsigned pk[4];
@@ -338,7 +348,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             const float w0 = m0 == -INFINITY ? 0.f : fast_exp2(m0 - m);
             const float w1 = (T < 2 || m1 == -INFINITY) ? 0.f : fast_exp2(m1 - m);
             const float l = l0 * w0 + l1 * w1 + (sink2 == -INFINITY ? 0.f : fast_exp2(sink2 - m));
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (p.gate != nullptr && r < nrows) inv /= 1.f + __expf(-__bfloat162float(p.gate[(size_t)(row0 + r) * p.ldg + head]));
             constexpr int COLS = HD / 2;                  // this group's share of the columns
 #pragma unroll 1
             for (int c = 0; c < COLS / 32; ++c) {
@@ -381,11 +392,13 @@ TIS_API int tis_attn_tc_supported() { return 1; }
 // Attention of `num_tiles` tiles of up to 128 consecutive rows of one request each.  q is
 // (n, >= H*hd) with row stride q_stride, out (n, H*hd); plane is [pages, 2, KVH, page_size, hd];
 // page_size 16, 32, 64 or 128.  `sink` (null: none): exp(sink[h]) is one more term of head h's softmax denominator.
+// `window`: first_key in common.cuh; `softcap` > 0 bounds the scores; `gate` (n, H; null: none) multiplies head h's output
+// by sigmoid(gate[row][h]).
 TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int out_stride, const void* plane,
                         const int* block_table, int bt_stride, int num_pages, const int* positions,
                         const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles, int H,
-                        int KVH, int page_size, int window, float scale, const float* sink, int* fault,
-                        cudaStream_t stream) {
+                        int KVH, int page_size, int window, float scale, float softcap, const void* gate, int ldg,
+                        const float* sink, int* fault, cudaStream_t stream) {
     if (num_tiles <= 0) return TIS_OK;
     if (page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) {
         tis_set_error("attn_tc: page size %d; this kernel takes 16, 32, 64 or 128", page_size);
@@ -414,6 +427,8 @@ TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int 
     p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.num_tiles = num_tiles;
     p.H = H; p.KVH = KVH; p.page_size = page_size; p.window = window;
     p.scale_log2 = scale * 1.4426950408889634f;
+    p.cap = soft_cap(softcap, scale);
+    p.gate = static_cast<const bf16*>(gate); p.ldg = ldg;
     p.sink = sink;
     p.fault = fault;
     tis_launch(attn_tc_kernel, dim3(num_tiles * H), dim3(NTH), (size_t)smem, stream, mq, mkv, p);
@@ -425,7 +440,7 @@ TIS_API int tis_attn_tc(const void* q, int q_stride, int n_rows, void* out, int 
 TIS_API int tis_attn_tc_supported() { return 0; }
 
 TIS_API int tis_attn_tc(const void*, int, int, void*, int, const void*, const int*, int, int, const int*, const int*,
-                        const int*, const int*, int, int, int, int, int, float, const float*, int*, cudaStream_t) {
+                        const int*, const int*, int, int, int, int, int, float, float, const void*, int, const float*, int*, cudaStream_t) {
     tis_set_error("attn_tc: built for a head size it does not take (64 and 128 only)");
     return TIS_BAD_SIZE;
 }

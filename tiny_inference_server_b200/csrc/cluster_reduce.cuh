@@ -18,14 +18,15 @@ namespace cluster_reduce {
 
 constexpr int STRIP = 64;             // columns of a strip
 constexpr int CONSUMERS = 128;        // threads that hold accumulators: four warps, 16 columns each
-// EPI_RELU2 .. EPI_SILU: a store through an activation (the square of relu; gelu in its tanh form; silu), applied to the
+// EPI_RELU2 .. EPI_TANH: a store through an activation (the square of relu; gelu in its tanh form; silu; tanh), applied to the
 // 32-bit sum
-enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_GELU_TANH = 4, EPI_SILU = 5 };
+enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_GELU_TANH = 4, EPI_SILU = 5, EPI_TANH = 6 };
 
 __device__ __forceinline__ float epilogue_act(float x, int epi) {
     if (epi == EPI_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
     if (epi == EPI_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     if (epi == EPI_SILU) return x / (1.f + expf(-x));
+    if (epi == EPI_TANH) return tanhf(x);
     return x;
 }
 

@@ -83,9 +83,9 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 // The factor a norm of the RMS family multiplies a row with, from the row's sum of squares s over a width d:
-// kind 0: sqrt(d) / (sqrt(s) + eps) (eps added to the L2 norm); kind 1: rsqrt(s / d + eps).  Both are
+// kind 0: sqrt(d) / (sqrt(s) + eps) (eps added to the L2 norm); kind 1: rsqrt(s / d + eps); kind 2: 1 (the row as it is).  All are
 // num / (sqrt(s * mul + add) + plus) with constants the host works out, so that a kernel has no case to tell apart.
-enum { TIS_NORM_L2_EPS = 0, TIS_NORM_MEAN_EPS = 1 };
+enum { TIS_NORM_L2_EPS = 0, TIS_NORM_MEAN_EPS = 1, TIS_NORM_NONE = 2 };
 struct NormFactor {
     float num, mul, add, plus;
     __device__ __forceinline__ float of(float sum_sq) const { return num / (sqrtf(fmaf(sum_sq, mul, add)) + plus); }
@@ -94,6 +94,7 @@ inline NormFactor norm_factor(int kind, int width, float eps) {
     NormFactor f;
     const float d = (float)(width > 0 ? width : 1);
     if (kind == TIS_NORM_MEAN_EPS) { f.num = 1.f; f.mul = 1.f / d; f.add = eps; f.plus = 0.f; }
+    else if (kind == TIS_NORM_NONE) { f.num = 1.f; f.mul = 0.f; f.add = 1.f; f.plus = 0.f; }
     else { f.num = sqrtf(d); f.mul = 1.f; f.add = 0.f; f.plus = eps; }
     return f;
 }
@@ -101,6 +102,30 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
+}
+
+// ---- which keys a row sees, and bounded scores ------------------------------------------------
+// `window` of the attention kernels: 0, every key up to the row's own; W > 0, the last W of them; -C < 0, those of the row's
+// own chunk of C positions (chunks are counted from position 0).  The first key never moves back from row to row.
+__device__ __forceinline__ int first_key(int pos, int window) {
+    if (window == 0) return 0;
+    return window > 0 ? max(0, pos - window + 1) : pos - pos % (-window);
+}
+// A score q . k * scale bounded smoothly, cap * tanh(score / cap).  The kernels bound the raw products, so that what
+// multiplies them with the scale afterwards stays as it is: raw -> c * tanh(raw * scale / cap) with c = cap / scale.
+// k = 2 log2(e) scale / cap; k 0: no bound.
+struct SoftCap { float k, c; };
+inline SoftCap soft_cap(float cap, float scale) {
+    SoftCap s;
+    s.k = cap > 0.f && scale != 0.f ? 2.f * 1.4426950408889634f * scale / cap : 0.f;
+    s.c = s.k != 0.f ? cap / scale : 0.f;
+    return s;
+}
+// tanh(x) = 1 - 2 / (1 + e^(2x)): one exponential and one division of the fast kinds, absolute error of the order of 1e-7 c
+__device__ __forceinline__ float soft_capped(float raw, const SoftCap& s) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(raw * s.k));
+    return fmaf(-2.f * s.c, __fdividef(1.f, 1.f + e), s.c);
 }
 
 // ---- gated units -----------------------------------------------------------------------------

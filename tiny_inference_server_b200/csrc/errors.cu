@@ -35,7 +35,7 @@ bool tis_pdl_enabled() {
 
 // Version of the launcher interface; the Python side refuses a library built from
 // other sources than its own.
-TIS_API int tis_abi_version() { return 12; }
+TIS_API int tis_abi_version() { return 13; }
 
 #ifdef TIS_TIMELINE
 static thread_local unsigned long long* g_timeline = nullptr;

@@ -34,6 +34,7 @@ using cluster_reduce::EPI_SWIGLU;
 using cluster_reduce::EPI_RESIDUAL;
 using cluster_reduce::EPI_RELU2;
 using cluster_reduce::EPI_SILU;
+using cluster_reduce::EPI_TANH;
 
 constexpr int BN = 64;            // columns of a strip
 constexpr int BK = 64;            // rows of K per tile
@@ -49,6 +50,11 @@ struct GemmParams {
     int kc;                       // rows of K per CTA of a cluster (a multiple of BK)
     int stages;                   // ring length: min(tiles per CTA, MAX_STAGES)
     cluster_reduce::Epilogue e;   // rows, columns, where the result goes
+    // several products in one launch (GROUPED kernels): `groups` equal ones of group_cols columns (a multiple of 64), product
+    // g of rows x + g * x_group and weights w + g * w_group, and behind them one of rows x + groups * x_group and weights
+    // `w_last` (N - groups * group_cols columns, row stride ld_last), whose sums pass the epilogue `last_epi`
+    int groups, group_cols; size_t x_group, w_group;
+    const bf16* w_last; int ld_last, last_epi;
     TIS_TIMELINE_MEMBER           // (instrumented builds only; stamps: 0 entry, 1 weights ordered, 2 dependency wait over,
                                   //  3 first tile ready, 4 loop done, 5 cluster barrier passed, 6 stored)
 };
@@ -98,8 +104,24 @@ __device__ __forceinline__ void load_x(bf16* xs, const GemmParams& p, int k0, in
     }
 }
 
-template <int MT, bool FORM>
-__global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams p) {
+// The parameters of the product that the strip of columns from n0 on belongs to (column numbers stay the whole launch's).
+__device__ __forceinline__ GemmParams product_of(const GemmParams& all, int n0) {
+    GemmParams p = all;
+    const int g = min(n0 / all.group_cols, all.groups);
+    p.x = all.x + (size_t)g * all.x_group;
+    if (g < all.groups) {
+        p.w = all.w + (size_t)g * all.w_group - (size_t)g * all.group_cols;
+    } else {
+        p.w = all.w_last - (size_t)g * all.group_cols;
+        p.ldw = all.ld_last;
+        p.e.epi = all.last_epi;
+    }
+    return p;
+}
+
+template <int MT, bool FORM, bool GROUPED = false>
+__global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams all) {
+    const GemmParams p = GROUPED ? product_of(all, (int)blockIdx.x * BN) : all;
     namespace cg = cooperative_groups;
     extern __shared__ __align__(16) unsigned char smem[];
     constexpr int W_ELEMS = BK * WROW, X_ELEMS = MT * 16 * XROW;
@@ -262,7 +284,7 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
         tis_set_error("gemm_skinny: ksplit %d must be 1, 2, 4 or 8", ksplit);
         return TIS_BAD_SIZE;
     }
-    if (epi < EPI_STORE || epi > EPI_SILU) {
+    if (epi < EPI_STORE || epi > EPI_TANH) {
         tis_set_error("gemm_skinny: unknown epilogue %d", epi);
         return TIS_BAD_SIZE;
     }
@@ -335,6 +357,67 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
         return TIS_CUDA_ERROR;
     }
     return tis_check_launch("gemm_skinny");
+}
+
+// Several products of few rows in one launch, their results side by side: out (M x N) = [x_0 W_0 | x_1 W_1 | .. | act(x_g W_last)].
+// x (M, groups + 1, K): row r of operand g at x + r * ldx + g * x_group; w (groups, K, group_cols) contiguous, group_cols a
+// multiple of 64; w_last (K, n_last), n_last a multiple of 8 (0: none), through the epilogue `last_epi` (EPI_STORE or an
+// activation).  bfloat16.
+TIS_API int tis_gemm_skinny_groups(const void* x, int ldx, size_t x_group, const void* w, int groups, int group_cols,
+                                   const void* w_last, int n_last, int last_epi, void* out, int ldo, int M, int K, int ksplit,
+                                   int* fault, cudaStream_t stream) {
+    if (M <= 0 || K <= 0) return TIS_OK;
+    if (M > 64 || K % 8 || ldx % 8 || x_group % 8 || groups <= 0 || group_cols <= 0 || group_cols % 64 || n_last < 0 || n_last % 8 ||
+        (n_last > 0 && w_last == nullptr) || (last_epi != EPI_STORE && (last_epi < EPI_RELU2 || last_epi > EPI_TANH)) ||
+        !(ksplit == 1 || ksplit == 2 || ksplit == 4 || ksplit == 8) ||
+        ((uintptr_t)x | (uintptr_t)w | (uintptr_t)w_last) % 16) {
+        tis_set_error("gemm_skinny_groups: %d rows of %d, %d groups of %d columns and %d more, epilogue %d, ksplit %d", M, K, groups,
+                      group_cols, n_last, last_epi, ksplit);
+        return TIS_BAD_SIZE;
+    }
+    const int N = groups * group_cols + n_last;
+    GemmParams p = {};
+    p.x = (const bf16*)x; p.ldx = ldx; p.w = (const bf16*)w; p.ldw = group_cols; p.K = K;
+    p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = EPI_STORE; p.e.fault = fault;
+    p.e.in_factor = norm_factor(0, 0, 0.f);
+    p.groups = groups; p.group_cols = group_cols; p.x_group = x_group; p.w_group = (size_t)K * group_cols;
+    p.w_last = (const bf16*)w_last; p.ld_last = n_last; p.last_epi = last_epi;
+    p.kc = ((K + ksplit - 1) / ksplit + BK - 1) / BK * BK;
+    const int mt = M <= 16 ? 1 : (M <= 32 ? 2 : 4);
+    const int tiles = p.kc / BK;
+    p.stages = tiles < MAX_STAGES ? tiles : MAX_STAGES;
+    const size_t smem = (size_t)p.stages * (BK * WROW + mt * 16 * XROW) * sizeof(bf16) +
+                        cluster_reduce::recv_floats(mt * 16, ksplit) * sizeof(float);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((N + BN - 1) / BN, ksplit, 1);
+    cfg.blockDim = dim3(NTH, 1, 1);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    cudaLaunchAttribute attrs[2];
+    attrs[0].id = cudaLaunchAttributeClusterDimension;
+    attrs[0].val.clusterDim.x = 1;
+    attrs[0].val.clusterDim.y = ksplit;
+    attrs[0].val.clusterDim.z = 1;
+    attrs[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attrs[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attrs;
+    cfg.numAttrs = tis_pdl_enabled() ? 2 : 1;
+    static bool configured = false;
+    if (!configured) {
+        cudaFuncSetAttribute(gemm_skinny_kernel<1, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<2, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        cudaFuncSetAttribute(gemm_skinny_kernel<4, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024);
+        configured = true;
+    }
+    cudaError_t e;
+    if (mt == 1) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<1, false, true>, p);
+    else if (mt == 2) e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<2, false, true>, p);
+    else e = cudaLaunchKernelEx(&cfg, gemm_skinny_kernel<4, false, true>, p);
+    if (e != cudaSuccess) {
+        tis_set_error("gemm_skinny_groups: %s", cudaGetErrorString(e));
+        return TIS_CUDA_ERROR;
+    }
+    return tis_check_launch("gemm_skinny_groups");
 }
 
 TIS_API int tis_gemm_skinny(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int N, int K,

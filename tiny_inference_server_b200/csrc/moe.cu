@@ -202,7 +202,8 @@ __device__ __forceinline__ float unit_act(float x, int kind) {
 template <typename T>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ chosen, const T* __restrict__ w_gu,
-                   T* __restrict__ hidden, int d, int top, int E, int F, int act, GateForm gate) {
+                   T* __restrict__ hidden, int d, int top, int E, int F, int act, GateForm gate,
+                   const float* __restrict__ in_weights) {
     extern __shared__ __align__(16) float smem[];
     pdl_launch_dependents();
     const int pair = blockIdx.x, r = pair / top;
@@ -215,6 +216,8 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
     __syncthreads();
     const T* wg = w_gu + (size_t)e * (act >= 0 ? 1 : 2) * F * d;
     const T* wu = wg + (size_t)F * d;
+    // a weight on the unit's input multiplies both projections of it
+    const float iw = in_weights != nullptr ? in_weights[pair] : 1.f;
     const int j_end = min(F, (int)(blockIdx.y + 1) * MOE_COLS);
     if (act >= 0) {                                        // no gate: two columns are two dot products
         for (int j = blockIdx.y * MOE_COLS + 2 * warp; j < j_end; j += 2 * nw) {
@@ -224,8 +227,8 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
             float r[2];
             warp_dots<T, 2>(w, x2, d, lane, vec, r);
             if (lane == 0) {
-                hidden[(size_t)pair * F + j] = from_f32<T>(unit_act(r[0], act));
-                if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(unit_act(r[1], act));
+                hidden[(size_t)pair * F + j] = from_f32<T>(unit_act(r[0] * iw, act));
+                if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(unit_act(r[1] * iw, act));
             }
         }
         return;
@@ -238,14 +241,14 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
         float r[4];
         warp_dots<T, 4>(w, x4, d, lane, vec, r);
         if (lane == 0) {
-            hidden[(size_t)pair * F + j] = from_f32<T>(gated_unit(r[0], r[1], gate));
-            if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(gated_unit(r[2], r[3], gate));
+            hidden[(size_t)pair * F + j] = from_f32<T>(gated_unit(r[0] * iw, r[1] * iw, gate));
+            if (j1 != j) hidden[(size_t)pair * F + j1] = from_f32<T>(gated_unit(r[2] * iw, r[3] * iw, gate));
         }
     }
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// out[r][c] = sum_k weights[r][k] * (Wd[e_k][c] . hidden[r * top + k])  (+ shared_gate[r] * shared[r][c]);
+// out[r][c] = sum_k weights[r][k] * (Wd[e_k][c] . hidden[r * top + k])  (+ shared_gate[r] * shared[r][c]);  weights null: 1;
 // w_down (E, d, F).  A CTA per (row, block of COLS output columns).
 // ------------------------------------------------------------------------------------------------------------
 template <typename T>
@@ -274,7 +277,7 @@ moe_down_kernel(const T* __restrict__ hidden, const int* __restrict__ chosen, co
             for (int j = 0; j < 4; ++j) {
                 const int k = min(k0 + j, top - 1);
                 int e = chosen[(size_t)r * top + k];
-                wt[j] = (k0 + j < top && e >= 0 && e < E) ? weights[(size_t)r * top + k] : 0.f;
+                wt[j] = (k0 + j < top && e >= 0 && e < E) ? (weights != nullptr ? weights[(size_t)r * top + k] : 1.f) : 0.f;
                 e = min(max(e, 0), E - 1);
                 w[j] = w_down + ((size_t)e * d + c) * F;
                 x4[j] = smem + (size_t)k * F;
@@ -323,8 +326,9 @@ TIS_API int tis_moe_route(int dtype, const void* x, int ldx, const float* wr, co
     return tis_check_launch("moe_route");
 }
 
+// `in_weights` (n * top; null: 1): multiplies the input of every (row, choice)'s unit.
 TIS_API int tis_moe_gate_up(int dtype, const void* x, int ldx, const int* chosen, const void* w_gu, void* hidden, int n,
-                            int d, int top, int E, int F, int act, GateForm gate, cudaStream_t stream) {
+                            int d, int top, int E, int F, int act, GateForm gate, const float* in_weights, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || top <= 0 || E <= 0 || F <= 0) {
         tis_set_error("moe_gate_up: width %d, top %d, %d experts of %d hidden", d, top, E, F);
@@ -335,7 +339,7 @@ TIS_API int tis_moe_gate_up(int dtype, const void* x, int ldx, const int* chosen
         const int st = set_smem(moe_gate_up_kernel<T>, smem, "moe_gate_up");
         if (st != TIS_OK) return st;
         tis_launch(moe_gate_up_kernel<T>, dim3(n * top, (F + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
-                   (const T*)x, ldx, chosen, (const T*)w_gu, (T*)hidden, d, top, E, F, act, gate);
+                   (const T*)x, ldx, chosen, (const T*)w_gu, (T*)hidden, d, top, E, F, act, gate, in_weights);
     });
     return tis_check_launch("moe_gate_up");
 }
@@ -433,7 +437,7 @@ template <bool GATED, bool GATHER>
 __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ sorted_pair, int top,
                    const int* __restrict__ tile_expert, const bf16* __restrict__ W, size_t expert_stride,
-                   bf16* __restrict__ C, int ldc, int N, int K, int act, GateForm gate) {
+                   bf16* __restrict__ C, int ldc, int N, int K, int act, GateForm gate, const float* __restrict__ in_weights) {
     constexpr int BROWS = GATED ? 2 * GT_COLS : GT_COLS;
     __shared__ __align__(16) bf16 As[GT_STAGES][GT_ROWS][GT_LD];
     __shared__ __align__(16) bf16 Bs[GT_STAGES][BROWS][GT_LD];
@@ -520,13 +524,15 @@ moe_grouped_kernel(const bf16* __restrict__ A, int lda, const int* __restrict__ 
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const size_t row = (size_t)tile * GT_ROWS + wm * 32 + mi * 16 + g + 8 * half;
+            float iw = 1.f;                                // a weight on the unit's input
+            if (GATHER && in_weights != nullptr) { const int pr = sorted_pair[row]; iw = pr >= 0 ? in_weights[pr] : 0.f; }
 #pragma unroll
             for (int n = 0; n < 4; ++n) {
                 const int col = n0 + wn * 32 + n * 8 + 2 * t4;
-                float v0 = acc[0][mi][n][2 * half], v1 = acc[0][mi][n][2 * half + 1];
+                float v0 = acc[0][mi][n][2 * half] * iw, v1 = acc[0][mi][n][2 * half + 1] * iw;
                 if (GATED) {
-                    v0 = gated_unit_fast(v0, acc[GATED ? 1 : 0][mi][n][2 * half], gate);
-                    v1 = gated_unit_fast(v1, acc[GATED ? 1 : 0][mi][n][2 * half + 1], gate);
+                    v0 = gated_unit_fast(v0, acc[GATED ? 1 : 0][mi][n][2 * half] * iw, gate);
+                    v1 = gated_unit_fast(v1, acc[GATED ? 1 : 0][mi][n][2 * half + 1] * iw, gate);
                 } else if (act >= 0) {
                     v0 = unit_act(v0, act);
                     v1 = unit_act(v1, act);
@@ -552,7 +558,7 @@ moe_combine_kernel(const bf16* __restrict__ y, int ldy, const int* __restrict__ 
         for (int k = 0; k < top; ++k) {
             const int place = pair_place[(size_t)r * top + k];
             if (place < 0) continue;
-            const float w = weights[(size_t)r * top + k];
+            const float w = weights != nullptr ? weights[(size_t)r * top + k] : 1.f;
             const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(y + (size_t)place * ldy + c);
             a0 = fmaf(w, __bfloat162float(v.x), a0);
             a1 = fmaf(w, __bfloat162float(v.y), a1);
@@ -588,13 +594,16 @@ TIS_API int tis_moe_grouped_tiles(int pairs, int E) { return (pairs + GT_ROWS - 
 
 // The experts' products for many rows in bfloat16.  x (n, d) with row stride ldx; w_gu (E, 2, F, d), or (E, F, d) with
 // act >= 0 (units without a gate); w_down (E, d, F);
+// weigh_input: a choice's weight multiplies its unit's input instead of its output;
 // scratch: sorted_pair and hidden / y rows for tis_moe_grouped_tiles(n * top, E) * 64 places, pair_place n * top,
 // tile_expert that many tiles.  d and F multiples of 32; ldx, lds multiples of 8 and even; operands 16-byte aligned.
 TIS_API int tis_moe_grouped(const void* x, int ldx, const int* chosen, const float* weights, const void* w_gu,
                             const void* w_down, const void* shared, int lds, const float* shared_gate, void* out,
                             int* sorted_pair, int* pair_place, int* tile_expert, void* hidden, void* y, int n, int d,
-                            int top, int E, int F, int act, GateForm gate, cudaStream_t stream) {
+                            int top, int E, int F, int act, GateForm gate, int weigh_input, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
+    const float* in_weights = weigh_input ? weights : nullptr;
+    if (weigh_input) weights = nullptr;
     if (d <= 0 || F <= 0 || d % GT_BK || F % GT_BK || ldx % 8 || lds % 2 || E <= 0 || E > 4096 || top <= 0 ||
         ((uintptr_t)x | (uintptr_t)w_gu | (uintptr_t)w_down | (uintptr_t)hidden | (uintptr_t)y) % 16 ||
         ((uintptr_t)shared | (uintptr_t)out) % 4) {
@@ -608,16 +617,16 @@ TIS_API int tis_moe_grouped(const void* x, int ldx, const int* chosen, const flo
     if (act >= 0)
         tis_launch(moe_grouped_kernel<false, true>, dim3(tiles, (F + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                    (const bf16*)x, ldx, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_gu, (size_t)F * d,
-                   (bf16*)hidden, F, F, d, act, gate);
+                   (bf16*)hidden, F, F, d, act, gate, in_weights);
     else
         tis_launch(moe_grouped_kernel<true, true>, dim3(tiles, (F + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                    (const bf16*)x, ldx, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_gu,
-                   (size_t)2 * F * d, (bf16*)hidden, F, F, d, -1, gate);
+                   (size_t)2 * F * d, (bf16*)hidden, F, F, d, -1, gate, in_weights);
     st = tis_check_launch("moe_grouped_gate_up");
     if (st != TIS_OK) return st;
     tis_launch(moe_grouped_kernel<false, false>, dim3(tiles, (d + GT_COLS - 1) / GT_COLS), dim3(128), 0, stream,
                (const bf16*)hidden, F, (const int*)sorted_pair, top, (const int*)tile_expert, (const bf16*)w_down, (size_t)d * F,
-               (bf16*)y, d, d, F, -1, gate);
+               (bf16*)y, d, d, F, -1, gate, (const float*)nullptr);
     st = tis_check_launch("moe_grouped_down");
     if (st != TIS_OK) return st;
     return tis_moe_combine_launch(y, d, pair_place, weights, shared, lds, shared_gate, out, n, d, top, stream);

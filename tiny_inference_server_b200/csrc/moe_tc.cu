@@ -29,6 +29,7 @@ struct MoeTcParams {
     int up_offset;          // gated: the expert's up rows start this many rows after its gate rows
     int tiles_m, tiles_n;
     const int* tile_expert;
+    const float* in_weights; const int* sorted_pair;    // a weight on the input of every sorted row's unit (null: none)
     int* fault;
     GateForm gate;          // gated: the form of the gating
     int act;                // not gated: -1 none, else the activation of the output (0 relu^2, 1 gelu (tanh), 2 silu)
@@ -137,6 +138,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             if (!mbar_wait(&acc_full[b], (acc_it >> 1) & 1, abort, p.fault, 7)) break;
             fence_after();
             const size_t row = (size_t)m0 + quarter * 32 + lane;
+            float iw = 1.f;
+            if (p.in_weights != nullptr) { const int pr = p.sorted_pair[row]; iw = pr >= 0 ? p.in_weights[pr] : 0.f; }
             const unsigned taddr = tmem_base + ((unsigned)(quarter * 32) << 16) + b * BN;
 #pragma unroll 1
             for (int c = 0; c < BH / 32; ++c) {
@@ -146,10 +149,10 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
                     float u[32];
                     tmem_ld32(taddr + BH + c * 32, u);
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) g[i] = gated_unit_fast(g[i], u[i], p.gate);
+                    for (int i = 0; i < 32; ++i) g[i] = gated_unit_fast(g[i] * iw, u[i] * iw, p.gate);
                 } else if (p.act >= 0) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) g[i] = tile_act(g[i], p.act);
+                    for (int i = 0; i < 32; ++i) g[i] = tile_act(g[i] * iw, p.act);
                 }
                 bf16* o = p.out + row * p.ldo + n0 + c * 32;
 #pragma unroll
@@ -218,11 +221,12 @@ TIS_API int tis_moe_tc_tiles(int pairs, int E) { return (pairs + BM - 1) / BM + 
 
 // The experts' products for many rows in bfloat16 on the tcgen05 tensor cores.  x (n, d) with row stride ldx; w_gu
 // (E, 2, F, d), or (E, F, d) with act >= 0 (units without a gate, the activation on the first product); w_down (E, d, F); scratch for T = tis_moe_tc_tiles(n * top, E) tiles: sorted_pair T * 128, pair_place
-// n * top, tile_expert T, xs (T * 128, d), hidden (T * 128, F), y (T * 128, d).  d and F multiples of 64.
+// n * top, tile_expert T; weigh_input: a choice's weight multiplies its unit's input instead of its output; xs (T * 128, d), hidden (T * 128, F), y (T * 128, d).  d and F multiples of 64.
 TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const float* weights, const void* w_gu,
                                const void* w_down, const void* shared, int lds, const float* shared_gate, void* out,
                                int* sorted_pair, int* pair_place, int* tile_expert, void* xs, void* hidden, void* y, int n,
-                               int d, int top, int E, int F, int act, GateForm gate, int* fault, cudaStream_t stream) {
+                               int d, int top, int E, int F, int act, GateForm gate, int weigh_input, int* fault,
+                               cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (d <= 0 || F <= 0 || d % BK || F % BK || ldx % 8 || lds % 2 || E <= 0 || E > 4096 || top <= 0 ||
         ((uintptr_t)x | (uintptr_t)w_gu | (uintptr_t)w_down | (uintptr_t)xs | (uintptr_t)hidden | (uintptr_t)y) % 16 ||
@@ -241,6 +245,8 @@ TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const 
     CUtensorMap ma, mb;
     MoeTcParams p;
     p.fault = fault;
+    p.in_weights = weigh_input ? weights : nullptr;
+    p.sorted_pair = sorted_pair;
     p.gate = gate;
     p.tile_expert = tile_expert;
     p.tiles_m = tiles_m;
@@ -271,7 +277,7 @@ TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const 
     }
     if (st != TIS_OK) return st;
     // down: K = F, the stacked matrix has E * d rows of F elements
-    p.out = static_cast<bf16*>(y); p.ldo = d; p.N = d; p.K = F; p.rows_per_expert = d; p.up_offset = 0; p.act = -1;
+    p.out = static_cast<bf16*>(y); p.ldo = d; p.N = d; p.K = F; p.rows_per_expert = d; p.up_offset = 0; p.act = -1; p.in_weights = nullptr;
     if (d >= 256) {
         if (!tensor_map(hidden, F, rows, F, BM, true, &ma) || !tensor_map(w_down, F, (long long)E * d, F, 256, true, &mb))
             return TIS_CUDA_ERROR;
@@ -282,5 +288,5 @@ TIS_API int tis_moe_grouped_tc(const void* x, int ldx, const int* chosen, const 
         st = launch<128, 6, false>(ma, mb, p, stream);
     }
     if (st != TIS_OK) return st;
-    return tis_moe_combine_launch(y, d, pair_place, weights, shared, lds, shared_gate, out, n, d, top, stream);
+    return tis_moe_combine_launch(y, d, pair_place, weigh_input ? nullptr : weights, shared, lds, shared_gate, out, n, d, top, stream);
 }

@@ -175,6 +175,140 @@ rotate_norm_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__
     }
 }
 
+// The other order: queries and keys are normed first, each over all of its heads at once and with weights `w` (H * dim for the
+// queries, then G * dim for the keys), and then rotated, neighbouring elements paired.  Whole 16-byte vectors, a CTA a row,
+// VPT vectors of the row a thread.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256)
+norm_rotate_vec_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__ v_pages, const float* __restrict__ w,
+                       const RotateNorm p) {
+    constexpr int N = Vec16<T>::N;
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    const int r = blockIdx.x, tid = threadIdx.x;
+    const int slot = p.row_slot[r];
+    if (slot < 0) return;
+    const int pos = p.positions[r];
+    const int page = p.G > 0 ? page_of(p, slot, pos, tid == 0) : -1;
+    const int in_page = pos % p.page_size;
+    const float* ct = p.cos_t + (size_t)pos * (p.rot >> 1);
+    const float* st = p.sin_t + (size_t)pos * (p.rot >> 1);
+    const int nq = p.H * p.dim, nk = p.G * p.dim, nv = (nq + nk) / N;
+    pdl_wait();
+    T* row = qkv + (size_t)r * p.ld;
+    float v[VPT][N];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int e = (tid + k * 256) * N;
+        if (e < nv * N) {
+            Vec16<T>::load(row + e, v[k]);
+            float s = 0.f;
+#pragma unroll
+            for (int j = 0; j < N; ++j) s = fmaf(v[k][j], v[k][j], s);
+            if (e < nq) sq += s; else sk += s;
+        }
+    }
+    const float fq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + p.eps);
+    const float fk = nk > 0 ? 1.f / sqrtf(block_sum(sk, red) / (float)nk + p.eps) : 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int e = (tid + k * 256) * N;
+        if (e >= nv * N || (e >= nq && page < 0)) continue;
+        const float f = e < nq ? fq : fk;
+        const int hh = e / p.dim, i = e - hh * p.dim;
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[k][j] *= f * w[e + j];
+#pragma unroll
+        for (int j = 0; j < N / 2; ++j)
+            if (i + 2 * j < p.rot) {
+                const float c = ct[(i >> 1) + j], s = st[(i >> 1) + j];
+                const float a = v[k][2 * j], b = v[k][2 * j + 1];
+                v[k][2 * j] = a * c - b * s;
+                v[k][2 * j + 1] = b * c + a * s;
+            }
+        if (e < nq) Vec16<T>::store(row + e, v[k]);
+        else
+            Vec16<T>::store(k_pages + (size_t)page * p.k_page_stride + (size_t)(hh - p.H) * p.k_head_stride + (size_t)in_page * p.dim +
+                            (p.permuted ? cache_chunk(i / N, pos, p.dim / N) * N : i), v[k]);
+    }
+    if (page < 0) return;
+    const T* vals = row + nq + nk;
+    const int nch = p.v_dim / N;
+    for (int idx = tid; idx < p.G * nch; idx += 256) {
+        const int g = idx / nch, c = idx - g * nch;
+        *reinterpret_cast<uint4*>(v_pages + (size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim +
+                                  (p.permuted ? cache_chunk(c, pos, nch) : c) * N) = *reinterpret_cast<const uint4*>(vals + idx * N);
+    }
+}
+
+// The same for any size and pairing.  A thread owns whole rotation pairs, so that queries can be replaced in place.
+template <typename T>
+__global__ void __launch_bounds__(256)
+norm_rotate_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__ v_pages, const float* __restrict__ w,
+                   const RotateNorm p) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    const int r = blockIdx.x, tid = threadIdx.x;
+    const int slot = p.row_slot[r];
+    if (slot < 0) return;
+    const int pos = p.positions[r];
+    const int page = p.G > 0 ? page_of(p, slot, pos, tid == 0) : -1;
+    const int in_page = pos % p.page_size;
+    const int half = p.rot >> 1;
+    const float* ct = p.cos_t + (size_t)pos * half;
+    const float* st = p.sin_t + (size_t)pos * half;
+    const int nq = p.H * p.dim, nk = p.G * p.dim;
+    pdl_wait();
+    T* row = qkv + (size_t)r * p.ld;
+    constexpr int N = Vec16<T>::N;
+    auto place = [&](int i, int width, bool permuted) {
+        return permuted ? cache_chunk(i / N, pos, width / N) * N + i % N : i;
+    };
+    float sq = 0.f, sk = 0.f;
+    for (int e = tid; e < nq + nk; e += blockDim.x) {
+        const float x = to_f32(row[e]);
+        if (e < nq) sq = fmaf(x, x, sq); else sk = fmaf(x, x, sk);
+    }
+    const float fq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + p.eps);
+    const float fk = nk > 0 ? 1.f / sqrtf(block_sum(sk, red) / (float)nk + p.eps) : 0.f;
+    const int heads = p.H + (page >= 0 ? p.G : 0);
+    const int units = half + (p.dim - p.rot);                 // rotation pairs and single elements of a head
+    for (int idx = tid; idx < heads * units; idx += blockDim.x) {
+        const int hh = idx / units, u = idx - hh * units;
+        T* src = row + (size_t)hh * p.dim;
+        const float* wh = w + (size_t)hh * p.dim;
+        const bool perm = p.permuted && hh >= p.H;
+        const float f = hh < p.H ? fq : fk;
+        T* dst = hh < p.H ? src : k_pages + (size_t)page * p.k_page_stride + (size_t)(hh - p.H) * p.k_head_stride + (size_t)in_page * p.dim;
+        if (u < half) {
+            const int ia = p.interleaved ? 2 * u : u, ib = p.interleaved ? 2 * u + 1 : u + half;
+            const float a = to_f32(src[ia]) * f * wh[ia], b = to_f32(src[ib]) * f * wh[ib];
+            dst[place(ia, p.dim, perm)] = from_f32<T>(a * ct[u] - b * st[u]);
+            dst[place(ib, p.dim, perm)] = from_f32<T>(b * ct[u] + a * st[u]);
+        } else {
+            const int i = p.rot + u - half;
+            dst[place(i, p.dim, perm)] = from_f32<T>(to_f32(src[i]) * f * wh[i]);
+        }
+    }
+    if (page < 0) return;
+    const T* vals = row + nq + nk;
+    for (int idx = tid; idx < p.G * p.v_dim; idx += blockDim.x) {
+        const int g = idx / p.v_dim, e = idx - g * p.v_dim;
+        v_pages[(size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim + place(e, p.v_dim, p.permuted)] = vals[idx];
+    }
+}
+
+template <typename T>
+void launch_norm_rotate(T* qkv, T* k_pages, T* v_pages, const float* w, const RotateNorm& p, bool vec, cudaStream_t stream) {
+    const int per = ((p.H + p.G) * p.dim / Vec16<T>::N + 255) / 256;
+    if (!vec || per > 8) tis_launch(norm_rotate_kernel<T>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    else if (per <= 1) tis_launch(norm_rotate_vec_kernel<T, 1>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    else if (per <= 2) tis_launch(norm_rotate_vec_kernel<T, 2>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    else if (per <= 4) tis_launch(norm_rotate_vec_kernel<T, 4>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    else tis_launch(norm_rotate_vec_kernel<T, 8>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+}
+
 template <typename T, int LPH, int VPL>
 void launch_vec(T* qkv, T* k_pages, T* v_pages, const RotateNorm& p, cudaStream_t stream) {
     const size_t threads = (size_t)p.n * (p.H + 2 * p.G) * LPH;
@@ -197,8 +331,11 @@ void launch_any(T* qkv, T* k_pages, T* v_pages, const RotateNorm& p, bool vec, c
 
 }  // namespace
 
+// `whole_w` (null: none; else (H + G) * dim weights): the norm comes before the rotation and runs over all query heads, and over
+// all key heads, at once (`norm` is then not looked at).
 TIS_API int tis_rotate_norm_store(int dtype, void* qkv, int ld, int H, int G, int dim, int v_dim, int rot, int interleaved,
-                                  int permuted, const float* cos_t, const float* sin_t, int norm, float eps, void* k_pages,
+                                  int permuted, const float* cos_t, const float* sin_t, int norm, float eps,
+                                  const float* whole_w, void* k_pages,
                                   size_t k_page_stride, size_t k_head_stride, void* v_pages, size_t v_page_stride,
                                   size_t v_head_stride, int page_size, int num_pages, const int* block_table, int bt_stride,
                                   const int* positions, const int* row_slot, int* fault, int n, cudaStream_t stream) {
@@ -223,6 +360,10 @@ TIS_API int tis_rotate_norm_store(int dtype, void* qkv, int ld, int H, int G, in
     const bool vec = (interleaved || rot == 0) && dim % N == 0 && ld % N == 0 && (uintptr_t)qkv % 16 == 0 &&
                      (G == 0 || (v_dim % N == 0 && ((k_page_stride | k_head_stride | v_page_stride | v_head_stride) % N) == 0 &&
                                  ((uintptr_t)k_pages | (uintptr_t)v_pages) % 16 == 0));
+    if (whole_w != nullptr) {
+        TIS_DISPATCH_DTYPE(dtype, T, launch_norm_rotate<T>((T*)qkv, (T*)k_pages, (T*)v_pages, whole_w, p, vec, stream));
+        return tis_check_launch("norm_rotate_store");
+    }
     TIS_DISPATCH_DTYPE(dtype, T, launch_any<T>((T*)qkv, (T*)k_pages, (T*)v_pages, p, vec, stream));
     return tis_check_launch("rotate_norm_store");
 }

@@ -42,7 +42,7 @@ TIS_API int tis_embed_rows(int dtype, const void* table, const int* tokens, floa
 // ----------------------------------------------------------------------------------
 // residual += delta ; out = residual * factor(sum of squares) * scale, with the factor of the norm's kind:
 // sqrt(d) / (||residual||_2 + eps) (eps added to the L2 norm itself: main_models_new.py:38-42 of the upstream
-// project) or 1 / sqrt(mean of squares + eps)
+// project), 1 / sqrt(mean of squares + eps), or 1
 // ----------------------------------------------------------------------------------
 template <typename T>
 __global__ void add_rmsnorm_kernel(float* __restrict__ res, const T* __restrict__ delta,
@@ -225,7 +225,7 @@ TIS_API int tis_add_rmsnorm(int dtype, float* residual, const void* delta, const
                             int kind, void* out, int n, int d, const float* delta_weight, float delta_eps,
                             int delta_kind, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
-    if (kind < TIS_NORM_L2_EPS || kind > TIS_NORM_MEAN_EPS || delta_kind < TIS_NORM_L2_EPS || delta_kind > TIS_NORM_MEAN_EPS) {
+    if (kind < TIS_NORM_L2_EPS || kind > TIS_NORM_NONE || delta_kind < TIS_NORM_L2_EPS || delta_kind > TIS_NORM_NONE) {
         tis_set_error("add_rmsnorm: norm kinds %d, %d", kind, delta_kind);
         return TIS_BAD_SIZE;
     }
@@ -706,9 +706,10 @@ TIS_API int tis_softcap_f32(float* x, float cap, size_t total, cudaStream_t stre
 // out = act(x) element by element over (n, F), rows of x and out with strides of their own.
 // kind 0: relu(x)^2; 1: gelu in its tanh form, 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))); 2: silu.
 // ----------------------------------------------------------------------------------
-enum { TIS_ACT_RELU2 = 0, TIS_ACT_GELU_TANH = 1, TIS_ACT_SILU = 2 };
+enum { TIS_ACT_RELU2 = 0, TIS_ACT_GELU_TANH = 1, TIS_ACT_SILU = 2, TIS_ACT_TANH = 3 };
 
 __device__ __forceinline__ float activation_f(float x, int kind) {
+    if (kind == TIS_ACT_TANH) return tanhf(x);
     if (kind == TIS_ACT_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
     if (kind == TIS_ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     return x / (1.f + expf(-x));
@@ -749,7 +750,7 @@ activation_vec_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int
 TIS_API int tis_activation(int dtype, const void* x, int ldx, void* out, int ldo, int n, int F, int kind,
                            cudaStream_t stream) {
     if (n <= 0 || F <= 0) return TIS_OK;
-    if (kind < TIS_ACT_RELU2 || kind > TIS_ACT_SILU || ldx < F || ldo < F) {
+    if (kind < TIS_ACT_RELU2 || kind > TIS_ACT_TANH || ldx < F || ldo < F) {
         tis_set_error("activation: kind %d, %d columns, row lengths %d in and %d out", kind, F, ldx, ldo);
         return TIS_BAD_SIZE;
     }

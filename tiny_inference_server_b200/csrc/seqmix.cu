@@ -622,8 +622,8 @@ TIS_API int tis_diff_combine(int dtype, const void* a, int lda, float lambda, fl
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// Attention of one row and query head over the keys lo..pos of its request's pages, lo = max(0, pos - window + 1)
-// (window 0: lo = 0):  score_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * (pos - j)), softmax, times values,
+// Attention of one row and query head over the keys lo..pos of its request's pages, lo = first_key(pos, window)
+// (common.cuh; softcap > 0 bounds q . k_j * scale by softcap * tanh(. / softcap)):  score_j = q . k_j * scale - r1[head] * ln(1 + r2[head] * (pos - j)), softmax, times values,
 // times sigmoid(gate) element by element (gate_per_head: `gate` holds one number per head, for all its elements).
 // r1 null: no bias; gate null: no gate.
 // A CTA of 128 threads: 128 keys a tile, a thread a key for the scores; for the values the threads form
@@ -639,7 +639,7 @@ window_attention_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ 
                         const T* __restrict__ v_pages, size_t v_page_stride, size_t v_head_stride,
                         const int* __restrict__ block_table, int bt_stride, int num_pages,
                         const int* __restrict__ positions, const int* __restrict__ row_slot, int H, int G, int k_dim,
-                        int v_dim, int page_size, int window, float scale, const float* __restrict__ r1,
+                        int v_dim, int page_size, int window, float scale, float softcap, const float* __restrict__ r1,
                         const float* __restrict__ r2, const float* __restrict__ sink, int v_row, int gate_per_head,
                         int* __restrict__ fault) {
     extern __shared__ float smem[];
@@ -658,7 +658,7 @@ window_attention_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ 
     const int tid = threadIdx.x;
     pdl_wait();
     for (int i = tid; i < k_dim; i += WA_THREADS) qs[i] = to_f32(q[(size_t)r * ldq + (size_t)head * k_dim + i]);
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_key(pos, window);
     const int hi = pos + 1;
     // value columns
     const int groups = v_dim >= WA_THREADS ? 1 : WA_THREADS / v_dim;
@@ -685,7 +685,9 @@ window_attention_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ 
                               (size_t)(j % page_size) * k_dim;
                 float d = 0.f;
                 for (int i = 0; i < k_dim; ++i) d = fmaf(qs[i], to_f32(kr[i]), d);
-                s = d * scale - b1 * logf(1.f + b2 * (float)(pos - j));
+                d *= scale;
+                if (softcap > 0.f) d = softcap * tanhf(d / softcap);
+                s = d - b1 * logf(1.f + b2 * (float)(pos - j));
             }
         }
         page_of[tid] = page;
@@ -746,12 +748,12 @@ TIS_API int tis_window_attention(int dtype, const void* q, int ldq, const void* 
                                  const void* k_pages, size_t k_page_stride, size_t k_head_stride, const void* v_pages,
                                  size_t v_page_stride, size_t v_head_stride, const int* block_table, int bt_stride,
                                  int num_pages, const int* positions, const int* row_slot, int n, int H, int G,
-                                 int k_dim, int v_dim, int page_size, int window, float scale, const float* r1,
-                                 const float* r2, const float* sink, int v_row, int gate_per_head, int* fault,
-                                 cudaStream_t stream) {
+                                 int k_dim, int v_dim, int page_size, int window, float scale, float softcap,
+                                 const float* r1, const float* r2, const float* sink, int v_row, int gate_per_head,
+                                 int* fault, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
     if (H <= 0 || G <= 0 || H % G || k_dim <= 0 || v_dim <= 0 || v_dim > WA_THREADS * WA_MAX_COLS || page_size <= 0 ||
-        window < 0 || v_row < v_dim) {
+        v_row < v_dim) {
         tis_set_error("window_attention: %d query heads, %d kv heads, key width %d, value width %d (at most %d), "
                       "page size %d, window %d", H, G, k_dim, v_dim, WA_THREADS * WA_MAX_COLS, page_size, window);
         return TIS_BAD_SIZE;
@@ -762,7 +764,7 @@ TIS_API int tis_window_attention(int dtype, const void* q, int ldq, const void* 
         tis_launch(window_attention_kernel<T>, dim3(n, H), dim3(WA_THREADS), smem, stream, (const T*)q, ldq,
                    (const T*)gate, ldg, (T*)out, ldo, (const T*)k_pages, k_page_stride, k_head_stride, (const T*)v_pages,
                    v_page_stride, v_head_stride, block_table, bt_stride, num_pages, positions, row_slot, H, G, k_dim,
-                   v_dim, page_size, window, scale, r1, r2, sink, v_row, gate_per_head, fault));
+                   v_dim, page_size, window, scale, softcap, r1, r2, sink, v_row, gate_per_head, fault));
     return tis_check_launch("window_attention");
 }
 
@@ -799,8 +801,12 @@ __device__ __forceinline__ float gate_f(float x, int act) { const float s = 1.f 
 // or (DECAY_STEP) a step size per head and token: with `a_in` (n, H) its projection and `dt_bias` (H) its bias,
 // dt = softplus(a + bias), S <- exp(-exp(A_log[head]) * dt) S + k (dt v)^T, o = S^T q: a selective state space in its
 // recurrent form (k is the input matrix B, q the output matrix C, v the head's inputs); the outputs leave unnormalised
+// or (DECAY_BONUS) a decay per head and key channel with a bonus for the current token: with `a_in` the decay's projection,
+// `dt_bias` its bias and `A_log` the bonus u per head and key channel, g = exp(-exp(a + bias)), o = (S + diag(u) k v^T)^T q,
+// then S <- diag(g) S + k v^T: the outputs read the state before the token.  The bonus' share of o is (sum_i u_i q_i k_i) v,
+// one number a token (kept where the other forms keep beta).  The norm's weights are the head's own (H * v_dim of them)
 enum { DECAY_PER_CHANNEL = 0, DECAY_PER_HEAD = 1, DECAY_CONSTANT = 2, DECAY_FORGET_GATE = 3, DECAY_LOG_SIGMOID = 4,
-       DECAY_STEP = 5 };
+       DECAY_STEP = 5, DECAY_BONUS = 6 };
 
 template <typename T, int DIM>
 __global__ void __launch_bounds__(DIM > 0 ? 256 : 1024)
@@ -831,8 +837,10 @@ delta_rule_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in,
     const bool forget = decay_mode == DECAY_FORGET_GATE;
     const bool gated = decay_mode == DECAY_LOG_SIGMOID;
     const bool stepped = decay_mode == DECAY_STEP;
-    const bool corrects = !plain && !forget && !gated && !stepped;   // the delta rule proper: the state is corrected towards v
-    const float decay_rate = (plain || gated) ? A_log[head] : (forget ? 0.f : expf(A_log[head]));
+    const bool bonus = decay_mode == DECAY_BONUS;
+    if (bonus) norm_w += (size_t)head * v_dim;
+    const bool corrects = !plain && !forget && !gated && !stepped && !bonus;   // the delta rule proper: the state is corrected towards v
+    const float decay_rate = (plain || gated) ? A_log[head] : ((forget || bonus) ? 0.f : expf(A_log[head]));
     float* S_glob = state + (size_t)slot * state_stride + (size_t)head * k_dim * v_dim;
     // a state too large for shared memory is walked where it lies (DIM == 0 only): a thread touches its own column alone
     const bool in_place = DIM == 0 && state_in_place != 0;
@@ -881,6 +889,21 @@ delta_rule_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in,
                 if (lane == 0) betas[t] = dtv;
                 continue;
             }
+            if (bonus) {
+                const size_t rr = (size_t)(r0 + c0 + t);
+                float now = 0.f;
+                for (int i = lane; i < k_dim; i += 32) {
+                    const float qv = to_f32(row[q_off + i]) * q_scale, kv = to_f32(row[k_off + i]);
+                    qs[t * k_dim + i] = qv;
+                    ks[t * k_dim + i] = kv;
+                    gs[t * k_dim + i] = expf(-expf(to_f32(a_in[rr * lda + (size_t)head * k_dim + i]) + dt_bias[head * k_dim + i]));
+                    now = fmaf(qv * A_log[head * k_dim + i], kv, now);
+                }
+                for (int j = lane; j < v_dim; j += 32) vs[t * v_dim + j] = to_f32(row[v_off + j]);
+                now = warp_sum(now);
+                if (lane == 0) betas[t] = now;
+                continue;
+            }
             float sq = 0.f, sk = 0.f;
             for (int i = lane; i < k_dim; i += 32) {
                 const float qv = to_f32(row[q_off + i]), kv = to_f32(row[k_off + i]);
@@ -921,6 +944,24 @@ delta_rule_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in,
                 const float* qt = qs + t * k_dim;
                 const float* gt = gs + t * k_dim;
                 float dot = 0.f, o = 0.f;
+                if (bonus) {                            // the output first, from the state before the token
+                    const float v = vs[t * v_dim + tid];
+                    if (DIM > 0) {
+#pragma unroll
+                        for (int i = 0; i < REG; ++i) {
+                            o = fmaf(S[i], qt[i], o);
+                            S[i] = fmaf(S[i], gt[i], kt[i] * v);
+                        }
+                    } else {
+                        for (int i = 0; i < k_dim; ++i) {
+                            const float s = S_sh[i * v_dim + tid];
+                            o = fmaf(s, qt[i], o);
+                            S_sh[i * v_dim + tid] = fmaf(s, gt[i], kt[i] * v);
+                        }
+                    }
+                    os[t * v_dim + tid] = fmaf(betas[t], v, o);
+                    continue;
+                }
                 if (DIM > 0) {
 #pragma unroll
                     for (int i = 0; i < REG; ++i) {
@@ -992,7 +1033,7 @@ delta_rule_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in,
 // unnormalised, in 32-bit (`o_raw`, (n, H * v_dim)); delta_out_norm_kernel normalises them.
 // MODE 0: the delta rule (decays from projections, the state corrected towards v); 1: a constant decay per head,
 // silu on q, k and v, no correction; 2: the forget gate of DECAY_FORGET_GATE; 3: the powered gate of DECAY_LOG_SIGMOID;
-// 4: the step size of DECAY_STEP.
+// 4: the step size of DECAY_STEP; 5: the bonus of DECAY_BONUS.
 template <typename T, int DL, int LANES, int COLS, int MODE>
 __global__ void __launch_bounds__(COLS * LANES)
 delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in, int ldb, const T* __restrict__ a_in,
@@ -1023,8 +1064,8 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
     const int col = tid / LANES, part = tid % LANES;
     // PLAIN: the decay is a constant per head and the state takes k v^T as it is, so the walk needs neither the decays of
     // the chunk nor the first of its two sums over the lanes of a column
-    constexpr bool plain = MODE == 1, forget = MODE == 2, gated = MODE == 3, stepped = MODE == 4;
-    const float decay_rate = (plain || gated) ? A_log[head] : (forget ? 0.f : expf(A_log[head]));
+    constexpr bool plain = MODE == 1, forget = MODE == 2, gated = MODE == 3, stepped = MODE == 4, bonus = MODE == 5;
+    const float decay_rate = (plain || gated) ? A_log[head] : ((forget || bonus) ? 0.f : expf(A_log[head]));
     float* S_glob = state + (size_t)slot * state_stride + (size_t)head * KDIM * v_dim + col0 + col;
     float S[DL];
     pdl_wait();
@@ -1055,7 +1096,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
         bias[i] = plain ? 0.f : dt_bias[a_at + (sub * CH + i) * a_step];
-        low[i] = forget ? A_log[a_at + sub * CH + i] : 0.f;
+        low[i] = (forget || bonus) ? A_log[a_at + sub * CH + i] : 0.f;
     }
     fetch(0);
     for (int c0 = 0; c0 < rows; c0 += DELTA_CHUNK) {
@@ -1064,7 +1105,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
         {
             float sq = 0.f, sk = 0.f;
 #pragma unroll
-            for (int i = 0; i < CH; ++i) { sq = fmaf(rq[i], rq[i], sq); sk = fmaf(rk[i], rk[i], sk); }
+            for (int i = 0; i < CH; ++i) { sq = fmaf(bonus ? rq[i] * low[i] : rq[i], bonus ? rk[i] : rq[i], sq); sk = fmaf(rk[i], rk[i], sk); }
 #pragma unroll
             for (int o = 1; o < PT; o <<= 1) {
                 sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -1072,7 +1113,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
             }
             const float fq = q_scale / sqrtf(sq + unit_eps), fk = 1.f / sqrtf(sk + unit_eps);
             // a decay per head is one number for all of a token's key channels: made once, not once a channel
-            const float g_head = (a_step == 0 && !plain && !forget && !gated) ? expf(-decay_rate * softplus_f(ra[0] + bias[0])) : 0.f;
+            const float g_head = (a_step == 0 && !plain && !forget && !gated && !bonus) ? expf(-decay_rate * softplus_f(ra[0] + bias[0])) : 0.f;
 #pragma unroll
             for (int i = 0; i < CH; ++i) {
                 const int ch = sub * CH + i;
@@ -1082,6 +1123,10 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
                     qs[pt][at] = silu_f(rq[i]);
                     ks[pt][at] = (1.f - low[i]) * open;                          // 1 - f
                     gs[pt][at] = low[i] + (1.f - low[i]) * (1.f - open);         // f
+                } else if (bonus) {
+                    qs[pt][at] = rq[i] * q_scale;
+                    ks[pt][at] = rk[i];
+                    gs[pt][at] = expf(-expf(ra[i] + bias[i]));
                 } else if (gated || stepped) {
                     qs[pt][at] = rq[i] * q_scale;
                     ks[pt][at] = rk[i];
@@ -1094,7 +1139,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
             }
 #pragma unroll
             for (int i = 0; i < VPT; ++i) vs[pt][sub * VPT + i] = plain ? silu_f(rv[i]) : rv[i];
-            if (sub == 0) betas[pt] = stepped ? softplus_f(ra[0] + bias[0]) : 1.f / (1.f + expf(-rb));
+            if (sub == 0) betas[pt] = bonus ? sq * q_scale : stepped ? softplus_f(ra[0] + bias[0]) : 1.f / (1.f + expf(-rb));
         }
         __syncthreads();
         if (c0 + DELTA_CHUNK < rows) fetch(c0 + DELTA_CHUNK);
@@ -1137,6 +1182,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
             if (plain) {
 #pragma unroll
                 for (int i = 0; i < DL; ++i) S[i] *= decay_rate;
+            } else if (bonus) {
             } else if (forget || gated || stepped) {
 #pragma unroll
                 for (int i = 0; i < DL / 2; ++i) { S[2 * i] *= gc[i].x; S[2 * i + 1] *= gc[i].y; }
@@ -1153,6 +1199,14 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
                 u = bc * (vc - dot);
             }
             d0 = d1 = 0.f;
+            if (bonus) {                                // the output reads the state before the token
+#pragma unroll
+                for (int i = 0; i < DL / 2; ++i) {
+                    d0 = fmaf(S[2 * i], qc[i].x, d0); d1 = fmaf(S[2 * i + 1], qc[i].y, d1);
+                    S[2 * i] = fmaf(S[2 * i], gc[i].x, kc[i].x * vc); S[2 * i + 1] = fmaf(S[2 * i + 1], gc[i].y, kc[i].y * vc);
+                }
+                if (part == 0) d0 = fmaf(bc, vc, d0);
+            } else
 #pragma unroll
             for (int i = 0; i < DL / 2; ++i) {
                 S[2 * i] = fmaf(kc[i].x, u, S[2 * i]); S[2 * i + 1] = fmaf(kc[i].y, u, S[2 * i + 1]);
@@ -1168,12 +1222,13 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
     for (int i = 0; i < DL; ++i) S_glob[(size_t)(part * DL + i) * v_dim] = S[i];
 }
 
-// out[r, head, :] = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(gate) for every (row, head): a warp each.
+// out[r, head, :] = o / sqrt(mean(o^2) + eps) * norm_w * act(gate) for every (row, head): a warp each.  own_weights: norm_w
+// holds v_dim weights for every head, else v_dim for all of them.
 template <typename T>
 __global__ void __launch_bounds__(128)
 delta_out_norm_kernel(const float* __restrict__ o_raw, const T* __restrict__ gate, int ldg, const float* __restrict__ norm_w,
                       float eps, T* __restrict__ out, int ldo, const int* __restrict__ row_slot, int n, int H, int v_dim,
-                      int gate_act) {
+                      int gate_act, int own_weights) {
     pdl_launch_dependents();
     const int idx = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (idx >= n * H) return;
@@ -1181,12 +1236,13 @@ delta_out_norm_kernel(const float* __restrict__ o_raw, const T* __restrict__ gat
     if (row_slot[r] < 0) return;
     pdl_wait();
     const float* o = o_raw + (size_t)r * H * v_dim + (size_t)head * v_dim;
+    const float* w = norm_w + (own_weights ? (size_t)head * v_dim : 0);
     float ss = 0.f;
     for (int j = lane; j < v_dim; j += 32) ss += o[j] * o[j];
     ss = warp_sum(ss);
     const float f = rsqrtf(ss / (float)v_dim + eps);
     for (int j = lane; j < v_dim; j += 32) {
-        float x = o[j] * f * norm_w[j];
+        float x = o[j] * f * w[j];
         if (gate != nullptr) x *= gate_f(to_f32(gate[(size_t)r * ldg + head * v_dim + j]), gate_act);
         out[(size_t)r * ldo + head * v_dim + j] = from_f32<T>(x);
     }
@@ -1259,6 +1315,10 @@ static int launch_delta_rule_split(const T* qkv, int ld, const T* b_in, int ldb,
         tis_launch(delta_rule_split_kernel<T, DL, LANES, COLS, 4>, grid, dim3(COLS * LANES), 0, stream, qkv, ld, b_in, ldb, a_in,
                    lda, A_log, dt_bias, unit_eps, q_scale, state, state_stride, o_raw, row_slot, row_last, seg_row0, H, G, v_dim,
                    decay_mode);
+    else if (decay_mode == DECAY_BONUS)
+        tis_launch(delta_rule_split_kernel<T, DL, LANES, COLS, 5>, grid, dim3(COLS * LANES), 0, stream, qkv, ld, b_in, ldb, a_in,
+                   lda, A_log, dt_bias, unit_eps, q_scale, state, state_stride, o_raw, row_slot, row_last, seg_row0, H, G, v_dim,
+                   decay_mode);
     else
         tis_launch(delta_rule_split_kernel<T, DL, LANES, COLS, 0>, grid, dim3(COLS * LANES), 0, stream, qkv, ld, b_in, ldb, a_in,
                    lda, A_log, dt_bias, unit_eps, q_scale, state, state_stride, o_raw, row_slot, row_last, seg_row0, H, G, v_dim,
@@ -1271,7 +1331,7 @@ static int launch_delta_rule_split(const T* qkv, int ld, const T* b_in, int ldb,
         return tis_check_launch("row_out_norm");
     }
     tis_launch(delta_out_norm_kernel<T>, dim3((n * H + 3) / 4), dim3(128), 0, stream, (const float*)o_raw, gate, ldg, norm_w, eps,
-               out, ldo, row_slot, n, H, v_dim, gate_act);
+               out, ldo, row_slot, n, H, v_dim, gate_act, (int)(decay_mode == DECAY_BONUS));
     return tis_check_launch("delta_out_norm");
 }
 
@@ -1320,7 +1380,7 @@ static int matrix_state_recurrence(int dtype, const void* qkv, int ld, const voi
                                    int k_dim, int v_dim, int narrow, const int* seg_row0, int segments, int decay_mode,
                                    int gate_act, cudaStream_t stream) {
     if (n <= 0) return TIS_OK;
-    if (decay_mode < DECAY_PER_CHANNEL || decay_mode > DECAY_STEP || gate_act < 0 || gate_act > 1 ||
+    if (decay_mode < DECAY_PER_CHANNEL || decay_mode > DECAY_BONUS || gate_act < 0 || gate_act > 1 ||
         ((decay_mode == DECAY_CONSTANT || decay_mode == DECAY_STEP) && o_raw == nullptr)) {
         tis_set_error("delta_rule: decay mode %d, gate activation %d%s", decay_mode, gate_act,
                       o_raw == nullptr ? ", no scratch for the outputs" : "");
@@ -1454,4 +1514,18 @@ TIS_API int tis_state_space_scan(int dtype, const void* cbx, int ld, const void*
     return matrix_state_recurrence(dtype, cbx, ld, nullptr, 0, dt_in, ldd, nullptr, 0, A_log, dt_bias, nullptr, 0.f, 0.f, 1.f,
                                    state, state_stride, nullptr, 0, o_raw, row_slot, row_last, n, H, G, state_dim, v_dim,
                                    narrow, seg_row0, segments, DECAY_STEP, 0, stream);
+}
+
+// The recurrence with a bonus for the current token (DECAY_BONUS): a row of `rkvg` holds r, k and v of H heads (dim each) and
+// the projection of the gate (H * dim); `w_in` (n, H * dim) the decay's projection, `w_bias` its bias, `u` the bonus (H * dim
+// each).  o = (S + diag(u) k v^T)^T r, S <- diag(exp(-exp(w_in + w_bias))) S + k v^T; per head out = o / sqrt(mean(o^2) + eps)
+// * norm_w (H * dim weights) * silu(gate).  `o_raw`: n * H * dim floats of scratch where tis_delta_rule_splits.
+TIS_API int tis_time_mix(int dtype, const void* rkvg, int ld, const void* w_in, int ldw, const float* u, const float* w_bias,
+                         const float* norm_w, float eps, float* state, size_t state_stride, void* out, int ldo, float* o_raw,
+                         const int* row_slot, const int* row_last, int n, int H, int dim, int narrow, const int* seg_row0,
+                         int segments, cudaStream_t stream) {
+    const size_t gate_at = (size_t)3 * H * dim * (dtype == TIS_BF16 ? 2 : 4);
+    return matrix_state_recurrence(dtype, rkvg, ld, nullptr, 0, w_in, ldw, (const char*)rkvg + gate_at, ld, u, w_bias, norm_w,
+                                   eps, 0.f, 1.f, state, state_stride, out, ldo, o_raw, row_slot, row_last, n, H, H, dim, dim,
+                                   narrow, seg_row0, segments, DECAY_BONUS, 1, stream);
 }

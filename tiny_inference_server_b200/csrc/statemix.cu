@@ -6,7 +6,8 @@
 //     their own: what a layer whose two sublayers read the same stream needs in one pass;
 //   * the step between the projections and the cache of an attention whose values are its keys before rotation:
 //     rotate queries in place, write rotated keys as key rows and the unrotated keys as value rows;
-//   * what follows the scan of a selective state space: skip, gate, norm in groups.
+//   * what follows the scan of a selective state space: skip, gate, norm in groups;
+//   * mixes of every row with the row of the token before it, which is part of a request's state.
 //
 // One CTA per row of the step.  A row whose request slot is negative is padding.
 #include "common.cuh"
@@ -274,6 +275,52 @@ skip_gate_group_norm_kernel(const float* __restrict__ o_raw, const T* __restrict
     grouped_norm_write<T>(row, d, groups, eps, w, out + (size_t)r * ldo, nullptr, (T*)nullptr, nullptr, red);
 }
 
+// ------------------------------------------------------------------------------------------------------------
+// out[r, s] = x[r] + (before - x[r]) * mu[s] for every s of S mixes: `before` is the row of the token before (the row ahead of
+// r when that belongs to the same request, else the request's state, zero at the start of a sequence), mu (S, d).  The CTA
+// of a request's first row in the step reads the state and then sets it to the request's last row.  `out` (n, S, d).
+// ------------------------------------------------------------------------------------------------------------
+template <typename T, int N>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ mu, int S, float* __restrict__ state,
+                   size_t state_stride, T* __restrict__ out, const int* __restrict__ row_slot, const int* __restrict__ row_last,
+                   int d) {
+    pdl_launch_dependents();
+    const int r = blockIdx.x;
+    const int slot = row_slot[r];
+    if (slot < 0) return;
+    const bool first = !(r > 0 && row_slot[r - 1] == slot);
+    const int last = first ? row_last[r] : 0;
+    pdl_wait();
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * N; i < d; i += gridDim.y * blockDim.x * N) {
+        float h[N], b[N];
+        if (N > 1) {
+            if constexpr (N > 1) Vec16<T>::load(x + (size_t)r * ldx + i, h);
+        } else h[0] = to_f32(x[(size_t)r * ldx + i]);
+        if (first) {
+            float* s = state + (size_t)slot * state_stride + i;
+            float keep[N];
+            if constexpr (N > 1) Vec16<T>::load(x + (size_t)last * ldx + i, keep);
+            else keep[0] = to_f32(x[(size_t)last * ldx + i]);
+#pragma unroll
+            for (int j = 0; j < N; ++j) { b[j] = s[j]; s[j] = keep[j]; }
+        } else {
+            if constexpr (N > 1) Vec16<T>::load(x + (size_t)(r - 1) * ldx + i, b);
+            else b[0] = to_f32(x[(size_t)(r - 1) * ldx + i]);
+        }
+#pragma unroll
+        for (int j = 0; j < N; ++j) b[j] -= h[j];
+        for (int s = 0; s < S; ++s) {
+            float o[N];
+#pragma unroll
+            for (int j = 0; j < N; ++j) o[j] = fmaf(b[j], mu[(size_t)s * d + i + j], h[j]);
+            T* dst = out + ((size_t)r * S + s) * d + i;
+            if constexpr (N > 1) Vec16<T>::store(dst, o);
+            else dst[0] = from_f32<T>(o[0]);
+        }
+    }
+}
+
 // out = a * sa + b * sb, element by element over n rows of d (row strides free), the sum in 32-bit.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -357,6 +404,25 @@ TIS_API int tis_skip_gate_group_norm(int dtype, const float* o_raw, const void* 
                    ldz, w, groups, eps, (T*)out, ldo, row_slot, H, v_dim);
     });
     return tis_check_launch("skip_gate_group_norm");
+}
+
+TIS_API int tis_token_shift(int dtype, const void* x, int ldx, const float* mu, int mixes, float* state, size_t state_stride,
+                            void* out, const int* row_slot, const int* row_last, int n, int d, cudaStream_t stream) {
+    if (n <= 0) return TIS_OK;
+    if (d <= 0 || mixes <= 0 || ldx < d) {
+        tis_set_error("token_shift: %d mixes of rows of %d elements (stride %d)", mixes, d, ldx);
+        return TIS_BAD_SIZE;
+    }
+    TIS_DISPATCH_DTYPE(dtype, T, {
+        constexpr int N = Vec16<T>::N;
+        if (d % N == 0 && ldx % N == 0 && ((uintptr_t)x | (uintptr_t)out) % 16 == 0)
+            tis_launch(token_shift_kernel<T, N>, dim3(n, (d / N + 127) / 128), dim3(128), 0, stream, (const T*)x, ldx, mu, mixes,
+                       state, state_stride, (T*)out, row_slot, row_last, d);
+        else
+            tis_launch(token_shift_kernel<T, 1>, dim3(n, (d + 127) / 128), dim3(128), 0, stream, (const T*)x, ldx, mu, mixes, state,
+                       state_stride, (T*)out, row_slot, row_last, d);
+    });
+    return tis_check_launch("token_shift");
 }
 
 TIS_API int tis_scaled_sum(int dtype, const void* a, int lda, float sa, const void* b, int ldb, float sb, void* out, int ldo,

@@ -1,6 +1,7 @@
 // Attention over a window of the paged cache on the tensor cores (bfloat16, mma.sync m16n8k16), for keys of
 // TIS_KD and values of TIS_VD elements (compiled per pair of widths):
-//   score = q . k * scale - r1[head] * ln(1 + r2[head] * distance),  keys pos - window < j <= pos,
+//   score = q . k * scale (bounded by a tanh if asked) - r1[head] * ln(1 + r2[head] * distance),  keys
+//   first_key(pos, window) .. pos (common.cuh),
 //   softmax in 32-bit, out = softmax . v * sigmoid(gate).
 // A CTA takes one tile of consecutive rows of one request and one kv head, with all the query heads that share
 // the kv head: row r and query head h of the group are packed row r * (H / G) + h of a block of 64 packed rows, so
@@ -67,6 +68,7 @@ struct Params {
     const int* tile_row0; const int* tile_rows;
     int H, G, page_size, window;
     float scale;
+    SoftCap cap;             // bounds the raw scores (k 0: not)
     const float* r1; const float* r2;
     const float* sink;       // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     int v_row;               // elements from one value row of a page to the next (VD, or more when the rows are slices)
@@ -125,7 +127,7 @@ window_attention_mma_kernel(const Params p) {
     const int g = lane >> 2, t4 = lane & 3;
     if (tid == 0) bad = 0;
     const int last = pos0 + nrows - 1;                         // the last key any row of the tile sees
-    const int first = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    const int first = first_key(pos0, p.window);
     int ntiles = (last - first) / KEYS + 1;
     int kt_begin = 0;
     const int splits = gridDim.z;
@@ -178,6 +180,8 @@ window_attention_mma_kernel(const Params p) {
     }
     // positions of the first and last row among this warp's packed rows
     const int w_lo = pos0 + base / gq, w_hi = min(pos0 + (base + 15) / gq, last);
+    const int w_lo_first = first_key(w_lo, p.window), w_hi_first = first_key(w_hi, p.window);
+    const int lo_a = first_key(pos_a, p.window), lo_b = first_key(pos_b, p.window);
     for (int kt = kt_begin; kt < ntiles; ++kt) {
         const int stage = (kt - kt_begin) & 1;
         if (kt + 1 < ntiles)
@@ -189,7 +193,7 @@ window_attention_mma_kernel(const Params p) {
         const bf16* vs = vbuf + stage * KEYS * VS;
         const int j0 = first + kt * KEYS;
         // does this warp see any key of the tile?
-        bool any = base < packed && j0 <= w_hi && (p.window <= 0 || j0 + KEYS - 1 > w_lo - p.window);
+        bool any = base < packed && j0 <= w_hi && j0 + KEYS - 1 >= w_lo_first;
         if (split_keys) any = any && (kt & 3) == warp;
         if (any) {
             float s[KEYS / 8][4];
@@ -207,7 +211,13 @@ window_attention_mma_kernel(const Params p) {
             }
             // scale, bias, mask; the maximum of each row over the tile.  A tile that every row of the warp sees
             // whole (the usual case inside a window) needs no mask.
-            const bool whole = base + 15 < packed && j0 + KEYS - 1 <= w_lo && (p.window <= 0 || j0 > w_hi - p.window);
+            const bool whole = base + 15 < packed && j0 + KEYS - 1 <= w_lo && j0 >= w_hi_first;
+            if (p.cap.k != 0.f) {
+#pragma unroll
+                for (int n = 0; n < KEYS / 8; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[n][e] = soft_capped(s[n][e], p.cap);
+            }
             float mx[2] = {-INFINITY, -INFINITY};
             if (whole) {
 #pragma unroll
@@ -228,7 +238,7 @@ window_attention_mma_kernel(const Params p) {
                     for (int e = 0; e < 4; ++e) {
                         const int j = j0 + n * 8 + 2 * t4 + (e & 1);
                         const int pos = (e & 2) ? pos_b : pos_a;
-                        const bool ok = ((e & 2) ? row_b : row_a) && j <= pos && (p.window <= 0 || j > pos - p.window);
+                        const bool ok = ((e & 2) ? row_b : row_a) && j <= pos && j >= ((e & 2) ? lo_b : lo_a);
                         float v = -INFINITY;
                         if (ok) v = s[n][e] * p.scale - ((e & 2) ? b1_b : b1_a) * __logf(fmaf((e & 2) ? b2_b : b2_a, (float)(pos - j), 1.f));
                         s[n][e] = v;
@@ -439,7 +449,7 @@ TIS_API int tis_window_attention_mma(const void* q, int ldq, const void* gate, i
                                      const void* v_pages, size_t v_page_stride, size_t v_head_stride,
                                      const int* block_table, int bt_stride, int num_pages, const int* positions,
                                      const int* row_slot, const int* tile_row0, const int* tile_rows, int num_tiles,
-                                     int H, int G, int page_size, int window, float scale, const float* r1,
+                                     int H, int G, int page_size, int window, float scale, float softcap, const float* r1,
                                      const float* r2, int splits, float* partial, const float* sink, int v_row,
                                      int gate_per_head, int* fault, cudaStream_t stream) {
     if (num_tiles <= 0) return TIS_OK;
@@ -447,7 +457,7 @@ TIS_API int tis_window_attention_mma(const void* q, int ldq, const void* gate, i
         tis_set_error("window_attention_mma: %d key splits%s", splits, splits > 1 ? " without scratch" : "");
         return TIS_BAD_SIZE;
     }
-    if (H <= 0 || G <= 0 || H % G || H / G > ROWS || page_size <= 0 || window < 0 || ldq % 8 || (ldg % 2 && !gate_per_head) ||
+    if (H <= 0 || G <= 0 || H % G || H / G > ROWS || page_size <= 0 || ldq % 8 || (ldg % 2 && !gate_per_head) ||
         ldo % 2 ||
         v_row < VD || v_row % 8 ||
         k_page_stride % 8 || k_head_stride % 8 || v_page_stride % 8 || v_head_stride % 8 ||
@@ -464,7 +474,7 @@ TIS_API int tis_window_attention_mma(const void* q, int ldq, const void* gate, i
     p.v_pages = (const bf16*)v_pages; p.v_page_stride = v_page_stride; p.v_head_stride = v_head_stride;
     p.block_table = block_table; p.bt_stride = bt_stride; p.num_pages = num_pages;
     p.positions = positions; p.row_slot = row_slot; p.tile_row0 = tile_row0; p.tile_rows = tile_rows;
-    p.H = H; p.G = G; p.page_size = page_size; p.window = window; p.scale = scale; p.r1 = r1; p.r2 = r2; p.fault = fault; p.partial = partial; p.sink = sink; p.v_row = v_row;
+    p.H = H; p.G = G; p.page_size = page_size; p.window = window; p.scale = scale; p.cap = soft_cap(softcap, scale); p.r1 = r1; p.r2 = r2; p.fault = fault; p.partial = partial; p.sink = sink; p.v_row = v_row;
     const size_t smem = sizeof(bf16) * ((size_t)2 * KEYS * KS + 2 * KEYS * VS);
     static bool attr_set = false;
     if (!attr_set && smem > 48 * 1024) {

@@ -117,7 +117,7 @@ class ModelRunner:
                                  f"the context limit {self.max_positions}")
         for grp in self.cache.groups:
             need = 0
-            windowed = grp.window is not None
+            windowed = grp.trims
             for e in entries:
                 start = lengths[e.slot]
                 need += grp.pages_to_grow(e.slot, start + len(e.tokens))

@@ -19,7 +19,7 @@ import torch
 from . import build as _build
 
 _lib = None
-ABI_VERSION = 12
+ABI_VERSION = 13
 #: launches of this library's kernels so far (library matrix products are not counted)
 launches = 0
 #: calls by kind, for tests that must know which kernel a product or an attention went to
@@ -116,7 +116,7 @@ SKINNY_SWIGLU_MAX_ROWS = int(os.environ.get("TIS_SKINNY_SWIGLU_MAX_ROWS", "16"))
 SWAP_SWIGLU_MAX_ROWS = int(os.environ.get("TIS_SWAP_SWIGLU_MAX_ROWS", "32"))
 EPI_STORE, EPI_SWIGLU, EPI_RESIDUAL = 0, 1, 2
 #: a store through an activation, by the activation's name (the weight-streaming products)
-EPI_ACT = {"relu2": 3, "gelu_tanh": 4, "silu": 5}
+EPI_ACT = {"relu2": 3, "gelu_tanh": 4, "silu": 5, "tanh": 6}
 #: the norm between two weight-streaming products is folded into them (``ResidualSink`` / ``ScaledRows``);
 #: TIS_FUSED_NORM=0 keeps the norm kernel
 FUSED_NORM = os.environ.get("TIS_FUSED_NORM", "1") != "0"
@@ -148,8 +148,9 @@ def gate_clamped(limit: float, alpha: float = 1.702, shift: float = 1.0) -> Gate
 SILU = gate_silu()
 
 #: the factor a norm multiplies a row with, as a function of the row's sum of squares s over a width d:
-#: "l2_eps": sqrt(d) / (sqrt(s) + eps) (eps added to the L2 norm); "mean_eps": rsqrt(s / d + eps)
-NORM_KINDS = {"l2_eps": 0, "mean_eps": 1}
+#: "l2_eps": sqrt(d) / (sqrt(s) + eps) (eps added to the L2 norm); "mean_eps": rsqrt(s / d + eps); "none": 1 (the row kernels
+#: only: the stream as it is, in the type of the products)
+NORM_KINDS = {"l2_eps": 0, "mean_eps": 1, "none": 2}
 
 
 class ResidualSink:
@@ -159,7 +160,7 @@ class ResidualSink:
     product instead of before it.  ``norm`` is whoever made the sink (the reader checks it is the same norm)."""
 
     def __init__(self, values: torch.Tensor, weight: torch.Tensor, eps: float, norm=None, kind: str = "l2_eps"):
-        if kind not in NORM_KINDS:
+        if kind not in NORM_KINDS or kind == "none":
             raise KernelError(f"norm factor {kind!r}: the products know {sorted(NORM_KINDS)}")
         self.values, self.weight, self.eps, self.norm, self.kind = values, weight, float(eps), norm, kind
 
@@ -713,6 +714,16 @@ def plan_splits(num_tiles: int, kv_heads: int, max_kv: int, mode_keys: bool, res
 ATTN_ROTARY = os.environ.get("TIS_ATTN_ROTARY", "1") != "0"
 
 
+def _window_code(window: Optional[int], chunked: bool) -> int:
+    """What the attention kernels take: 0 every earlier key, W > 0 the last W, -C < 0 those of the row's chunk of C positions
+    (``first_key`` in csrc/common.cuh)."""
+    if not window:
+        return 0
+    if window < 0:
+        raise KernelError(f"a window of {window} keys")
+    return -int(window) if chunked else int(window)
+
+
 class PairRotary:
     """A rotation of the first elements of every head, twice as many as ``cos`` and ``sin`` (positions, rot / 2; None: none)
     have columns, element 2i with 2i + 1, and (``norm_eps`` not None) the division of the head by its root mean square
@@ -735,7 +746,8 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
                     positions: torch.Tensor, row_slot: torch.Tensor, num_heads: int, kv_heads: int,
                     head_dim: int, page_size: int, window: Optional[int], fault: torch.Tensor,
                     step=None, rotary=None, write_kv: bool = True, scale: Optional[float] = None,
-                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, chunked: bool = False, softcap: Optional[float] = None,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the step's rows over the cache.  ``q`` is (n, >= H*hd) with the
     queries first in each row (row stride free); ``out`` is (n, H*hd).  The row at position
     p of slot s sees keys max(0, p-window+1)..p of ``plane`` through ``block_table[s]``.
@@ -750,9 +762,17 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
     neighbouring elements paired, and the norm of every head (``rotate_norm_store`` everywhere else).
 
     ``scale`` (positive; 1 / sqrt(head_dim) unless given) multiplies the scores.  ``sink`` (H,) float32: head h's softmax
-    denominator also holds ``exp(sink[h])`` (unscaled; it has no key and no value)."""
+    softmax denominator also holds ``exp(sink[h])`` (unscaled; it has no key and no value).  ``chunked``: instead of the last
+    ``window`` keys a row sees those of its own chunk of ``window`` positions, counted from position 0.  ``softcap`` (not with
+    ``rotary``): a score s becomes ``softcap * tanh(s / softcap)``.  ``gate`` (n, H), row stride free (not with ``rotary``):
+    head h's output is multiplied by ``sigmoid(gate[row, h])``."""
     lib = library()
     n = q.shape[0]
+    window = _window_code(window, chunked)
+    cap = float(softcap or 0.0)
+    ldg = gate.stride(0) if gate is not None else 0
+    if rotary is not None and (cap or gate is not None):
+        raise KernelError("paged_attention: bounded scores and gates go with rows that are rotated already")
     scale = 1.0 / math.sqrt(head_dim) if scale is None else float(scale)
     if not scale > 0:
         raise KernelError(f"paged_attention: the scores are multiplied by a positive number, not {scale}")
@@ -763,7 +783,7 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         _check(lib.tis_paged_attention_simt(
             _dt(q), _p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table), block_table.stride(0),
             plane.shape[0], _p(positions), _p(row_slot), n, num_heads, kv_heads, head_dim, page_size,
-            int(window or 0), _f(scale), _p(sink), _p(fault), _stream()), lib)
+            window, _f(scale), _f(cap), _p(gate), ldg, _p(sink), _p(fault), _stream()), lib)
         return out
     if kv_heads <= 0 or num_heads % kv_heads:
         raise KernelError(f"paged_attention: {num_heads} query heads are not a multiple of {kv_heads} kv heads")
@@ -784,7 +804,7 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
     rows_tiles = tiles.rows
     # keys that the key splits share out: with a window those from the tile's first one on (a tile's rows see at most
     # 63 keys more than one of them does, and the share starts at a multiple of 64)
-    split_kv = max_kv if not window else min(max_kv, int(window) + 128)
+    split_kv = max_kv if not window else min(max_kv, abs(window) + 128)
     w0, wn, wide_count = getattr(tiles, "wide", (None, None, 0))
     # One CTA of the tcgen05 kernel walks all keys of its 128 rows (no key splits yet).  Measured at the
     # 0.9B sizes: with two or more such tiles in the step it wins (256 rows ending at 4096: 51 against
@@ -796,8 +816,8 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         calls["attn_tc"] += 1
         _check(alib.tis_attn_tc(_p(q), q.stride(0), n, _p(out), out.stride(0), _p(plane), _p(block_table),
                                 block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(w0), _p(wn),
-                                wide_count, num_heads, kv_heads, page_size, int(window or 0), _f(scale), _p(sink),
-                                _p(fault), _stream()), alib)
+                                wide_count, num_heads, kv_heads, page_size, window, _f(scale), _f(cap), _p(gate), ldg,
+                                _p(sink), _p(fault), _stream()), alib)
         skip = tiles.rows_in_wide
         if skip == tiles.rows[2]:
             rows_tiles = (None, None, 0)
@@ -823,7 +843,7 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
             row0 = rows = None          # tile i is row i: the kernel reads no tile arrays
         _check(alib.tis_attn_decode_rope(_p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table),
                                          block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(row0),
-                                         _p(rows), count, n, num_heads, kv_heads, page_size, int(window or 0),
+                                         _p(rows), count, n, num_heads, kv_heads, page_size, window,
                                          _f(scale), per, splits, _p(cos), _p(sin), int(bool(write_kv)), *how, _p(sink),
                                          _p(fault), _stream()), alib)
         return out
@@ -841,8 +861,8 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
         # at most eight splits (plan_splits): they merge inside a thread-block cluster, without scratch
         _check(alib.tis_attn_mma_sink(mode, _p(q), q.stride(0), _p(out), out.stride(0), _p(plane), _p(block_table),
                                  block_table.stride(0), plane.shape[0], _p(positions), _p(row_slot), _p(row0),
-                                 _p(rows), count, max_rows, n, num_heads, kv_heads, page_size, int(window or 0), _f(scale),
-                                 per, splits, _p(None), _p(sink), _p(fault), _stream()), alib)
+                                 _p(rows), count, max_rows, n, num_heads, kv_heads, page_size, window, _f(scale),
+                                 per, splits, _p(None), _p(sink), _f(cap), _p(gate), ldg, _p(fault), _stream()), alib)
     return out
 
 
@@ -883,12 +903,12 @@ def softcap_f32(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 #: activations of a feed-forward without a gate
-ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
+ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "tanh": 3}
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
     """out = act(x) element by element over (n, F) (row strides free): ``relu2`` the square of relu, ``gelu_tanh``
-    0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), ``silu``."""
+    0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), ``silu``, ``tanh``."""
     lib = library()
     if kind not in ACTIVATIONS:
         raise KernelError(f"activation {kind!r}: known are {sorted(ACTIVATIONS)}")
@@ -992,13 +1012,15 @@ def window_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
                      v_pages: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor, row_slot: torch.Tensor,
                      num_heads: int, page_size: int, window: Optional[int], scale: float,
                      bias_slope: Optional[torch.Tensor], bias_rate: Optional[torch.Tensor], fault: torch.Tensor,
-                     step=None, sink: Optional[torch.Tensor] = None, gate_per_head: bool = False) -> torch.Tensor:
+                     step=None, sink: Optional[torch.Tensor] = None, gate_per_head: bool = False,
+                     chunked: bool = False, softcap: Optional[float] = None) -> torch.Tensor:
     """Attention of the step's rows over the paged cache with keys and values of any widths:
     ``score = q . k * scale - bias_slope[h] * ln(1 + bias_rate[h] * distance)``, softmax over the keys
     ``max(0, p - window + 1) .. p``, the result times ``sigmoid(gate)`` element by element.  ``q`` (n, H * k_dim),
     ``gate`` (n, H * v_dim) or None, ``out`` (n, H * v_dim); row strides free.  ``sink`` (H,) float32: the softmax's
     denominator of head h also holds ``exp(sink[h])`` (unscaled; it has no value).  ``gate_per_head``: ``gate`` is (n, H),
-    one number per head for all of the head's elements.  The value rows may be a slice of
+    one number per head for all of the head's elements.  ``chunked`` and ``softcap`` (on ``q . k * scale``, before the bias) as in
+    ``paged_attention``.  The value rows may be a slice of
     wider rows (``v_pages`` with a row stride above its width, for instance the first elements of the key rows).
 
     float32, and widths that are not multiples of 16: a CUDA-core kernel, a CTA per row and head.  bfloat16 inside
@@ -1009,6 +1031,7 @@ def window_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     kv_heads, k_dim, v_dim = k_pages.shape[1], k_pages.shape[3], v_pages.shape[3]
     kps, khs = _page_strides(k_pages, k_dim)
     vps, vhs, v_row = _page_strides(v_pages, v_dim, free_rows=True)
+    code, cap = _window_code(window, chunked), float(softcap or 0.0)
     if step is not None and num_heads // kv_heads <= 64 and window_attention_mma_usable(q, gate, out, k_pages, v_pages,
                                                                                           gate_per_head):
         from . import window_plan
@@ -1032,14 +1055,14 @@ def window_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
                                              _p(out), out.stride(0), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
                                              _p(block_table), block_table.stride(0), k_pages.shape[0], _p(positions),
                                              _p(row_slot), _p(row0), _p(rows), count, num_heads, kv_heads, page_size,
-                                             int(window or 0), _f(scale), _p(bias_slope), _p(bias_rate), splits, _p(partial),
+                                             code, _f(scale), _f(cap), _p(bias_slope), _p(bias_rate), splits, _p(partial),
                                              _p(sink), v_row, int(gate_per_head), _p(fault), _stream()), wlib)
         return out
     calls["window_attention"] += 1
     _check(lib.tis_window_attention(_dt(q), _p(q), q.stride(0), _p(gate), gate.stride(0) if gate is not None else 0,
                                     _p(out), out.stride(0), _p(k_pages), kps, khs, _p(v_pages), vps, vhs, _p(block_table),
                                     block_table.stride(0), k_pages.shape[0], _p(positions), _p(row_slot), n, num_heads,
-                                    kv_heads, k_dim, v_dim, page_size, int(window or 0), _f(scale), _p(bias_slope),
+                                    kv_heads, k_dim, v_dim, page_size, code, _f(scale), _f(cap), _p(bias_slope),
                                     _p(bias_rate), _p(sink), v_row, int(gate_per_head), _p(fault), _stream()), lib)
     return out
 
@@ -1289,6 +1312,92 @@ def skip_gate_group_norm(o_raw: torch.Tensor, x: torch.Tensor, skip: torch.Tenso
     return out
 
 
+def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, row_slot: torch.Tensor,
+                row_last: torch.Tensor) -> torch.Tensor:
+    """``out[r, s] = x[r] + (before - x[r]) * mu[s]``: ``before`` is the row of the token before r in its request, zero for a
+    sequence's first token.  ``x`` (n, d), ``mu`` (S, d) float32, ``state`` (slots, >= d) float32: every request's last row so
+    far, read for its first row of the step and brought up to date.  Returns (n, S, d)."""
+    lib = library()
+    n, d = x.shape
+    out = torch.empty((n, mu.shape[0], d), dtype=x.dtype, device=x.device)
+    _check(lib.tis_token_shift(_dt(x), _p(x), x.stride(0), _p(mu), mu.shape[0], _p(state), ctypes.c_size_t(state.stride(0)),
+                               _p(out), _p(row_slot), _p(row_last), n, d, _stream()), lib)
+    return out
+
+
+def gemm_side_by_side(a: torch.Tensor, w: torch.Tensor, w_last: torch.Tensor, act: Optional[str] = None):
+    """Products of several inputs: ``a`` (n, G + 1, K), ``w`` (G, K, N), ``w_last`` (K, M).  Returns (``out`` (n, G * N) with
+    ``a[:, g] @ w[g]`` side by side, ``act(a[:, G] @ w_last)`` (n, M)).  Few bfloat16 rows: one launch of the weight-streaming
+    kernel for all of them; else a batched library product and one more product."""
+    n, groups, k = a.shape[0], w.shape[0], a.shape[2]
+    cols, last = w.shape[2], w_last.shape[1]
+    total = groups * cols + last
+    if (a.dtype == torch.bfloat16 and 0 < n <= SKINNY_MAX_ROWS and k % 8 == 0 and cols % 64 == 0 and last % 8 == 0
+            and _ring_tiles(total, k) <= RING_MAX_TILES and a.is_contiguous() and w.is_contiguous() and w_last.is_contiguous()
+            and a.data_ptr() % 16 == 0):
+        lib = library()
+        out = torch.empty((n, total), dtype=a.dtype, device=a.device)
+        calls["gemm_skinny_groups"] += 1
+        _check(lib.tis_gemm_skinny_groups(_p(a), a.stride(0), ctypes.c_size_t(a.stride(1)), _p(w), groups, cols, _p(w_last), last,
+                                          EPI_ACT[act] if act is not None else EPI_STORE, _p(out), out.stride(0), n, k,
+                                          _ksplit(total, k), _p(tc_fault()), _stream()), lib)
+        return out[:, :groups * cols], out[:, groups * cols:]
+    out = torch.empty((n, groups * cols), dtype=a.dtype, device=a.device)
+    gemm_heads(a[:, :groups], w, out.unflatten(1, (groups, cols)))
+    return out, gemm(a[:, groups], w_last, act=act)
+
+
+def time_mix(rkvg: torch.Tensor, w_in: torch.Tensor, u: torch.Tensor, w_bias: torch.Tensor, norm_weight: torch.Tensor, eps: float,
+             state: torch.Tensor, out: torch.Tensor, row_slot: torch.Tensor, row_last: torch.Tensor, num_heads: int, dim: int,
+             requests: Optional[int] = None, segments=None) -> torch.Tensor:
+    """A matrix state per head with a decay per key channel and a bonus for the current token, over the rows of every request,
+    from and into ``state`` (slots, H, dim, dim) float32 (a view with a free slot stride).  A row of ``rkvg``: r, k, v of H heads
+    (``dim`` each) and the gate's projection (H * dim); ``w_in`` (n, H * dim) the decay's projection, ``w_bias`` and the bonus
+    ``u`` (H * dim) float32.  Per head ``o = (S + diag(u) k v^T)^T r``, then ``S <- diag(exp(-exp(w_in + w_bias))) S + k v^T``;
+    ``out = o / rms(o) * norm_weight * silu(gate)`` (H * dim weights).  ``requests`` and ``segments`` as for ``delta_rule``."""
+    lib = library()
+    n = rkvg.shape[0]
+    if rkvg.dtype != w_in.dtype or rkvg.stride(1) != 1 or w_in.stride(1) != 1:
+        raise KernelError("time_mix: the rows and the decays' projection are dense and of one type")
+    narrow = _recurrence_spread(requests, num_heads, dim)
+    raw = None
+    if lib.tis_delta_rule_splits(dim, dim):
+        raw = torch.empty((n, num_heads * dim), dtype=torch.float32, device=rkvg.device)
+        global launches
+        launches += 1
+    _check(lib.tis_time_mix(_dt(rkvg), _p(rkvg), rkvg.stride(0), _p(w_in), w_in.stride(0), _p(u), _p(w_bias), _p(norm_weight),
+                            _f(eps), _p(state), ctypes.c_size_t(state.stride(0)), _p(out), out.stride(0), _p(raw), _p(row_slot),
+                            _p(row_last), n, num_heads, dim, int(narrow), _p(segments[0] if segments is not None else None),
+                            int(segments[1]) if segments is not None else 0, _stream()), lib)
+    return out
+
+
+#: (requests x channels) of a step below which a selective scan keeps two states a lane instead of four
+SCAN_FINE_MAX_CHANNELS = int(os.environ.get("TIS_SCAN_FINE_MAX_CHANNELS", "0"))
+
+
+def selective_scan(x: torch.Tensor, dt_in: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, b: torch.Tensor,
+                   c: torch.Tensor, skip: torch.Tensor, z: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                   row_slot: torch.Tensor, row_last: torch.Tensor, segments=None) -> torch.Tensor:
+    """A selective scan with a decay per channel and state over the rows of every request, from and into ``state`` (slots,
+    channels, N) float32 (a view with a free slot stride): ``dt = softplus(dt_in + dt_bias)``; ``S <- exp(-dt exp(a_log)) S +
+    dt x b^T``; ``out = (S c + skip * x) * silu(z)``.  ``x, z, out`` (n, channels), ``b, c`` (n, N) with free row strides (the
+    same for both), ``dt_in`` (n, channels) float32, ``a_log`` (channels, N), ``dt_bias, skip`` (channels) float32.  N at most
+    256.  ``segments`` as for ``delta_rule``."""
+    lib = library()
+    n, channels = x.shape
+    states = a_log.shape[1]
+    if b.stride(0) != c.stride(0) or dt_in.dtype != torch.float32 or not (x.dtype == b.dtype == c.dtype == z.dtype == out.dtype):
+        raise KernelError("selective_scan: b and c are slices of the same rows, the step sizes 32-bit, the rest of one type")
+    requests = int(segments[1]) if segments is not None else n
+    calls["selective_scan"] += 1
+    _check(lib.tis_selective_scan(_dt(x), _p(x), x.stride(0), _p(dt_in), dt_in.stride(0), _p(dt_bias), _p(a_log), _p(b), _p(c),
+                                  b.stride(0), _p(skip), _p(z), z.stride(0), _p(state), ctypes.c_size_t(state.stride(0)), _p(out),
+                                  out.stride(0), _p(row_slot), _p(row_last), _p(segments[0] if segments is not None else None),
+                                  requests, n, channels, states, int(requests * channels <= SCAN_FINE_MAX_CHANNELS), _stream()), lib)
+    return out
+
+
 def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, tokens: torch.Tensor, positions: torch.Tensor,
                 row_slot: torch.Tensor, row_last: torch.Tensor, prev: torch.Tensor, out: torch.Tensor, scale: float,
                 buckets: int, mul_prev: int, mul_cur: int) -> torch.Tensor:
@@ -1335,14 +1444,17 @@ def add_layer_norm(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delt
 def rotate_norm_store(qkv: torch.Tensor, num_heads: int, kv_heads: int, dim: int, v_dim: int, cos: Optional[torch.Tensor],
                       sin: Optional[torch.Tensor], interleaved: bool, norm: bool, eps: float, k_pages: Optional[torch.Tensor],
                       v_pages: Optional[torch.Tensor], block_table: torch.Tensor, positions: torch.Tensor,
-                      row_slot: torch.Tensor, page_size: int, fault: torch.Tensor, permuted: bool = False) -> None:
+                      row_slot: torch.Tensor, page_size: int, fault: torch.Tensor, permuted: bool = False,
+                      whole_weight: Optional[torch.Tensor] = None) -> None:
     """Between the projections and the cache of an attention whose queries and keys are rotated and then normed head by
     head.  A row of ``qkv``: H query heads and G key heads of ``dim`` elements, G value heads of ``v_dim``.  The first
     elements of every query and key head, twice as many as ``cos`` and ``sin`` (positions, rot / 2; None: none) have columns,
     are rotated by the row's position (``interleaved``: element 2i with 2i + 1, else i with i + rot / 2); with ``norm`` the
     head is then divided by its root mean square (eps inside the root).  Queries in place; keys and values into the row's
     page, in the row format of ``paged_attention`` if ``permuted`` (16-byte chunks permuted by the position), else as they
-    are.  ``kv_heads`` 0: the rows hold queries only and nothing is stored.  Everything is computed in 32-bit."""
+    are.  ``kv_heads`` 0: the rows hold queries only and nothing is stored.  ``whole_weight`` ((H + G) * dim float32: the queries'
+    weights, then the keys'): the norm comes *before* the rotation and runs over all query heads, and over all key heads, at
+    once (``norm`` is then not looked at).  Everything is computed in 32-bit."""
     lib = library()
     n = qkv.shape[0]
     rot = 0 if cos is None else 2 * cos.shape[1]
@@ -1356,8 +1468,11 @@ def rotate_norm_store(qkv: torch.Tensor, num_heads: int, kv_heads: int, dim: int
         k_pages = v_pages = None
     if qkv.stride(1) != 1:
         raise KernelError("rotate_norm_store: the rows are not dense")
+    if whole_weight is not None and (whole_weight.numel() != (num_heads + kv_heads) * dim or whole_weight.dtype != torch.float32
+                                     or not whole_weight.is_contiguous()):
+        raise KernelError("rotate_norm_store: one 32-bit weight for every query and key element")
     _check(lib.tis_rotate_norm_store(_dt(qkv), _p(qkv), qkv.stride(0), num_heads, kv_heads, dim, v_dim, rot, int(interleaved),
-                                     int(permuted), _p(cos), _p(sin), int(norm), _f(eps), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
+                                     int(permuted), _p(cos), _p(sin), int(norm), _f(eps), _p(whole_weight), _p(k_pages), kps, khs, _p(v_pages), vps, vhs,
                                      page_size, k_pages.shape[0] if k_pages is not None else 0, _p(block_table),
                                      block_table.stride(0), _p(positions), _p(row_slot), _p(fault), n, _stream()), lib)
 
@@ -1423,24 +1538,24 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torc
 
 
 def moe_gate_up(x: torch.Tensor, chosen: torch.Tensor, w_gate_up: torch.Tensor, act: Optional[str] = None,
-                form: GateForm = SILU) -> torch.Tensor:
+                form: GateForm = SILU, in_weights: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``hidden[r * top + k] = gated(Wg[e] x[r], Wu[e] x[r])`` in the form ``form`` with ``e = chosen[r, k]``: ``w_gate_up`` (E, 2, F, d)
     holds every expert's gate and up matrices (out, in); the result is (n * top, F) in the dtype of ``x``.  ``act``
-    (``ACTIVATIONS``): units without a gate, ``hidden = act(Wu[e] x[r])`` with ``w_gate_up`` (E, F, d)."""
+    (``ACTIVATIONS``): units without a gate, ``hidden = act(Wu[e] x[r])`` with ``w_gate_up`` (E, F, d).  ``in_weights`` (n, top): multiplies every unit's input."""
     lib = library()
     n, d = x.shape
     top = chosen.shape[1]
     experts, hidden = w_gate_up.shape[0], w_gate_up.shape[-2]
     out = torch.empty((n * top, hidden), dtype=x.dtype, device=x.device)
     _check(lib.tis_moe_gate_up(_dt(x), _p(x), x.stride(0), _p(chosen), _p(w_gate_up), _p(out), n, d, top, experts, hidden,
-                               ACTIVATIONS[act] if act is not None else -1, form, _stream()), lib)
+                               ACTIVATIONS[act] if act is not None else -1, form, _p(in_weights), _stream()), lib)
     return out
 
 
-def moe_down(hidden: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_down: torch.Tensor,
+def moe_down(hidden: torch.Tensor, chosen: torch.Tensor, weights: Optional[torch.Tensor], w_down: torch.Tensor,
              shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor]) -> torch.Tensor:
     """``out[r] = sum_k weights[r, k] * Wd[chosen[r, k]] hidden[r * top + k] (+ shared_gate[r] * shared[r]; the gate None: + shared[r])``:
-    ``w_down`` (E, d, F) (out, in), ``hidden`` (n * top, F), ``shared`` (n, d) or None; the result is (n, d)."""
+    ``w_down`` (E, d, F) (out, in), ``hidden`` (n * top, F), ``shared`` (n, d) or None; ``weights`` None: 1; the result is (n, d)."""
     lib = library()
     n, top = chosen.shape
     experts, d, f = w_down.shape
@@ -1503,10 +1618,11 @@ MOE_TC_MIN_PAIRS = int(os.environ.get("TIS_MOE_TC_MIN_PAIRS", "1024"))
 
 def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                 shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor], act: Optional[str] = None,
-                form: GateForm = SILU) -> torch.Tensor:
+                form: GateForm = SILU, weigh_input: bool = False) -> torch.Tensor:
     """``out[r] = sum_k weights[r, k] * unit(chosen[r, k])(x[r]) (+ shared_gate[r] * shared[r], or + shared[r])`` with the gated
     units ``unit(e)(x) = Wd[e] gated(Wg[e] x, Wu[e] x)`` in the form ``form``: ``w_gate_up`` (E, 2, F, d), ``w_down`` (E, d, F); or, with ``act``
-    (``ACTIVATIONS``), units without a gate, ``Wd[e] act(Wu[e] x)`` and ``w_gate_up`` (E, F, d).  Few rows, and
+    (``ACTIVATIONS``), units without a gate, ``Wd[e] act(Wu[e] x)`` and ``w_gate_up`` (E, F, d).  ``weigh_input``: ``sum_k unit(chosen[r, k])(weights[r, k] *
+    x[r])`` instead (the weight multiplies both projections of the unit in 32-bit).  Few rows, and
     float32: ``moe_gate_up`` and ``moe_down`` (a dot product per output element, the weights read where they lie).  Many
     bfloat16 rows: the rows are sorted by expert on the device and every expert's rows run as tiles on the tensor
     cores; nothing is read back, so either way the step can be captured in a graph."""
@@ -1533,7 +1649,7 @@ def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_
         _check(lib.tis_moe_grouped_tc(_p(x), x.stride(0), _p(chosen), _p(weights), _p(w_gate_up), _p(w_down), _p(shared),
                                       shared.stride(0) if shared is not None else 0, _p(shared_gate), _p(out), _p(sorted_pair),
                                       _p(pair_place), _p(tile_expert), _p(xs), _p(hid), _p(y), n, d, top, experts, hidden,
-                                      act_code, form, _p(tc_fault()), _stream()), lib)
+                                      act_code, form, int(weigh_input), _p(tc_fault()), _stream()), lib)
         return out
     if (grouped and n * top >= MOE_GROUPED_MIN_PAIRS and d % 32 == 0
             and hidden % 32 == 0):
@@ -1550,6 +1666,7 @@ def moe_experts(x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, w_
         _check(lib.tis_moe_grouped(_p(x), x.stride(0), _p(chosen), _p(weights), _p(w_gate_up), _p(w_down), _p(shared),
                                    shared.stride(0) if shared is not None else 0, _p(shared_gate), _p(out), _p(sorted_pair),
                                    _p(pair_place), _p(tile_expert), _p(hid), _p(y), n, d, top, experts, hidden, act_code,
-                                   form, _stream()), lib)
+                                   form, int(weigh_input), _stream()), lib)
         return out
-    return moe_down(moe_gate_up(x, chosen, w_gate_up, act, form), chosen, weights, w_down, shared, shared_gate)
+    hid = moe_gate_up(x, chosen, w_gate_up, act, form, weights if weigh_input else None)
+    return moe_down(hid, chosen, None if weigh_input else weights, w_down, shared, shared_gate)

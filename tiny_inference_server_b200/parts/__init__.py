@@ -3,8 +3,8 @@ their arrangement in a block, embedding and output head."""
 from .base import (BuildContext, FeedForward, KVSpec, LayerBinding, Mixer, Norm, Part, PositionEncoding,
                    StateSpec, WeightSpec)
 from .stream import ResidualStream
-from .norms import LayerNorm, RMSNormGrouped, RMSNormL2, RMSNormMeanEps, RMSNormOnePlus, RMSNormScalar
-from .positions import RotaryHalf, RotaryInterleaved, RotaryRescaled
+from .norms import LayerNorm, RMSNormGrouped, RMSNormL2, RMSNormMeanEps, RMSNormOnePlus, RMSNormScalar, StreamAsIs
+from .positions import RotaryBanded, RotaryHalf, RotaryInterleaved, RotaryRescaled
 from .attention import GqaAttention
 from .feed_forward import ActMLP, ClampedGLU, RoutedExperts, SwiGLU
 from .short_conv import CausalConv
@@ -18,6 +18,8 @@ from .gated_linear_attention import GatedLinearAttention
 from .sink_attention import TiedValueAttention
 from .normed_attention import NormedRotaryAttention
 from .state_space import SelectiveStateSpace
+from .selective_scan import SelectiveScan
+from .time_mix import TimeMix
 from .side_by_side import SideBySide
 from .block import Block
 from .embedding import Embedding, LMHead, PairHashEmbedding
@@ -28,4 +30,4 @@ __all__ = ["BuildContext", "FeedForward", "KVSpec", "LayerBinding", "Mixer", "No
            "RotaryRescaled", "RotaryHalf",
            "RotaryInterleaved", "GqaAttention", "SwiGLU", "Block", "Embedding", "LMHead", "RMSNormScalar", "ActMLP",
            "DifferentialAttention", "ForgetGateRecurrence", "GatedLinearAttention", "TiedValueAttention", "SelectiveStateSpace",
-           "SideBySide", "PairHashEmbedding", "RMSNormGrouped"]
+           "SideBySide", "PairHashEmbedding", "RMSNormGrouped", "RotaryBanded", "SelectiveScan", "StreamAsIs", "TimeMix"]

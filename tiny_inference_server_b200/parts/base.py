@@ -34,6 +34,7 @@ class KVSpec:
     lag: int = 0                      # the plane is filled this many positions behind the trunk
     k_dim: Optional[int] = None       # elements of a key row (default head_dim)
     v_dim: Optional[int] = None       # elements of a value row (default head_dim)
+    chunks: Tuple[int, ...] = ()      # not empty (and no window): the sizes of the chunks whose keys the plane's readers see
 
     @property
     def key_dim(self) -> int:
@@ -44,7 +45,7 @@ class KVSpec:
         return self.head_dim if self.v_dim is None else self.v_dim
 
     def group_key(self):
-        return (self.kv_heads, self.key_dim, self.value_dim, self.window)
+        return (self.kv_heads, self.key_dim, self.value_dim, self.window, self.chunks)
 
 
 @dataclass(frozen=True)

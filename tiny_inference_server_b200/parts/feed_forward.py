@@ -158,7 +158,8 @@ class RoutedExperts(FeedForward):
     ``scores`` ``"softmax"``: ``s`` is the softmax over all experts; ``group_score`` ``"best"``: a group is as strong as its
     largest choosing score; ``renorm`` False: the weights are the chosen ``s`` as they are; ``form``, ``shared_form`` (a
     ``kernels.ops.GateForm``): the gating of the experts and of the shared unit instead of silu; ``shared_gated`` False: the
-    shared unit is added as it is, and there is no ``shared.sg``.
+    shared unit is added as it is, and there is no ``shared.sg``; ``weigh_input``: an expert's weight multiplies its input,
+    ``unit(w h)``, instead of its output.
 
     Tensor names below the prefix: ``e<i>.gate, e<i>.up, e<i>.down``, ``router``, ``correction``, ``shared.gate,
     shared.up, shared.down, shared.sg`` (matrices stored (out, in)).  On the device the experts' matrices are stacked:
@@ -170,8 +171,10 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, hidden: int, experts: int, top: int, groups: int = 0, keep: int = 0,
                  shared_hidden: int = 0, prefix: str = "", scores: str = "sigmoid", correction: bool = True,
                  unit_act: Optional[str] = None, group_score: str = "two_best", renorm: bool = True,
-                 form: Optional[ops.GateForm] = None, shared_form: Optional[ops.GateForm] = None, shared_gated: bool = True):
+                 form: Optional[ops.GateForm] = None, shared_form: Optional[ops.GateForm] = None, shared_gated: bool = True,
+                 weigh_input: bool = False):
         super().__init__(prefix)
+        self.weigh_input = weigh_input
         if group_score not in ops.GROUP_SCORES:
             raise ValueError(f"group score {group_score!r}: known are {sorted(ops.GROUP_SCORES)}")
         self.group_score, self.renorm, self.shared_gated = group_score, renorm, shared_gated
@@ -237,7 +240,7 @@ class RoutedExperts(FeedForward):
                                                      group_score=self.group_score, renorm=self.renorm)
         shared = self.shared.forward(x, step) if self.shared is not None else None
         return ops.moe_experts(x, chosen, weights, self.w_gate_up, self.w_down, shared, shared_gate, act=self.unit_act,
-                               form=self.form)
+                               form=self.form, weigh_input=self.weigh_input)
 
 
 register_part("ffn", "swiglu", SwiGLU)

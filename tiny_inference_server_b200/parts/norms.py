@@ -53,15 +53,17 @@ class RMSNormL2(Norm):
 class RMSNormMeanEps(Norm):
     """``y = x / sqrt(mean(x^2) + eps) * (offset + w)`` in float32, eps inside the root.  ``offset`` 1: the
     stored tensor is the weight's distance from one; 0: it is the weight.  ``keep_f32``: the result is float32
-    whatever the compute dtype."""
+    whatever the compute dtype.  ``gain``: a constant that multiplies the result (a norm behind a sublayer whose updates
+    enter the stream scaled)."""
 
     def __init__(self, width: int, eps: float, prefix: str = "", weight_name: str = "weight", offset: float = 0.0,
-                 keep_f32: bool = False):
+                 keep_f32: bool = False, gain: float = 1.0):
         super().__init__(prefix)
         self.width = width
         self.eps = float(eps)
         self.weight_name = weight_name
         self.offset = float(offset)
+        self.gain = float(gain)
         self.keep_f32 = keep_f32                  # the result stays in 32-bit (a norm that makes the residual stream)
         self.scale: Optional[torch.Tensor] = None
         self.out_dtype = torch.float32
@@ -75,7 +77,7 @@ class RMSNormMeanEps(Norm):
 
     def load(self, tensors, ctx: BuildContext) -> None:
         w = tensors[self.prefix + self.weight_name].to(device=ctx.device, dtype=torch.float32)
-        self.scale = (w + self.offset).contiguous()
+        self.scale = ((w + self.offset) * self.gain).contiguous()
         self.out_dtype = torch.float32 if self.keep_f32 else ctx.dtype
 
     def add_norm(self, residual: torch.Tensor, delta: Optional[torch.Tensor], delta_norm=None) -> torch.Tensor:
@@ -171,6 +173,32 @@ class RMSNormGrouped(Norm):
         return values
 
 
+class StreamAsIs(Norm):
+    """No norm: the stream itself in the compute dtype, for sublayers that read it as it is (a block whose norms stand behind its
+    sublayers only).  The pending update, with the norm it passes, is added in the same kernel."""
+
+    def __init__(self, width: int, prefix: str = ""):
+        super().__init__(prefix)
+        self.width = width
+        self.ones: Optional[torch.Tensor] = None
+        self.out_dtype = torch.float32
+
+    @classmethod
+    def from_config(cls, cfg, prefix: str):
+        return cls(cfg.hidden_size, prefix=prefix)
+
+    def load(self, tensors, ctx: BuildContext) -> None:
+        self.ones = torch.ones(self.width, dtype=torch.float32, device=ctx.device)
+        self.out_dtype = ctx.dtype
+
+    def add_norm(self, residual: torch.Tensor, delta: Optional[torch.Tensor], delta_norm=None) -> torch.Tensor:
+        out = torch.empty(residual.shape, dtype=self.out_dtype, device=residual.device)
+        return ops.add_rmsnorm(residual, delta, self.ones, 0.0, out, kind="none", delta_norm=delta_norm)
+
+    def forward(self, residual: torch.Tensor) -> torch.Tensor:
+        return self.add_norm(residual, None)
+
+
 class LayerNorm(Norm):
     """``y = (x - mean) / sqrt(variance + eps) * w + b`` in float32, the variance being the mean of the squared deviations and
     eps inside the root.  Tensor names: ``weight_name`` and ``weight_name + ".b"``.  ``add_norm(residual, delta, delta_b=...)``
@@ -208,6 +236,7 @@ class LayerNorm(Norm):
         return self.add_norm(residual, None)
 
 
+register_part("norm", "stream_as_is", StreamAsIs)
 register_part("norm", "layer_norm", LayerNorm)
 register_part("norm", "rmsnorm_grouped", RMSNormGrouped)
 register_part("norm", "rmsnorm_l2", RMSNormL2)

@@ -113,6 +113,35 @@ class RotaryRescaled(RotaryHalf):
         return None
 
 
+class RotaryBanded(RotaryInterleaved):
+    """``RotaryInterleaved`` whose frequencies are slowed down by their wavelength, in three bands: with w = 2 pi / f, waves shorter
+    than ``original / high`` keep f, those longer than ``original / low`` turn with f / factor, and between them the two are
+    blended, ``(1 - s) f / factor + s f`` with ``s = (original / w - low) / (high - low)``.  ``scaling`` None: plain
+    frequencies.  The tables are formed in float64 on the host."""
+
+    def __init__(self, head_dim: int, theta: float, max_positions: int, scaling: Optional[dict] = None,
+                 rotary_dim: Optional[int] = None, prefix: str = ""):
+        super().__init__(head_dim, theta, max_positions, rotary_dim, prefix=prefix)
+        self.scaling = dict(scaling) if scaling else None
+
+    def frequencies(self) -> torch.Tensor:
+        import math
+        i = torch.arange(0, self.rotary_dim // 2, dtype=torch.float64)
+        f = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / self.rotary_dim)
+        if not self.scaling:
+            return f
+        factor, low, high, original = (float(self.scaling[k]) for k in ("factor", "low", "high", "original"))
+        turns = original * f / (2.0 * math.pi)              # of a wave over the original context
+        s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+        blended = (1.0 - s) * f / factor + s * f
+        return torch.where(turns > high, f, torch.where(turns < low, f / factor, blended))
+
+    def tables(self):
+        ang = torch.outer(torch.arange(self.max_positions, dtype=torch.float64), self.frequencies())
+        return torch.cos(ang).to(torch.float32), torch.sin(ang).to(torch.float32)
+
+
+register_part("position", "rope_banded", RotaryBanded)
 register_part("position", "rope_half", RotaryHalf)
 register_part("position", "rope_rescaled", RotaryRescaled)
 register_part("position", "rope_interleaved", RotaryInterleaved)
