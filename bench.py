@@ -725,6 +725,86 @@ def reference_arm(args):
         return unavailable(f"upstream's code did not run here: {type(e).__name__}: {e}")
 
 
+def tazadra_config(width, heads, kv_heads, ffn, vocab, layers, chunk=1024, experts=16, top=4):
+    """A Tazadra model with the layer sizes of a member of the GQA family: per four layers one selective scan (inner 2 width, 16
+    states a channel, steps of rank width / 16), two time mixers (heads of 128) and one attention in chunks with bounded
+    scores, every other attention reading the keys and values of the one before it; feed-forwards in turn dense (clamped,
+    ffn hidden elements) and routed (``top`` of ``experts`` units that together hold as many weights a token)."""
+    fe = max(64, ffn // top // 64 * 64)
+    scan = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+    mix = {"heads": heads, "dim": 128, "decay_rank": 64}
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0, "mask": {"size": chunk},
+            "rot": {"base": 5e5, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    dense = {"kind": "dense", "ff": ffn, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": fe}, "router": {"experts": experts, "top": top}}
+    kinds = [("mamba1", scan), ("wkv", mix), ("attention", attn), ("wkv", mix)]
+    made, owner = [], None
+    for i in range(layers):
+        kind, mixer = kinds[i % 4][0], json.loads(json.dumps(kinds[i % 4][1]))
+        if kind == "attention":
+            if owner is not None:
+                mixer["kv_from"], owner = owner, None
+            else:
+                owner = i
+        made.append({"type": kind, "mixer": mixer, "mlp": json.loads(json.dumps(moe if i % 2 else dense))})
+    return dict(architecture="Tazadra", vocab=vocab, width=width, norm={"eps": 1e-6}, residual_mult=0.7, logit_softcap=40.0,
+                max_context=8192, layers=made)
+
+
+def compare_tazadra(args):
+    """``--compare tazadra``: prefill and decode of the Tazadra architecture beside the Kubolorn architecture (the closest earlier
+    one: a selective state space, a recurrence with gates per key channel, attention with a keyless term, routed experts), the
+    Lomutar architecture (the closest for its attention) and the rotary GQA model at equal layer sizes, and its kernels beside
+    the like kernels of those.  One JSON line; the default run is untouched."""
+    import gc
+    import types
+    import torch
+    from tiny_inference_server_b200.kernels import microbench, ops
+    from tiny_inference_server_b200.sampling import Sampler
+    pk = peaks()
+    count_ops = lambda: ops.launches  # noqa: E731
+    window, ctx, layers = 1024, 4096, 8
+    result = {"compare": "tazadra", "dtype": "bf16", "data": "synthetic", "layers": layers, "context": ctx, "window": window,
+              "peaks": pk, "sizes": {}}
+    for name in [x for x in args.compare_sizes.split(",") if x]:
+        base = SIZES[name][0]
+        twin = dict(base, num_layers=layers, num_mtp_heads=0, sliding_window=window, max_context=8192, tie_word_embeddings=False)
+        size = (base["hidden_size"], base["num_heads"], base["num_kv_heads"], base["ffn_hidden"], base["vocab_size"], layers)
+        point = {}
+        for label, cfg_dict in (("tazadra", tazadra_config(*size, chunk=window)), ("kubolorn", kubolorn_config(*size)),
+                                ("lomutar", lomutar_config(*size, window=window)), ("gqa", twin)):
+            runner = None
+            try:
+                _, runner = build_runner(cfg_dict, ctx, 8, mtp=False)
+                steps = max(8, args.steps // 2)
+                r = {}
+                for b in (1, 8):
+                    ms, launches = decode_run(runner, b, ctx - steps - args.warmup - 2, steps, args.warmup, Sampler, count_ops)
+                    r[f"decode_b{b}_tok_s"] = round(b / (ms * 1e-3), 1)
+                    r[f"decode_b{b}_ms"] = round(ms, 4)
+                    r[f"decode_b{b}_launches"] = round(launches, 1)
+                best, first = prefill_run(runner, PREFILL_TOKENS, reps=2)
+                r["prefill_tok_s"] = round(PREFILL_TOKENS / (best * 1e-3), 1)
+                r["prefill_ms"] = round(best, 3)
+                r["prefill_first_run_ms"] = round(first, 3)
+                point[label] = r
+            except Exception as e:                       # noqa: BLE001
+                point[label] = {"error": f"{type(e).__name__}: {e}"[:300]}
+            del runner
+            gc.collect()
+            torch.cuda.empty_cache()
+        margs = types.SimpleNamespace(width=base["hidden_size"], ffn=base["ffn_hidden"], heads=base["num_heads"],
+                                      kv_heads=base["num_kv_heads"], head_dim=128, page_size=PAGE, tokens=PREFILL_TOKENS, batch=8,
+                                      context=ctx, window=window, experts=16, top=4)
+        try:
+            point["kernels"] = microbench.scan_mix_chunked(margs)
+        except Exception as e:                           # noqa: BLE001
+            point["kernels"] = {"error": f"{type(e).__name__}: {e}"[:300]}
+        result["sizes"][name] = point
+    print(json.dumps(result))
+    return 0
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -735,7 +815,7 @@ def main(argv=None):
     ap.add_argument("--impl", default="engine", choices=["engine", "reference"])
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 / 64, other contexts, MTP heads and prefill")
     ap.add_argument("--sizes", default="3b,8b", help="larger members of the family to measure too (3b, 8b; '' = none)")
-    ap.add_argument("--compare", default=None, choices=["kefisun", "mizidra", "biruvik", "kubolorn", "lomutar"],
+    ap.add_argument("--compare", default=None, choices=["kefisun", "mizidra", "biruvik", "kubolorn", "lomutar", "tazadra"],
                     help="instead of the default run: another architecture beside the GQA model at equal layer sizes")
     ap.add_argument("--compare-sizes", default="0.9b,3b", help="with --compare: whose layer sizes (0.9b, 3b, 8b)")
     args = ap.parse_args(argv)
@@ -750,6 +830,9 @@ def main(argv=None):
     if args.compare == "lomutar":
         args.warmup = max(args.warmup, 3)
         return compare_lomutar(args)
+    if args.compare == "tazadra":
+        args.warmup = max(args.warmup, 3)
+        return compare_tazadra(args)
     if args.compare == "kubolorn":
         return compare_kubolorn(args)
     if args.compare == "biruvik":

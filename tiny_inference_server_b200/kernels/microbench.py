@@ -16,6 +16,9 @@
         sublayer, each beside the like kernel of an earlier model)
     python -m tiny_inference_server_b200.kernels.microbench normed-shared-clamped   (attention with normed heads and a
         sink, layer norm with two updates, gelu gating, clamped experts, each beside the like kernel of an earlier model)
+    python -m tiny_inference_server_b200.kernels.microbench scan-mix-chunked   (selective scan, time mixer with its token
+        shift and side-by-side products, attention in chunks with bounded scores and head gates, norms behind sublayers,
+        experts with weighed inputs, each beside the like kernel of an earlier model)
     python -m tiny_inference_server_b200.kernels.microbench all
 
 ``--reps N --no-timing`` launches the kernel N times and exits (a profiler attaches to that);
@@ -854,6 +857,188 @@ def normed_shared_clamped(args):
     return out
 
 
+def scan_mix_chunked(args):
+    """The kernels of a selective scan with a decay per channel and state, of a time mixer (token shift, side-by-side products,
+    recurrence with a bonus), of attention in chunks with bounded scores, head gates and heads normed as a whole, of norms that
+    stand behind sublayers only, of the clamped gated product and of experts whose inputs are weighed, each beside the kernel
+    of an earlier architecture of this engine that does the like work at equal sizes: Kubolorn's state space and gated linear
+    attention, Lomutar's attention, head norms and router, Biruvik's norm behind a sublayer, Kefisun's short convolution,
+    Mizidra's experts.  Returns {name: {us, rate, unit, like_us, like_rate}}."""
+    from .attention_plan import infer_tiles
+    dev = "cuda"
+    d, F, H, G, hd, page = args.width, args.ffn, args.heads, args.kv_heads, args.head_dim, args.page_size
+    n, B, ctx, W, E, top = args.tokens, args.batch, args.context, args.window, args.experts, args.top
+    bf, i32 = dict(device=dev, dtype=torch.bfloat16), dict(device=dev, dtype=torch.int32)
+    fault, out, bufs = torch.zeros(4, **i32), {}, 4
+
+    def put(name, us, work, unit, like_us, like_work=None):
+        div, digits = (1e3, 1) if unit in ("GB/s", "Gupdates/s") else (1e6, 1)
+        like_work = work if like_work is None else like_work
+        out[name] = {"us": round(us, 2), "rate": round(work / us / div, digits), "unit": unit, "like_us": round(like_us, 2),
+                     "like_rate": round(like_work / like_us / div, digits)}
+        e = out[name]
+        print(f"{name:58s} {e['us']:9.2f} us {e['rate']:9.1f} {unit}   like kernel {e['like_us']:9.2f} us {e['like_rate']:9.1f} {unit}",
+              file=sys.stderr)
+
+    pos, slot, last = torch.arange(n, **i32), torch.zeros(n, **i32), torch.full((n,), n - 1, **i32)
+    slot_b = torch.arange(B, **i32)
+    one, each = (torch.zeros(1, **i32), 1), (slot_b, B)
+    # ---- the selective scan (inner 2 d, 16 states a channel; skip and gate inside) beside the scan of a state space (heads of
+    # hd, a state of hd x hd each, as many channels) and the skip, gate and norm behind it.  Work: updates of a state number.
+    inner, N = 2 * d, 16
+    heads = inner // hd
+    xs = [torch.randn(n, inner, **bf) for _ in range(bufs)]
+    zs = [torch.randn(n, inner, **bf) for _ in range(bufs)]
+    dts = [torch.randn(n, inner, device=dev) - 3.0 for _ in range(bufs)]
+    bc = torch.randn(n, 2 * N, **bf)
+    bias, skip = torch.zeros(inner, device=dev), torch.ones(inner, device=dev)
+    a_log = torch.rand(inner, N, device=dev)
+    st = torch.zeros(B, inner * N, device=dev)
+    od = torch.empty(n, inner, **bf)
+    gs = max(1, heads // 4)
+    while heads % gs:
+        gs -= 1
+    cbx = [torch.randn(n, 2 * gs * hd + inner, **bf) for _ in range(2)]
+    dt2, al2, db2 = torch.randn(n, heads, **bf), torch.zeros(heads, device=dev), torch.zeros(heads, device=dev)
+    st2 = torch.zeros(B, heads * hd * hd, device=dev)
+    skip2, nw2 = torch.ones(heads, device=dev), torch.ones(inner, device=dev)
+
+    def space(i, rows, sl, la, seg):
+        raw = ops.state_space_scan(cbx[i % 2][:rows], dt2[:rows], al2, db2, st2, sl, la, heads, gs, hd, hd, requests=seg[1], segments=seg)
+        ops.skip_gate_group_norm(raw, cbx[i % 2][:rows, 2 * gs * hd:], skip2, zs[i % bufs][:rows], nw2, 1, 1e-6, od[:rows], sl, heads, hd)
+
+    for rows, sl, la, seg in ((n, slot, last, one), (B, slot_b, slot_b, each)):
+        t_new = _graph_time(lambda i: ops.selective_scan(xs[i % bufs][:rows], dts[i % bufs][:rows], bias, a_log, bc[:rows, :N],
+                                                         bc[:rows, N:], skip, zs[i % bufs][:rows], st, od[:rows], sl, la,
+                                                         segments=seg), 8)
+        t_like = _graph_time(lambda i: space(i, rows, sl, la, seg), 8)
+        put(f"selective scan, skip, gate, {rows} rows of {inner} x {N}", t_new, 1.0 * rows * inner * N, "Gupdates/s", t_like,
+            1.0 * rows * inner * hd)
+        out[f"selective scan, skip, gate, {rows} rows of {inner} x {N}"]["gb_s"] = round(
+            (rows * inner * 10 + (2 * 4 * inner * N * seg[1])) / t_new / 1e3, 1)
+    del xs, zs, dts, cbx
+    # ---- the time mixer: its recurrence beside gated linear attention's
+    nv = H * hd
+    rows4 = [torch.randn(n, 4 * nv, **bf) for _ in range(2)]
+    win = torch.randn(n, nv, **bf)
+    u, wb, nwf = torch.rand(nv, device=dev), torch.full((nv,), -2.0, device=dev), torch.ones(nv, device=dev)
+    power, ab, nwh = torch.full((H,), 1 / 8, device=dev), torch.full((nv,), 3.0, device=dev), torch.ones(hd, device=dev)
+    stm = torch.zeros(B, H * hd * hd + d, device=dev)
+    om = torch.empty(n, nv, **bf)
+    for rows, sl, la, seg in ((n, slot, last, one), (B, slot_b, slot_b, each)):
+        stm.zero_()
+        t_new = _graph_time(lambda i: ops.time_mix(rows4[i % 2][:rows], win[:rows], u, wb, nwf, 1e-6, stm, om[:rows], sl, la, H, hd,
+                                                   requests=seg[1], segments=seg), 4)
+        stm.zero_()
+        t_like = _graph_time(lambda i: ops.gated_linear_attention(rows4[i % 2][:rows, :3 * nv], win[:rows], power, ab,
+                                                                  rows4[i % 2][:rows, 3 * nv:], nwh, 1e-6, 1.0, stm, om[:rows], sl, la,
+                                                                  H, hd, hd, requests=seg[1], segments=seg), 4)
+        work, unit = (4.0 * rows * H * hd * hd, "TFLOP/s") if rows == n else (8.0 * rows * H * hd * hd, "GB/s")
+        put(f"recurrence with a bonus, {rows} rows", t_new, work, unit, t_like)
+    # the token shift (five mixes) beside the short convolution of four taps
+    x = [torch.randn(n, d, **bf) for _ in range(bufs)]
+    mu = torch.rand(5, d, device=dev)
+    wc, stc, oc = torch.randn(4, d, device=dev), torch.zeros(B, 3 * d, device=dev), torch.empty(n, d, **bf)
+    for rows, sl, la in ((n, slot, last), (B, slot_b, slot_b)):
+        t_new = _graph_time(lambda i: ops.token_shift(x[i % bufs][:rows], mu, stm[:, H * hd * hd:], sl, la), 12)
+        t_like = _graph_time(lambda i: ops.causal_conv(x[i % bufs][:rows], wc, stc, oc[:rows], sl, la, residual=True), 12)
+        put(f"token shift, five mixes, {rows} rows", t_new, rows * d * 12, "GB/s", t_like, rows * d * 4)
+    # its products side by side, beside one product of as many columns
+    rank = 64
+    w4 = [torch.randn(4, d, nv, **bf) * 0.02 for _ in range(2)]
+    wl = torch.randn(d, rank, **bf) * 0.02
+    w1 = [torch.randn(d, 4 * nv + rank, **bf) * 0.02 for _ in range(2)]
+    mixes = torch.randn(n, 5, d, **bf)
+    for rows in (B, n):
+        work, unit = (d * (4 * nv + rank) * 2, "GB/s") if rows == B else (2.0 * rows * d * (4 * nv + rank), "TFLOP/s")
+        t_new = _graph_time(lambda i: ops.gemm_side_by_side(mixes[:rows], w4[i % 2], wl, act="tanh"), 12)
+        t_like = _graph_time(lambda i: ops.gemm(x[i % bufs][:rows], w1[i % 2]), 12)
+        put(f"products side by side, {rows} rows", t_new, work, unit, t_like)
+    del w4, w1, mixes
+    # ---- attention in chunks, bounded scores, head gates, a keyless term, beside the window with a keyless term
+    num_pages = (n + page - 1) // page
+    nq, nk = H * hd, G * hd
+    planes = [torch.randn(num_pages, 2, G, page, hd, **bf) for _ in range(2)]
+    table = torch.arange(num_pages, **i32).reshape(1, num_pages).contiguous()
+    qkv = [torch.randn(n, nq + 2 * nk, **bf) for _ in range(bufs)]
+    gates = torch.randn(n, H, **bf)
+    o, sink = torch.empty(n, nq, **bf), torch.zeros(H, device=dev)
+    step = _Step(infer_tiles(pos, slot, H // G), n - 1)
+    step.decode_only, step.min_position = False, 0
+    for size in (W, None):
+        chunk_flops = 4.0 * nq * sum(p % size + 1 if size else p + 1 for p in range(n))
+        win_flops = 4.0 * nq * sum(min(p + 1, size) if size else p + 1 for p in range(n))
+        t_new = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs], o, planes[i % 2], table, pos, slot, H, G, hd, page, size, fault,
+                                                          step, sink=sink, chunked=True, softcap=30.0, gate=gates), 10)
+        t_like = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs], o, planes[i % 2], table, pos, slot, H, G, hd, page, size, fault,
+                                                           step, sink=sink), 10)
+        put(f"bounded, gated attention, {n} rows, " + (f"chunks of {size}" if size else "every key"), t_new, chunk_flops, "TFLOP/s",
+            t_like, win_flops)
+    half = hd // 2
+    cos, sin = torch.ones(ctx + n, half, device=dev), torch.zeros(ctx + n, half, device=dev)
+    ww = torch.ones((H + G) * hd, device=dev)
+    for rows, sl, ps in ((n, slot, pos), (B, slot_b, torch.full((B,), page - 1, **i32))):
+        plane = torch.zeros(max(num_pages, B), 2, G, page, hd, **bf)
+        tb = table if rows == n else torch.arange(B, **i32).reshape(B, 1).contiguous()
+        t_new = _graph_time(lambda i: ops.rotate_norm_store(qkv[i % bufs][:rows], H, G, hd, hd, cos, sin, True, False, 1e-6, plane[:, 0],
+                                                            plane[:, 1], tb, ps, sl, page, fault, permuted=True, whole_weight=ww), 12)
+        t_like = _graph_time(lambda i: ops.rotate_norm_store(qkv[i % bufs][:rows], H, G, hd, hd, cos, sin, True, True, 1e-6, plane[:, 0],
+                                                             plane[:, 1], tb, ps, sl, page, fault, permuted=True), 12)
+        put(f"norm of all heads, rotation, cache write, {rows} rows", t_new, rows * (nq + 2 * nk) * 4, "GB/s", t_like)
+    pages_per = (ctx + page - 1) // page
+    n_planes = max(2, min(12, (300 << 20) // max(1, B * ctx * 2 * nk * 2)))
+    planes = [torch.randn(B * pages_per, 2, G, page, hd, **bf) for _ in range(n_planes)]
+    dtable = torch.arange(B * pages_per, **i32).reshape(B, pages_per).contiguous()
+    pos_b = torch.full((B,), ctx - 1, **i32)
+    dstep = _Step(infer_tiles(pos_b, slot_b, H // G), ctx - 1)
+    for size in (W, None):
+        kv_bytes = B * min(size or ctx, ctx) * 2 * nk * 2
+        t_new = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs][:B], o[:B], planes[i % n_planes], dtable, pos_b, slot_b, H, G, hd,
+                                                          page, size, fault, dstep, sink=sink, chunked=True, softcap=30.0, gate=gates[:B]))
+        t_like = _graph_time(lambda i: ops.paged_attention(qkv[i % bufs][:B], o[:B], planes[i % n_planes], dtable, pos_b, slot_b, H, G, hd,
+                                                           page, size, fault, dstep, sink=sink))
+        put(f"bounded, gated attention, {B} decode rows, " + (f"chunks of {size}" if size else f"all of {ctx}"), t_new, kv_bytes, "GB/s",
+            t_like)
+    del planes, qkv
+    # ---- a norm behind a sublayer, and the stream as it is, beside the same with a norm in front of the next sublayer
+    res = [torch.randn(n, d, device=dev) for _ in range(bufs)]
+    da, y, w = [torch.randn(n, d, **bf) for _ in range(bufs)], torch.empty(n, d, **bf), torch.ones(d, device=dev)
+    for rows in (n, B):
+        t_new = _graph_time(lambda i: ops.add_rmsnorm(res[i % bufs][:rows], da[i % bufs][:rows], w, 0.0, y[:rows], kind="none",
+                                                      delta_norm=(w, 1e-6, "mean_eps")), 12)
+        t_like = _graph_time(lambda i: ops.add_rmsnorm(res[i % bufs][:rows], da[i % bufs][:rows], w, 1e-6, y[:rows], kind="mean_eps",
+                                                       delta_norm=(w, 1e-6, "mean_eps")), 12)
+        put(f"norm behind a sublayer, {rows} rows", t_new, rows * d * 12, "GB/s", t_like)
+    # ---- gate and up with the clamped gating beside silu's
+    wgu = [torch.randn(d, 2 * F, **bf) * 0.02 for _ in range(4)]
+    form = ops.gate_clamped(7.0)
+    for rows in (B, n):
+        work, unit = (2 * d * F * 2, "GB/s") if rows == B else (4.0 * rows * d * F, "TFLOP/s")
+        t_new = _graph_time(lambda i: ops.gemm_swiglu(x[i % bufs][:rows], wgu[i % 4], F, 32, form), 8)
+        t_like = _graph_time(lambda i: ops.gemm_swiglu(x[i % bufs][:rows], wgu[i % 4], F, 32), 8)
+        put(f"gate, up, clamped gating, {rows} rows", t_new, work, unit, t_like)
+    del wgu
+    # ---- router and experts, weights on the inputs, beside the weights on the outputs
+    fe = max(64, F // top // 64 * 64)
+    wr = torch.randn(E, d, device=dev) * d ** -0.5
+    corr = torch.zeros(E, device=dev)
+    for rows in (n, B):
+        t_new = _graph_time(lambda i: ops.moe_route(x[i % bufs][:rows], wr, None, None, 0, 0, top, renorm=False), 12)
+        t_like = _graph_time(lambda i: ops.moe_route(x[i % bufs][:rows], wr, corr, None, 0, 0, top), 12)
+        put(f"router, sigmoid scores as they are, {rows} rows", t_new, rows * d * 2 + E * d * 4, "GB/s", t_like)
+    gu = [torch.randn(E, 2, fe, d, **bf) * 0.02 for _ in range(2)]
+    dn = [torch.randn(E, d, fe, **bf) * 0.02 for _ in range(2)]
+    chosen, weights, _ = ops.moe_route(x[0], wr, None, None, 0, 0, top, renorm=False)
+    used = len(set(chosen[:B].flatten().tolist()))
+    for rows in (n, B):
+        work, unit = (6.0 * rows * top * d * fe, "TFLOP/s") if rows == n else (used * 3 * d * fe * 2, "GB/s")
+        t_new = _graph_time(lambda i: ops.moe_experts(x[0][:rows], chosen[:rows], weights[:rows], gu[i % 2], dn[i % 2], None, None,
+                                                      weigh_input=True), 8)
+        t_like = _graph_time(lambda i: ops.moe_experts(x[0][:rows], chosen[:rows], weights[:rows], gu[i % 2], dn[i % 2], None, None), 8)
+        put(f"experts with weighed inputs, {rows} rows", t_new, work, unit, t_like)
+    return out
+
+
 def sampling(args):
     """The sampling kernel at ``--rows`` rows of ``--vocab`` logits, for the kinds of setting a row can have."""
     dev = "cuda"
@@ -1057,7 +1242,7 @@ def timeline(args):
 def main(argv=None):
     ap = argparse.ArgumentParser(prog="microbench", description=__doc__.split("\n\n")[0])
     ap.add_argument("what", choices=["attention", "attention-prefill", "rowwise", "gemm", "prefill", "sampling", "timeline",
-                                     "seqmix", "latent-linear-routed", "differential-latent-forget", "gated-space-tied", "normed-shared-clamped", "all"])
+                                     "seqmix", "latent-linear-routed", "differential-latent-forget", "gated-space-tied", "normed-shared-clamped", "scan-mix-chunked", "all"])
     ap.add_argument("--rank", type=int, default=128, help="latent-linear-routed: compressed elements a token")
     ap.add_argument("--rot", type=int, default=64, help="latent-linear-routed: rotated elements a token")
     ap.add_argument("--experts", type=int, default=16)
@@ -1112,6 +1297,8 @@ def main(argv=None):
         gated_space_tied(args)
     if args.what in ("normed-shared-clamped", "all"):
         normed_shared_clamped(args)
+    if args.what in ("scan-mix-chunked", "all"):
+        scan_mix_chunked(args)
     return 0
 
 
