@@ -176,69 +176,103 @@ rotate_norm_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__
 }
 
 // The other order: queries and keys are normed first, each over all of its heads at once and with weights `w` (H * dim for the
-// queries, then G * dim for the keys), and then rotated, neighbouring elements paired.  Whole 16-byte vectors, a CTA a row,
-// VPT vectors of the row a thread.
+// queries, then G * dim for the keys), and then rotated, neighbouring elements paired.  Whole 16-byte vectors, a CTA takes
+// `rows` rows one after the other, VPT vectors of a row a thread, whose weights stay in registers.  What does not come from the
+// kernel before (weights, cosines and sines, block table) is loaded before the wait for it.
 template <typename T, int VPT>
 __global__ void __launch_bounds__(256)
 norm_rotate_vec_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__ v_pages, const float* __restrict__ w,
-                       const RotateNorm p) {
+                       const RotateNorm p, int rows) {
     constexpr int N = Vec16<T>::N;
-    __shared__ float red[33];
+    __shared__ float red[2][8];
     pdl_launch_dependents();
-    const int r = blockIdx.x, tid = threadIdx.x;
-    const int slot = p.row_slot[r];
-    if (slot < 0) return;
-    const int pos = p.positions[r];
-    const int page = p.G > 0 ? page_of(p, slot, pos, tid == 0) : -1;
-    const int in_page = pos % p.page_size;
-    const float* ct = p.cos_t + (size_t)pos * (p.rot >> 1);
-    const float* st = p.sin_t + (size_t)pos * (p.rot >> 1);
-    const int nq = p.H * p.dim, nk = p.G * p.dim, nv = (nq + nk) / N;
-    pdl_wait();
-    T* row = qkv + (size_t)r * p.ld;
-    float v[VPT][N];
-    float sq = 0.f, sk = 0.f;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nq = p.H * p.dim, nk = p.G * p.dim, total = nq + nk;
+    float wv[VPT][N];
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
         const int e = (tid + k * 256) * N;
-        if (e < nv * N) {
-            Vec16<T>::load(row + e, v[k]);
-            float s = 0.f;
+        if (e < total) {
 #pragma unroll
-            for (int j = 0; j < N; ++j) s = fmaf(v[k][j], v[k][j], s);
-            if (e < nq) sq += s; else sk += s;
+            for (int j = 0; j < N; j += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(w + e + j);
+                wv[k][j] = x.x; wv[k][j + 1] = x.y; wv[k][j + 2] = x.z; wv[k][j + 3] = x.w;
+            }
         }
     }
-    const float fq = 1.f / sqrtf(block_sum(sq, red) / (float)nq + p.eps);
-    const float fk = nk > 0 ? 1.f / sqrtf(block_sum(sk, red) / (float)nk + p.eps) : 0.f;
+    bool waited = false;
+    const int r_end = min(p.n, (int)(blockIdx.x + 1) * rows);
+    for (int r = blockIdx.x * rows; r < r_end; ++r) {
+        const int slot = p.row_slot[r];
+        if (slot < 0) continue;                               // (the same for all threads)
+        const int pos = p.positions[r];
+        const int page = p.G > 0 ? page_of(p, slot, pos, tid == 0) : -1;
+        const int in_page = pos % p.page_size;
+        const float* ct = p.cos_t + (size_t)pos * (p.rot >> 1);
+        const float* st = p.sin_t + (size_t)pos * (p.rot >> 1);
+        float cs[VPT][N / 2], sn[VPT][N / 2];
 #pragma unroll
-    for (int k = 0; k < VPT; ++k) {
-        const int e = (tid + k * 256) * N;
-        if (e >= nv * N || (e >= nq && page < 0)) continue;
-        const float f = e < nq ? fq : fk;
-        const int hh = e / p.dim, i = e - hh * p.dim;
+        for (int k = 0; k < VPT; ++k) {
+            const int i = ((tid + k * 256) * N) % p.dim;
 #pragma unroll
-        for (int j = 0; j < N; ++j) v[k][j] *= f * w[e + j];
-#pragma unroll
-        for (int j = 0; j < N / 2; ++j)
-            if (i + 2 * j < p.rot) {
-                const float c = ct[(i >> 1) + j], s = st[(i >> 1) + j];
-                const float a = v[k][2 * j], b = v[k][2 * j + 1];
-                v[k][2 * j] = a * c - b * s;
-                v[k][2 * j + 1] = b * c + a * s;
+            for (int j = 0; j < N / 2; ++j) {
+                const bool turns = (tid + k * 256) * N < total && i + 2 * j < p.rot;
+                cs[k][j] = turns ? ct[(i >> 1) + j] : 1.f;
+                sn[k][j] = turns ? st[(i >> 1) + j] : 0.f;
             }
-        if (e < nq) Vec16<T>::store(row + e, v[k]);
-        else
-            Vec16<T>::store(k_pages + (size_t)page * p.k_page_stride + (size_t)(hh - p.H) * p.k_head_stride + (size_t)in_page * p.dim +
-                            (p.permuted ? cache_chunk(i / N, pos, p.dim / N) * N : i), v[k]);
-    }
-    if (page < 0) return;
-    const T* vals = row + nq + nk;
-    const int nch = p.v_dim / N;
-    for (int idx = tid; idx < p.G * nch; idx += 256) {
-        const int g = idx / nch, c = idx - g * nch;
-        *reinterpret_cast<uint4*>(v_pages + (size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim +
-                                  (p.permuted ? cache_chunk(c, pos, nch) : c) * N) = *reinterpret_cast<const uint4*>(vals + idx * N);
+        }
+        if (!waited) { pdl_wait(); waited = true; }
+        T* row = qkv + (size_t)r * p.ld;
+        float v[VPT][N];
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) {
+            const int e = (tid + k * 256) * N;
+            if (e < total) {
+                Vec16<T>::load(row + e, v[k]);
+                float s = 0.f;
+#pragma unroll
+                for (int j = 0; j < N; ++j) s = fmaf(v[k][j], v[k][j], s);
+                if (e < nq) sq += s; else sk += s;
+            }
+        }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        __syncthreads();                                      // the sums of the row before have been read
+        if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
+        const float fq = 1.f / sqrtf(sq / (float)nq + p.eps);
+        const float fk = nk > 0 ? 1.f / sqrtf(sk / (float)nk + p.eps) : 0.f;
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) {
+            const int e = (tid + k * 256) * N;
+            if (e >= total || (e >= nq && page < 0)) continue;
+            const float f = e < nq ? fq : fk;
+            const int hh = e / p.dim, i = e - hh * p.dim;
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[k][j] *= f * wv[k][j];
+#pragma unroll
+            for (int j = 0; j < N / 2; ++j) {
+                const float a = v[k][2 * j], b = v[k][2 * j + 1];
+                v[k][2 * j] = a * cs[k][j] - b * sn[k][j];
+                v[k][2 * j + 1] = b * cs[k][j] + a * sn[k][j];
+            }
+            if (e < nq) Vec16<T>::store(row + e, v[k]);
+            else
+                Vec16<T>::store(k_pages + (size_t)page * p.k_page_stride + (size_t)(hh - p.H) * p.k_head_stride + (size_t)in_page * p.dim +
+                                (p.permuted ? cache_chunk(i / N, pos, p.dim / N) * N : i), v[k]);
+        }
+        if (page < 0) continue;
+        const T* vals = row + total;
+        const int nch = p.v_dim / N;
+        for (int idx = tid; idx < p.G * nch; idx += 256) {
+            const int g = idx / nch, c = idx - g * nch;
+            *reinterpret_cast<uint4*>(v_pages + (size_t)page * p.v_page_stride + (size_t)g * p.v_head_stride + (size_t)in_page * p.v_dim +
+                                      (p.permuted ? cache_chunk(c, pos, nch) : c) * N) = *reinterpret_cast<const uint4*>(vals + idx * N);
+        }
     }
 }
 
@@ -302,11 +336,14 @@ norm_rotate_kernel(T* __restrict__ qkv, T* __restrict__ k_pages, T* __restrict__
 template <typename T>
 void launch_norm_rotate(T* qkv, T* k_pages, T* v_pages, const float* w, const RotateNorm& p, bool vec, cudaStream_t stream) {
     const int per = ((p.H + p.G) * p.dim / Vec16<T>::N + 255) / 256;
-    if (!vec || per > 8) tis_launch(norm_rotate_kernel<T>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
-    else if (per <= 1) tis_launch(norm_rotate_vec_kernel<T, 1>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
-    else if (per <= 2) tis_launch(norm_rotate_vec_kernel<T, 2>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
-    else if (per <= 4) tis_launch(norm_rotate_vec_kernel<T, 4>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
-    else tis_launch(norm_rotate_vec_kernel<T, 8>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    // rows a CTA takes: enough CTAs for four on every SM, a thread's weights loaded once for all of its rows
+    const int rows = p.n >= 2 * 4 * 148 ? (p.n / (4 * 148) < 8 ? p.n / (4 * 148) : 8) : 1;
+    const dim3 grid((p.n + rows - 1) / rows);
+    if (!vec || per > 8 || (uintptr_t)w % 16) tis_launch(norm_rotate_kernel<T>, dim3(p.n), dim3(256), 0, stream, qkv, k_pages, v_pages, w, p);
+    else if (per <= 1) tis_launch(norm_rotate_vec_kernel<T, 1>, grid, dim3(256), 0, stream, qkv, k_pages, v_pages, w, p, rows);
+    else if (per <= 2) tis_launch(norm_rotate_vec_kernel<T, 2>, grid, dim3(256), 0, stream, qkv, k_pages, v_pages, w, p, rows);
+    else if (per <= 4) tis_launch(norm_rotate_vec_kernel<T, 4>, grid, dim3(256), 0, stream, qkv, k_pages, v_pages, w, p, rows);
+    else tis_launch(norm_rotate_vec_kernel<T, 8>, grid, dim3(256), 0, stream, qkv, k_pages, v_pages, w, p, rows);
 }
 
 template <typename T, int LPH, int VPL>

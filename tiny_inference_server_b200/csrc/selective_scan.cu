@@ -17,7 +17,19 @@ namespace {
 constexpr int SCAN_THREADS = 128;
 constexpr int SCAN_ROWS = 32;          // rows of a chunk
 
-__device__ __forceinline__ float scan_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+// softplus and x * sigmoid(x): the exact functions for 32-bit activations.  Otherwise the fast exponential and logarithm, and
+// for small e the series log(1 + e) = e - e^2 / 2 + e^3 / 3 - .. (the logarithm of a number next to 1 would lose its digits):
+// relative errors below 1e-5.
+template <typename T> __device__ __forceinline__ float scan_softplus(float x);
+template <> __device__ __forceinline__ float scan_softplus<float>(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+template <> __device__ __forceinline__ float scan_softplus<bf16>(float x) {
+    const float e = __expf(fminf(x, 20.f));
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 1.f / 3.f), -0.5f), 1.f);
+    return x > 20.f ? x : (e < 0.03125f ? series : __logf(1.f + e));
+}
+template <typename T> __device__ __forceinline__ float scan_silu(float x);
+template <> __device__ __forceinline__ float scan_silu<float>(float x) { return x / (1.f + expf(-x)); }
+template <> __device__ __forceinline__ float scan_silu<bf16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
 // 2^x: exact to the last bits for 32-bit activations, the fast form otherwise
 template <typename T> __device__ __forceinline__ float scan_exp2(float x);
@@ -26,6 +38,21 @@ template <> __device__ __forceinline__ float scan_exp2<bf16>(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
+}
+
+// Two multiply-adds (multiplications) in one instruction: neighbouring states of a lane.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("{\n.reg .b64 a, b, c, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmov.b64 c, {%6, %7};\nfma.rn.f32x2 d, a, b, c;\n"
+        "mov.b64 {%0, %1}, d;\n}\n"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+    return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("{\n.reg .b64 a, b, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmul.rn.f32x2 d, a, b;\nmov.b64 {%0, %1}, d;\n}\n"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+    return d;
 }
 
 struct ScanParams {
@@ -75,11 +102,13 @@ selective_scan_kernel(const ScanParams p) {
     const int tid = threadIdx.x, part = tid % LANES, cl = tid / LANES;
     const int c0 = blockIdx.x * CB, ch = c0 + cl;
     const bool mine = ch < p.channels;
-    float A2[DL], S[DL];                                   // decay rates in units of log2
+    constexpr int DP = DL / 2;                             // a lane's states in pairs
+    float2 A2[DP], S[DP];                                  // decay rates in units of log2
 #pragma unroll
-    for (int i = 0; i < DL; ++i) {
-        const int n = part * DL + i;
-        A2[i] = mine && n < p.N ? -expf(p.A_log[(size_t)ch * p.N + n]) * 1.4426950408889634f : 0.f;
+    for (int i = 0; i < DP; ++i) {
+        const int n = part * DL + 2 * i;
+        A2[i].x = mine && n < p.N ? -expf(p.A_log[(size_t)ch * p.N + n]) * 1.4426950408889634f : 0.f;
+        A2[i].y = mine && n + 1 < p.N ? -expf(p.A_log[(size_t)ch * p.N + n + 1]) * 1.4426950408889634f : 0.f;
     }
     // what a thread prepares of every row: channel `tid % CB` of rows tid / CB, + LANES, ...
     const int pc = tid % CB, pr = tid / CB, pch = c0 + pc;
@@ -89,15 +118,17 @@ selective_scan_kernel(const ScanParams p) {
     const T* z = static_cast<const T*>(p.z);
     const T* bs = static_cast<const T*>(p.b);
     const T* cs = static_cast<const T*>(p.c);
-    float rx[XPT], rd[XPT];
-    float rb[BPT], rc[BPT];
+    // raw values: a conversion next to the load would wait for it
+    const T none = from_f32<T>(0.f);
+    T rx[XPT], rb[BPT], rc[BPT];
+    float rd[XPT];
     auto fetch = [&](int at) {
 #pragma unroll
         for (int k = 0; k < XPT; ++k) {
             const int t = at + pr + k * LANES;
             const bool live = prepares && t < rows;
             const size_t rr = (size_t)(r0 + (live ? t : 0));
-            rx[k] = live ? to_f32(x[rr * p.ldx + pch]) : 0.f;
+            rx[k] = live ? x[rr * p.ldx + pch] : none;
             rd[k] = live ? p.dt_in[rr * p.ldd + pch] : 0.f;
         }
 #pragma unroll
@@ -105,14 +136,17 @@ selective_scan_kernel(const ScanParams p) {
             const int idx = tid + k * SCAN_THREADS, t = at + idx / NP, n = idx % NP;
             const bool live = t < rows && n < p.N;
             const size_t rr = (size_t)(r0 + (live ? t : 0));
-            rb[k] = live ? to_f32(bs[rr * p.ldbc + n]) : 0.f;
-            rc[k] = live ? to_f32(cs[rr * p.ldbc + n]) : 0.f;
+            rb[k] = live ? bs[rr * p.ldbc + n] : none;
+            rc[k] = live ? cs[rr * p.ldbc + n] : none;
         }
     };
     pdl_wait();
     float* S_glob = p.state + (size_t)slot * p.state_stride + (size_t)ch * p.N + part * DL;
 #pragma unroll
-    for (int i = 0; i < DL; ++i) S[i] = mine && part * DL + i < p.N ? S_glob[i] : 0.f;
+    for (int i = 0; i < DP; ++i) {
+        S[i].x = mine && part * DL + 2 * i < p.N ? S_glob[2 * i] : 0.f;
+        S[i].y = mine && part * DL + 2 * i + 1 < p.N ? S_glob[2 * i + 1] : 0.f;
+    }
     fetch(0);
     for (int at = 0; at < rows; at += SCAN_ROWS) {
         const int cnt = min(SCAN_ROWS, rows - at);
@@ -120,50 +154,86 @@ selective_scan_kernel(const ScanParams p) {
         for (int k = 0; k < XPT; ++k) {
             const int t = pr + k * LANES;
             if (k * LANES < cnt) {
-                const float dt = t < cnt ? scan_softplus(rd[k] + bias) : 0.f;      // (a row that does not exist changes nothing)
-                sdt[t][pc] = make_float2(dt, dt * rx[k]);
-                sy[t][pc] = skip * rx[k];
+                const float dt = t < cnt ? scan_softplus<T>(rd[k] + bias) : 0.f;      // (a row that does not exist changes nothing)
+                const float xv = to_f32(rx[k]);
+                sdt[t][pc] = make_float2(dt, dt * xv);
+                sy[t][pc] = skip * xv;
             }
         }
 #pragma unroll
         for (int k = 0; k < BPT; ++k) {
             const int idx = tid + k * SCAN_THREADS;
-            sb[idx / NP][idx % NP] = rb[k];
-            sc[idx / NP][idx % NP] = rc[k];
+            sb[idx / NP][idx % NP] = to_f32(rb[k]);
+            sc[idx / NP][idx % NP] = to_f32(rc[k]);
         }
         __syncthreads();
+        // the gates of this chunk and the raw values of the next one are on their way while this one is walked
+        T rz[XPT];
+#pragma unroll
+        for (int k = 0; k < XPT; ++k) {
+            const int t = pr + k * LANES;
+            rz[k] = prepares && t < cnt ? z[(size_t)(r0 + at + t) * p.ldz + pch] : none;
+        }
         if (at + SCAN_ROWS < rows) fetch(at + SCAN_ROWS);
-#pragma unroll 1
+        // with few lanes the operands of the group after are read from shared memory before this group is walked
+        constexpr bool AHEAD = LANES <= 8;
+        constexpr int AG = AHEAD ? LANES : 1;
+        float2 dn[AG];
+        float2 bn[AG][DP], cn[AG][DP];
+        auto operands = [&](int t, float2& d, float2 (&bv)[DP], float2 (&cv)[DP]) {
+            d = sdt[t][cl];
+            if (DL % 4 == 0) {
+#pragma unroll
+                for (int i = 0; i < DP; i += 2) {
+                    const float4 b4 = *reinterpret_cast<const float4*>(&sb[t][part * DL + 2 * i]);
+                    const float4 c4 = *reinterpret_cast<const float4*>(&sc[t][part * DL + 2 * i]);
+                    bv[i] = make_float2(b4.x, b4.y); bv[(i + 1) % DP] = make_float2(b4.z, b4.w);
+                    cv[i] = make_float2(c4.x, c4.y); cv[(i + 1) % DP] = make_float2(c4.z, c4.w);
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < DP; ++i) {
+                    bv[i] = *reinterpret_cast<const float2*>(&sb[t][part * DL + 2 * i]);
+                    cv[i] = *reinterpret_cast<const float2*>(&sc[t][part * DL + 2 * i]);
+                }
+            }
+        };
+        if (AHEAD) {
+#pragma unroll
+            for (int k = 0; k < AG; ++k) operands(k, dn[k], bn[k], cn[k]);
+        }
+#pragma unroll(AHEAD ? 2 : 1)
         for (int t0 = 0; t0 < cnt; t0 += LANES) {
             float y[LANES];
+            float2 dc[AG];
+            float2 bc[AG][DP], cc[AG][DP];
+            if (AHEAD) {
+#pragma unroll
+                for (int k = 0; k < AG; ++k) {
+                    dc[k] = dn[k];
+#pragma unroll
+                    for (int i = 0; i < DP; ++i) { bc[k][i] = bn[k][i]; cc[k][i] = cn[k][i]; }
+                }
+                const int nx = t0 + LANES < cnt ? t0 + LANES : t0;
+#pragma unroll
+                for (int k = 0; k < AG; ++k) operands(nx + k, dn[k], bn[k], cn[k]);
+            }
 #pragma unroll
             for (int k = 0; k < LANES; ++k) {
-                const float2 d = sdt[t0 + k][cl];
-                float bv[DL], cv[DL];
-                if (DL % 4 == 0) {
+                constexpr int LAST = AG - 1;
+                const int kk = AHEAD ? k : LAST;
+                if (!AHEAD) operands(t0 + k, dc[0], bc[0], cc[0]);
+                const float2 dt2 = make_float2(dc[kk].x, dc[kk].x), dx2 = make_float2(dc[kk].y, dc[kk].y);
+                float2 acc = make_float2(0.f, 0.f);
 #pragma unroll
-                    for (int i = 0; i < DL; i += 4) {
-                        const float4 b4 = *reinterpret_cast<const float4*>(&sb[t0 + k][part * DL + i]);
-                        const float4 c4 = *reinterpret_cast<const float4*>(&sc[t0 + k][part * DL + i]);
-                        bv[i] = b4.x; bv[(i + 1) % DL] = b4.y; bv[(i + 2) % DL] = b4.z; bv[(i + 3) % DL] = b4.w;
-                        cv[i] = c4.x; cv[(i + 1) % DL] = c4.y; cv[(i + 2) % DL] = c4.z; cv[(i + 3) % DL] = c4.w;
-                    }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < DL; i += 2) {
-                        const float2 b2 = *reinterpret_cast<const float2*>(&sb[t0 + k][part * DL + i]);
-                        const float2 c2 = *reinterpret_cast<const float2*>(&sc[t0 + k][part * DL + i]);
-                        bv[i] = b2.x; bv[i + 1] = b2.y;
-                        cv[i] = c2.x; cv[i + 1] = c2.y;
-                    }
+                for (int i = 0; i < DP; ++i) {
+                    float2 a = mul2(dt2, A2[i]);
+                    a.x = scan_exp2<T>(a.x);
+                    a.y = scan_exp2<T>(a.y);
+                    S[i] = fma2(a, S[i], mul2(dx2, bc[kk][i]));
+                    acc = fma2(S[i], cc[kk][i], acc);
                 }
-                float acc = 0.f;
-#pragma unroll
-                for (int i = 0; i < DL; ++i) {
-                    S[i] = fmaf(scan_exp2<T>(d.x * A2[i]), S[i], d.y * bv[i]);
-                    acc = fmaf(S[i], cv[i], acc);
-                }
-                y[k] = acc;
+                y[k] = acc.x + acc.y;
             }
             // lane `part` ends with the sum of row t0 + part: at every step a lane hands the half of its rows that the
             // other lane is to keep over and adds what it gets to its own half
@@ -183,18 +253,16 @@ selective_scan_kernel(const ScanParams p) {
 #pragma unroll
         for (int k = 0; k < XPT; ++k) {
             const int t = pr + k * LANES;
-            if (prepares && t < cnt) {
-                const size_t rr = (size_t)(r0 + at + t);
-                const float zz = to_f32(z[rr * p.ldz + pch]);
-                out[rr * p.ldo + pch] = from_f32<T>(sy[t][pc] * (zz / (1.f + expf(-zz))));
-            }
+            if (prepares && t < cnt) out[(size_t)(r0 + at + t) * p.ldo + pch] = from_f32<T>(sy[t][pc] * scan_silu<T>(to_f32(rz[k])));
         }
         // (the next chunk's sums are written by the threads that read these, its other arrays were read before the barrier)
     }
     if (mine) {
 #pragma unroll
-        for (int i = 0; i < DL; ++i)
-            if (part * DL + i < p.N) S_glob[i] = S[i];
+        for (int i = 0; i < DP; ++i) {
+            if (part * DL + 2 * i < p.N) S_glob[2 * i] = S[i].x;
+            if (part * DL + 2 * i + 1 < p.N) S_glob[2 * i + 1] = S[i].y;
+        }
     }
 }
 

@@ -1021,6 +1021,62 @@ delta_rule_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__ b_in,
     }
 }
 
+// ---- what the walk with a bonus needs besides (DECAY_BONUS: its outputs are no part of the recurrence, so it can walk whole
+// groups of tokens without exchanging anything) ----
+// `COUNT` neighbouring elements as raw 32-bit words, by the widest loads their size allows (the address is a multiple of
+// that size: the launcher checks the rows); a conversion next to the load would wait for it
+template <typename T, int COUNT>
+struct RawRun {
+    static constexpr int BYTES = COUNT * (int)sizeof(T);
+    static constexpr bool WORDS = BYTES % 4 == 0;
+    static constexpr int W = WORDS ? BYTES / 4 : COUNT;
+    unsigned w[W];
+    __device__ __forceinline__ void load(const T* p, bool live) {
+        if constexpr (BYTES % 16 == 0) {
+#pragma unroll
+            for (int i = 0; i < W; i += 4) {
+                const uint4 v = live ? *reinterpret_cast<const uint4*>(reinterpret_cast<const unsigned*>(p) + i) : make_uint4(0u, 0u, 0u, 0u);
+                w[i] = v.x; w[i + 1] = v.y; w[i + 2] = v.z; w[i + 3] = v.w;
+            }
+        } else if constexpr (BYTES % 8 == 0) {
+#pragma unroll
+            for (int i = 0; i < W; i += 2) {
+                const uint2 v = live ? *reinterpret_cast<const uint2*>(reinterpret_cast<const unsigned*>(p) + i) : make_uint2(0u, 0u);
+                w[i] = v.x; w[i + 1] = v.y;
+            }
+        } else if constexpr (WORDS) {
+#pragma unroll
+            for (int i = 0; i < W; ++i) w[i] = live ? reinterpret_cast<const unsigned*>(p)[i] : 0u;
+        } else {
+#pragma unroll
+            for (int i = 0; i < W; ++i) w[i] = live ? (unsigned)reinterpret_cast<const unsigned short*>(p)[i] : 0u;
+        }
+    }
+    __device__ __forceinline__ float at(int i) const {
+        if constexpr (sizeof(T) == 4) return __uint_as_float(w[i]);
+        else if constexpr (!WORDS) return __uint_as_float(w[i] << 16);
+        else return __uint_as_float((i & 1) ? (w[i >> 1] & 0xffff0000u) : (w[i >> 1] << 16));      // bfloat16: the upper half of a float
+    }
+};
+// the decay exp(-exp(x)): the exact functions for 32-bit activations
+template <typename T> __device__ __forceinline__ float double_exp_decay(float x);
+template <> __device__ __forceinline__ float double_exp_decay<float>(float x) { return expf(-expf(x)); }
+template <> __device__ __forceinline__ float double_exp_decay<bf16>(float x) { return __expf(-__expf(x)); }
+// two multiply-adds (multiplications) in one instruction
+__device__ __forceinline__ float2 fma_pair(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("{\n.reg .b64 a, b, c, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmov.b64 c, {%6, %7};\nfma.rn.f32x2 d, a, b, c;\n"
+        "mov.b64 {%0, %1}, d;\n}\n"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+    return d;
+}
+__device__ __forceinline__ float2 mul_pair(float2 a, float2 b) {
+    float2 d;
+    asm("{\n.reg .b64 a, b, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmul.rn.f32x2 d, a, b;\nmov.b64 {%0, %1}, d;\n}\n"
+        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+    return d;
+}
+
 // The same recurrence with more parallelism, for key widths LANES * DL and value widths that are multiples of the
 // columns a CTA takes: LANES lanes share a column of one head's state (lane p keeps the key channels p * DL .. + DL - 1
 // of it in registers) and add their partial sums with shuffles; a CTA takes COLS columns: 32 with four lanes each, or,
@@ -1092,20 +1148,60 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
         for (int i = 0; i < VPT; ++i) rv[i] = live ? to_f32(row[v_off + sub * VPT + i]) : 0.f;
         rb = (live && sub == 0 && MODE == 0) ? to_f32(b_in[rr * ldb + head]) : 0.f;
     };
+    RawRun<T, bonus ? CH : 2> wq, wk, wa;
+    RawRun<T, bonus ? VPT : 2> wv;
+    auto fetch_runs = [&](int c0) {
+        const bool live = c0 + pt < rows;
+        const size_t rr = (size_t)(r0 + (live ? c0 + pt : 0));
+        const T* row = qkv + rr * ld;
+        wq.load(row + q_off + sub * CH, live);
+        wk.load(row + k_off + sub * CH, live);
+        wa.load(a_in + rr * lda + a_at + sub * CH, live);
+        wv.load(row + v_off + sub * VPT, live);
+    };
     float bias[CH], low[CH];
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
         bias[i] = plain ? 0.f : dt_bias[a_at + (sub * CH + i) * a_step];
         low[i] = (forget || bonus) ? A_log[a_at + sub * CH + i] : 0.f;
     }
-    fetch(0);
+    if (bonus) fetch_runs(0); else fetch(0);
     for (int c0 = 0; c0 < rows; c0 += DELTA_CHUNK) {
         const int cnt = min(DELTA_CHUNK, rows - c0);
         __syncthreads();                                // the chunk before is done with the shared arrays
-        {
+        if constexpr (bonus) {
+            float now = 0.f, q[CH], k[CH], g[CH];
+#pragma unroll
+            for (int i = 0; i < CH; ++i) {
+                q[i] = wq.at(i) * q_scale;
+                k[i] = wk.at(i);
+                g[i] = double_exp_decay<T>(wa.at(i) + bias[i]);
+                now = fmaf(q[i] * low[i], k[i], now);
+            }
+#pragma unroll
+            for (int o = 1; o < PT; o <<= 1) now += __shfl_xor_sync(0xffffffffu, now, o);
+            if (CH % 4 == 0 && DL % 4 == 0) {
+#pragma unroll
+                for (int i = 0; i < CH; i += 4) {
+                    const int ch = sub * CH + i, at = ch + (ch / DL) * 4;
+                    *reinterpret_cast<float4*>(&qs[pt][at]) = make_float4(q[i], q[(i + 1) % CH], q[(i + 2) % CH], q[(i + 3) % CH]);
+                    *reinterpret_cast<float4*>(&ks[pt][at]) = make_float4(k[i], k[(i + 1) % CH], k[(i + 2) % CH], k[(i + 3) % CH]);
+                    *reinterpret_cast<float4*>(&gs[pt][at]) = make_float4(g[i], g[(i + 1) % CH], g[(i + 2) % CH], g[(i + 3) % CH]);
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < CH; ++i) {
+                    const int ch = sub * CH + i, at = ch + (ch / DL) * 4;
+                    qs[pt][at] = q[i]; ks[pt][at] = k[i]; gs[pt][at] = g[i];
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < VPT; ++i) vs[pt][sub * VPT + i] = wv.at(i);
+            if (sub == 0) betas[pt] = now;
+        } else {
             float sq = 0.f, sk = 0.f;
 #pragma unroll
-            for (int i = 0; i < CH; ++i) { sq = fmaf(bonus ? rq[i] * low[i] : rq[i], bonus ? rk[i] : rq[i], sq); sk = fmaf(rk[i], rk[i], sk); }
+            for (int i = 0; i < CH; ++i) { sq = fmaf(rq[i], rq[i], sq); sk = fmaf(rk[i], rk[i], sk); }
 #pragma unroll
             for (int o = 1; o < PT; o <<= 1) {
                 sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -1113,7 +1209,7 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
             }
             const float fq = q_scale / sqrtf(sq + unit_eps), fk = 1.f / sqrtf(sk + unit_eps);
             // a decay per head is one number for all of a token's key channels: made once, not once a channel
-            const float g_head = (a_step == 0 && !plain && !forget && !gated && !bonus) ? expf(-decay_rate * softplus_f(ra[0] + bias[0])) : 0.f;
+            const float g_head = (a_step == 0 && !plain && !forget && !gated) ? expf(-decay_rate * softplus_f(ra[0] + bias[0])) : 0.f;
 #pragma unroll
             for (int i = 0; i < CH; ++i) {
                 const int ch = sub * CH + i;
@@ -1123,10 +1219,6 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
                     qs[pt][at] = silu_f(rq[i]);
                     ks[pt][at] = (1.f - low[i]) * open;                          // 1 - f
                     gs[pt][at] = low[i] + (1.f - low[i]) * (1.f - open);         // f
-                } else if (bonus) {
-                    qs[pt][at] = rq[i] * q_scale;
-                    ks[pt][at] = rk[i];
-                    gs[pt][at] = expf(-expf(ra[i] + bias[i]));
                 } else if (gated || stepped) {
                     qs[pt][at] = rq[i] * q_scale;
                     ks[pt][at] = rk[i];
@@ -1139,10 +1231,51 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
             }
 #pragma unroll
             for (int i = 0; i < VPT; ++i) vs[pt][sub * VPT + i] = plain ? silu_f(rv[i]) : rv[i];
-            if (sub == 0) betas[pt] = bonus ? sq * q_scale : stepped ? softplus_f(ra[0] + bias[0]) : 1.f / (1.f + expf(-rb));
+            if (sub == 0) betas[pt] = stepped ? softplus_f(ra[0] + bias[0]) : 1.f / (1.f + expf(-rb));
         }
         __syncthreads();
-        if (c0 + DELTA_CHUNK < rows) fetch(c0 + DELTA_CHUNK);
+        if (c0 + DELTA_CHUNK < rows) {
+            if (bonus) fetch_runs(c0 + DELTA_CHUNK); else fetch(c0 + DELTA_CHUNK);
+        }
+        if constexpr (bonus) {
+            // whole groups of LANES tokens: every lane sums its channels of every token, then the lanes of a column add up
+            // their LANES sums at once, one token a lane (LANES - 1 shuffles); what is left of a chunk goes the usual way below
+            const int groups = cnt / LANES;
+#pragma unroll 1
+            for (int gr = 0; gr < groups; ++gr) {
+                const int t0 = gr * LANES;
+                float y[LANES];
+#pragma unroll
+                for (int k = 0; k < LANES; ++k) {
+                    const float2* kt = reinterpret_cast<const float2*>(&ks[t0 + k][part * QP]);
+                    const float2* qt = reinterpret_cast<const float2*>(&qs[t0 + k][part * QP]);
+                    const float2* gt = reinterpret_cast<const float2*>(&gs[t0 + k][part * QP]);
+                    const float v = vs[t0 + k][col];
+                    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+                    for (int i = 0; i < DL / 2; ++i) {
+                        float2 s2 = make_float2(S[2 * i], S[2 * i + 1]);
+                        acc = fma_pair(s2, qt[i], acc);
+                        s2 = fma_pair(s2, gt[i], mul_pair(kt[i], make_float2(v, v)));
+                        S[2 * i] = s2.x; S[2 * i + 1] = s2.y;
+                    }
+                    y[k] = acc.x + acc.y;
+                }
+#pragma unroll
+                for (int o = LANES / 2; o > 0; o >>= 1) {
+                    const bool upper = (part & o) != 0;
+#pragma unroll
+                    for (int i = 0; i < o; ++i) {
+                        const float give = upper ? y[i] : y[i + o], keep = upper ? y[i + o] : y[i];
+                        y[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                    }
+                }
+                const int t = t0 + part;
+                o_raw[(size_t)(r0 + c0 + t) * nv + head * v_dim + col0 + col] = fmaf(betas[t], vs[t][col], y[0]);
+            }
+            if (groups * LANES == cnt) continue;
+        }
+        const int t_begin = bonus ? cnt / LANES * LANES : 0;
         // With registers to spare (the narrow CTAs) a token's vectors are read from shared memory while the token
         // before is walked, so that the recurrence never waits for them.
         constexpr bool AHEAD = NT <= 128 && LANES >= 8;
@@ -1159,8 +1292,8 @@ delta_rule_split_kernel(const T* __restrict__ qkv, int ld, const T* __restrict__
                 bn = betas[t];
             }
         };
-        ahead(0);
-        for (int t = 0; t < cnt; ++t) {
+        ahead(t_begin);
+        for (int t = t_begin; t < cnt; ++t) {
             float2 kc[DL / 2], qc[DL / 2], gc[DL / 2];
             float vc, bc;
             if (AHEAD) {
@@ -1390,7 +1523,9 @@ static int matrix_state_recurrence(int dtype, const void* qkv, int ld, const voi
         tis_set_error("delta_rule: %d rows in one step (at most 65535)", n);
         return TIS_BAD_SIZE;
     }
-    if (o_raw != nullptr && H > 0 && G > 0 && H % G == 0 && tis_delta_rule_splits(k_dim, v_dim)) {
+    // (the walk with a bonus reads its rows in 16-byte vectors)
+    const bool rows_fit = decay_mode != DECAY_BONUS || (ld % 8 == 0 && lda % 8 == 0 && ((uintptr_t)qkv | (uintptr_t)a_in) % 16 == 0);
+    if (o_raw != nullptr && H > 0 && G > 0 && H % G == 0 && rows_fit && tis_delta_rule_splits(k_dim, v_dim)) {
 #define TIS_DELTA_SPLIT(K, DL, LANES, COLS)                                                                           \
     if (k_dim == K)                                                                                                    \
         TIS_DISPATCH_DTYPE(dtype, T, return (launch_delta_rule_split<T, DL, LANES, COLS>((const T*)qkv, ld,            \

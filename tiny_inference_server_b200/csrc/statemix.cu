@@ -321,6 +321,59 @@ token_shift_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ m
     }
 }
 
+// The same with S known and 16-byte vectors: a CTA takes `rows` rows one after the other, a thread its vector of all of them,
+// with the weights of the mixes and the row before in registers.
+template <typename T, int S>
+__global__ void __launch_bounds__(128)
+token_shift_rows_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ mu, float* __restrict__ state,
+                        size_t state_stride, T* __restrict__ out, const int* __restrict__ row_slot, const int* __restrict__ row_last,
+                        int n, int d, int rows) {
+    constexpr int N = Vec16<T>::N;
+    pdl_launch_dependents();
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * N;
+    if (i >= d) return;
+    float m[S][N];
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(mu + (size_t)s * d + i + j);
+            m[s][j] = v.x; m[s][j + 1] = v.y; m[s][j + 2] = v.z; m[s][j + 3] = v.w;
+        }
+    const int r0 = blockIdx.x * rows, r_end = min(n, r0 + rows);
+    int before_slot = r0 > 0 ? row_slot[r0 - 1] : -1;
+    bool held = false;                                        // `b` holds the row before
+    float b[N];
+    pdl_wait();
+    for (int r = r0; r < r_end; ++r) {
+        const int slot = row_slot[r];
+        const bool first = slot != before_slot;
+        before_slot = slot;
+        if (slot < 0) { held = false; continue; }
+        float h[N];
+        Vec16<T>::load(x + (size_t)r * ldx + i, h);
+        if (first) {
+            float* s = state + (size_t)slot * state_stride + i;
+            float keep[N];
+            Vec16<T>::load(x + (size_t)row_last[r] * ldx + i, keep);
+#pragma unroll
+            for (int j = 0; j < N; ++j) { b[j] = s[j]; s[j] = keep[j]; }
+        } else if (!held) {
+            Vec16<T>::load(x + (size_t)(r - 1) * ldx + i, b);
+        }
+#pragma unroll
+        for (int s = 0; s < S; ++s) {
+            float o[N];
+#pragma unroll
+            for (int j = 0; j < N; ++j) o[j] = fmaf(b[j] - h[j], m[s][j], h[j]);
+            Vec16<T>::store(out + ((size_t)r * S + s) * d + i, o);
+        }
+#pragma unroll
+        for (int j = 0; j < N; ++j) b[j] = h[j];
+        held = true;
+    }
+}
+
 // out = a * sa + b * sb, element by element over n rows of d (row strides free), the sum in 32-bit.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -415,7 +468,13 @@ TIS_API int tis_token_shift(int dtype, const void* x, int ldx, const float* mu, 
     }
     TIS_DISPATCH_DTYPE(dtype, T, {
         constexpr int N = Vec16<T>::N;
-        if (d % N == 0 && ldx % N == 0 && ((uintptr_t)x | (uintptr_t)out) % 16 == 0)
+        if (mixes == 5 && d % N == 0 && ldx % N == 0 && ((uintptr_t)x | (uintptr_t)out | (uintptr_t)mu) % 16 == 0) {
+            // rows a CTA takes: enough CTAs for about eight on every SM
+            const int cols = (d / N + 127) / 128, want = (int)((long long)n * cols / (8 * 148));
+            const int rows = want < 1 ? 1 : (want > 16 ? 16 : want);
+            tis_launch(token_shift_rows_kernel<T, 5>, dim3((n + rows - 1) / rows, cols), dim3(128), 0, stream, (const T*)x, ldx, mu,
+                       state, state_stride, (T*)out, row_slot, row_last, n, d, rows);
+        } else if (d % N == 0 && ldx % N == 0 && ((uintptr_t)x | (uintptr_t)out) % 16 == 0)
             tis_launch(token_shift_kernel<T, N>, dim3(n, (d / N + 127) / 128), dim3(128), 0, stream, (const T*)x, ldx, mu, mixes,
                        state, state_stride, (T*)out, row_slot, row_last, d);
         else
