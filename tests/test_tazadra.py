@@ -142,7 +142,7 @@ def make_tensors(cfg, seed):
         elif leaf == "mix.conv":
             t = rnd / math.sqrt(shape[1])
         elif len(shape) == 2:
-            t = rnd * {"mlp.router": 4.0, "mix.w2": 2.0, "mix.x": 1.5}.get(leaf, 1.0) / math.sqrt(shape[1])
+            t = rnd * {"mlp.router": 2.0}.get(leaf, 1.0) / math.sqrt(shape[1])
         else:
             raise AssertionError(f"no rule for {name} {shape}")
         out[name] = t.to(torch.bfloat16).contiguous()
@@ -161,16 +161,30 @@ def make_folder(raw, seed, folder, rank=8):
 _cache = {}
 
 
-def _setup(name, tmp_path_factory):
-    if name not in _cache:
+def all_chosen(raw):
+    """The configuration with routers that choose every expert.  A choice that hangs on a rounding replaces an expert by another
+    one, and behind the norm of its sublayer, and in the states of the layers above, that stays visible for many tokens: whole
+    models in bfloat16 are compared without choices.  The choice itself is compared in float32, and alone."""
+    raw = json.loads(json.dumps(raw))
+    for layer in raw["layers"]:
+        if layer["mlp"] and layer["mlp"]["kind"] == "moe":
+            layer["mlp"]["router"]["top"] = layer["mlp"]["router"]["experts"]
+    return raw
+
+
+def _setup(name, tmp_path_factory, dtype="float32"):
+    key = name, dtype
+    if key not in _cache:
         raw, page = CONFIGS[name]
+        if dtype == "bfloat16":
+            raw = all_chosen(raw)
         folder = make_folder(raw, 29 + ord(name[-1]), str(tmp_path_factory.mktemp(f"tazadra{name}")), RANKS[name])
         c, W = plain.read_config(folder), plain.read_weights(folder)
         g = torch.Generator().manual_seed(5)
         seqs = {f"r{i}": torch.randint(0, raw["vocab"], (n,), generator=g).tolist() for i, n in enumerate(LENGTHS[name])}
         ref = {rid: plain.plain_forward(c, W, toks).numpy() for rid, toks in seqs.items()}
-        _cache[name] = (raw, page, folder, seqs, ref, c, W)
-    return _cache[name]
+        _cache[key] = (raw, page, folder, seqs, ref, c, W)
+    return _cache[key]
 
 
 def rel_err(got, ref):
@@ -181,12 +195,12 @@ def rel_err(got, ref):
     return float(np.sqrt((d * d).mean()) / max(np.sqrt((r * r).mean()), 1e-9))
 
 
-TOL = {"float32": 1e-4, "bfloat16": 0.06}
-#: The share of positions that may differ by more than the tolerance, and by how much at most: a router whose scores at the
-#: edge of its choice lie within a rounding of each other picks another expert there, and what the expert adds stays in the
-#: states of the layers above for the tokens that follow.
-OUTLIERS = {"float32": 0.01, "bfloat16": 0.15}
-OUTLIER_CAP = {"float32": 1.0, "bfloat16": 1.3}
+TOL = {"float32": 1e-4, "bfloat16": 0.1}
+#: The share of positions that may differ by more than the tolerance, and by how much at most: in float32 a router whose scores
+#: at the edge of its choice lie within a rounding of each other; in bfloat16 positions whose scores or decays are steep, or
+#: whose head reads next to nothing of its state before the norm blows it up (a first token whose bonus nearly cancels).
+OUTLIERS = {"float32": 0.01, "bfloat16": 0.06}
+OUTLIER_CAP = {"float32": 1.0, "bfloat16": 0.9}
 
 
 def _steps(mode, seqs, max_live=4):
@@ -647,11 +661,11 @@ ATTENTION_CASES = [          # heads, kv heads, dim, vdim, rotated, chunk, page,
     (4, 1, 32, 48, None, 33, 16, None, 10.0),
     (20, 1, 16, 16, 8, 50, 16, None, 9.0),
     (12, 1, 80, 80, 8, 64, 16, None, None),
-    (4, 4, 256, 256, 128, 90, 16, None, 9.0),
+    (4, 4, 256, 256, 128, 90, 16, None, 6.0),
     (4, 2, 64, 64, 32, None, 16, (8.0, 1.0, 4.0, 128), 11.0),
     (6, 3, 24, 40, 10, None, 5, None, 5.0),
     (2, 1, 64, 64, 62, 128, 64, None, 12.0),
-    (8, 2, 96, 96, 96, 100, 16, (4.0, 1.0, 4.0, 200), 15.0),
+    (8, 2, 96, 96, 96, 100, 16, (4.0, 1.0, 4.0, 200), 6.5),
 ]
 
 
@@ -1067,7 +1081,7 @@ def test_clamped_unit_without_biases(dtype, n, K, F):
 @pytest.mark.parametrize("name", ["M1", "M2", "M3", "M4"])
 @pytest.mark.parametrize("mode", ["whole", "tail", "chunks", "mixed"])
 def test_replay_gpu(name, mode, dtype, tmp_path, tmp_path_factory):
-    raw, page, folder, seqs, ref, _, _ = _setup(name, tmp_path_factory)
+    raw, page, folder, seqs, ref, _, _ = _setup(name, tmp_path_factory, dtype)
     steps = _steps(mode, seqs, max_live=3)
     runner = _replay_and_compare(raw, page, folder, seqs, ref, steps, str(tmp_path / "out"), dtype, "cuda:0", TOL[dtype], max_live=3,
                                  poison=(mode == "mixed"), shuffle=(mode == "mixed"), outliers=OUTLIERS[dtype], cap=OUTLIER_CAP[dtype])
@@ -1134,6 +1148,8 @@ def test_configurations_drawn_at_random(seed, dtype, tmp_path):
     """Whatever config.json says runs without a change of code: configurations drawn at random, a mixed batch of five
     requests (one of them long) through three slots over shuffled pages."""
     raw, page, rank = random_configuration(seed)
+    if dtype == "bfloat16":
+        raw = all_chosen(raw)
     folder = make_folder(raw, 100 + seed, str(tmp_path / "m"), rank)
     c, W = plain.read_config(folder), plain.read_weights(folder)
     g = torch.Generator().manual_seed(seed)
@@ -1141,14 +1157,14 @@ def test_configurations_drawn_at_random(seed, dtype, tmp_path):
     ref = {rid: plain.plain_forward(c, W, toks).numpy() for rid, toks in seqs.items()}
     steps = trace_tools.trace_mixed(seqs, max_live=3, prefill_sizes=(64, 2, 130, 17))
     _replay_and_compare(raw, page, folder, seqs, ref, steps, str(tmp_path / "out"), dtype, "cuda:0", TOL[dtype], max_live=3,
-                        poison=True, shuffle=True, outliers={"float32": 0.01, "bfloat16": 0.25}[dtype], cap=OUTLIER_CAP[dtype])
+                        poison=True, shuffle=True, outliers=OUTLIERS[dtype], cap=OUTLIER_CAP[dtype])
 
 
 @gpu
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_two_slots_used_again_and_again(dtype, tmp_path, tmp_path_factory):
     """Eight requests through two slots over poisoned pages: a page that a request reads but does not hold shows."""
-    raw, page, folder, seqs, ref, _, _ = _setup("M1", tmp_path_factory)
+    raw, page, folder, seqs, ref, _, _ = _setup("M1", tmp_path_factory, dtype)
     steps = trace_tools.trace_mixed(seqs, max_live=2, prefill_sizes=(2, 7, 3, 2), skip_every=4)
     _replay_and_compare(raw, page, folder, seqs, ref, steps, str(tmp_path / "out"), dtype, "cuda:0", TOL[dtype], max_live=2,
                         poison=True, outliers=OUTLIERS[dtype], cap=OUTLIER_CAP[dtype])
@@ -1159,7 +1175,7 @@ def test_two_slots_used_again_and_again(dtype, tmp_path, tmp_path_factory):
 @pytest.mark.parametrize("name", ["M3", "M4"])
 def test_long_decoding(name, dtype, tmp_path, tmp_path_factory):
     """A short prompt, then 300 tokens one by one, replayed from a graph: every chunk passes over decoded tokens only."""
-    raw, page, folder, _, _, c, W = _setup(name, tmp_path_factory)
+    raw, page, folder, _, _, c, W = _setup(name, tmp_path_factory, dtype)
     g = torch.Generator().manual_seed(9)
     toks = torch.randint(0, raw["vocab"], (305,), generator=g).tolist()
     ref = plain.plain_forward(c, W, toks).numpy()

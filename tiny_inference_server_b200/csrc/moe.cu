@@ -112,7 +112,8 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ wr,
             for (int j = 0; j < (e1 != e0 ? 2 : 1); ++j) {
                 const int e = j == 0 ? e0 : e1;
                 const float s = (score_kind != 0 && e < E) ? z[j] : 1.f / (1.f + expf(-z[j]));
-                if (e < E) { sc[e] = s; pick[e] = s + (corr != nullptr ? corr[e] : 0.f); }
+                // (without a correction the logits choose: the order is the same, and scores that round to one another keep it)
+                if (e < E) { sc[e] = s; pick[e] = corr != nullptr ? s + corr[e] : ((groups == 0 || group_best) ? z[j] : s); }
                 else shared_gate[r] = s;
             }
         }
