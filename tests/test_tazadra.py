@@ -713,7 +713,7 @@ def test_attention_chunks_bounds_and_planted_keys(case, dtype):
     from tiny_inference_server_b200.kernels import ops
     before = dict(ops.calls)
     _check_attention(case, dtype, "cuda:0")
-    if dtype == "bfloat16" and case[2] == case[3] and case[2] % 16 == 0:
+    if dtype == "bfloat16" and case[2] == case[3] and case[2] % 16 == 0 and case[0] // case[1] <= 16:
         assert ops.calls["attn_keys"] > before.get("attn_keys", 0)
         if case[2] in (64, 128):
             assert ops.calls["attn_tc"] > before.get("attn_tc", 0)
