@@ -67,8 +67,6 @@ struct AttnParams {
     const int* tile_row0; const int* tile_rows;
     int H, KVH, G, page_size, window;
     float scale_log2;
-    SoftCap cap;            // bounds the raw scores (k 0: not)
-    const bf16* gate; int ldg;      // (n, H): head h's output times sigmoid(gate[row][h]) (null: none)
     int keys_per_split, num_splits;
     float* part_o; float* part_lse;
     int cluster_merge;      // the splits of a (tile, kv head) are one thread-block cluster and merge through
@@ -77,9 +75,12 @@ struct AttnParams {
     int stages;             // stages of the copy pipeline (2..MAX_STAGES)
     int recv_offset;        // bytes from the start of shared memory to where the cluster's partial results land
     // rotary encoding and cache write done by this kernel (decode rows; see FUSED below)
-    const float* rope_cos; const float* rope_sin;   // [positions][HD/2]
+    union {                 // (a kernel that rotates neither bounds scores nor gates: they share their place)
+        struct { const float* rope_cos; const float* rope_sin; };       // [positions][HD/2]
+        struct { SoftCap cap; const bf16* gate; };  // FUSED_NONE: bounds the raw scores (k 0: not); (n, H), head h's output times
+    };                                              // sigmoid(gate[row][h]) (null: none)
     bf16* plane_w;          // the plane, writable: where the row's key and value go (null: another entry fills it)
-    int rope_rot;           // FUSED_PAIRS: how many elements of a head are rotated (tables [positions][rope_rot / 2]),
+    union { int rope_rot; int ldg; };   // FUSED_PAIRS: how many elements of a head are rotated (tables [positions][rope_rot / 2]),
     int rope_norm; float rope_eps;      // and whether the head is then divided by its root mean square
     const float* sink;      // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     TIS_TIMELINE_MEMBER     // (instrumented builds only; the decode kernel's stamps: 0 entry, 1 before and 2 after the
@@ -214,6 +215,13 @@ __device__ __forceinline__ void add_sink(float& num, float& den, float mt, float
     den = den * f + fast_exp2(s2 - m);
 }
 
+// The first key that the row at `pos` sees: first_key (common.cuh); the kernels that rotate know windows only.
+template <int FUSED>
+__device__ __forceinline__ int range_start(int pos, int window) {
+    if (FUSED == FUSED_NONE) return first_key(pos, window);
+    return (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
+}
+
 // What the gate multiplies head hq's output of a row with.
 __device__ __forceinline__ float head_gate(const AttnParams& p, int row, int hq) {
     return 1.f / (1.f + __expf(-__bfloat162float(p.gate[(size_t)row * p.ldg + hq])));
@@ -328,8 +336,8 @@ __device__ __forceinline__ void merge_barrier_init(unsigned long long* merge_bar
     mbar_arrive_expect_tx(merge_bar, ms.own_blocks ? (int)ms.ns * ms.pairs * (ms.own_blocks * 8 + 2) * 4 : 0);
 }
 
-// SINK: the row's softmax may hold a keyless term (p.sink).
-template <int NR, bool SINK>
+// SINK: the row's softmax may hold a keyless term (p.sink).  GATE: the output may be gated (p.gate).
+template <int NR, bool SINK, bool GATE>
 __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, unsigned char* smem_raw, float* recv,
                                                         unsigned long long* merge_bar, const MergeShape& ms,
                                                         const float (&o)[DTILES][4], const float (&m_run)[2],
@@ -408,7 +416,7 @@ __device__ __forceinline__ void merge_splits_by_pushing(const AttnParams& p, uns
             }
         }
         if (SINK && p.sink != nullptr) add_sink(acc, lsum, mt, p.sink[kvh * G + g]);
-        if (SINK && p.gate != nullptr) acc *= head_gate(p, row0 + r, kvh * G + g);
+        if (GATE && p.gate != nullptr) acc *= head_gate(p, row0 + r, kvh * G + g);
         p.out[(size_t)(row0 + r) * p.out_stride + (size_t)(kvh * G + g) * HD + d] =
             __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
     }
@@ -480,7 +488,7 @@ attn_mma_kernel(const AttnParams p) {
         head[i] = kvh * G + g;
         const int pos = valid[i] ? p.positions[r_idx[i]] : 0;
         hi_row[i] = valid[i] ? pos + 1 : 0;
-        lo_row[i] = valid[i] ? first_key(pos, p.window) : 0;
+        lo_row[i] = valid[i] ? range_start<FUSED>(pos, p.window) : 0;
     }
 
     // key range of the tile and of this split
@@ -489,9 +497,9 @@ attn_mma_kernel(const AttnParams p) {
         slot = p.row_slot[row0 + rows - 1];
         const int pos_first = p.positions[row0 + first], pos_last = p.positions[row0 + rows - 1];
         range_hi = pos_last + 1;
-        range_lo = first_key(pos_first, p.window);
+        range_lo = range_start<FUSED>(pos_first, p.window);
         // the splits share out the keys from the window's first tile on
-        const int base = p.window != 0 ? range_lo / KT * KT : 0;
+        const int base = (FUSED == FUSED_NONE ? p.window != 0 : p.window > 0) ? range_lo / KT * KT : 0;
         range_lo = max(range_lo, base + split * p.keys_per_split);
         range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
@@ -679,7 +687,7 @@ attn_mma_kernel(const AttnParams p) {
                     mma_bf16(s[j + 1], qa[kk], b[2], b[3]);
                 }
             }
-            if (p.cap.k != 0.f) {
+            if (FUSED == FUSED_NONE && p.cap.k != 0.f) {
 #pragma unroll
                 for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -808,7 +816,7 @@ attn_mma_kernel(const AttnParams p) {
     }
 
     if (pushed_merge) {
-        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
+        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES, FUSED == FUSED_NONE>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
     } else if (MODE == MODE_KEYS) {
         // merge the four warps (each saw a quarter of the keys) through shared memory
         __syncthreads();
@@ -845,7 +853,7 @@ attn_mma_kernel(const AttnParams p) {
                 }
             }
             if (FUSED != FUSED_HALVES && p.num_splits == 1 && p.sink != nullptr) add_sink(acc, lt, mt, p.sink[hq]);
-            if (FUSED != FUSED_HALVES && p.num_splits == 1 && p.gate != nullptr) acc *= head_gate(p, row, hq);
+            if (FUSED == FUSED_NONE && p.num_splits == 1 && p.gate != nullptr) acc *= head_gate(p, row, hq);
             const float val = lt > 0.f ? acc / lt : 0.f;
             if (p.num_splits == 1) {
                 p.out[(size_t)row * p.out_stride + (size_t)hq * HD + d] = __float2bfloat16_rn(val);
@@ -1044,7 +1052,7 @@ attn_decode_kernel(const AttnParams p) {
         head[i] = kvh * G + g;
         const int pos = valid[i] ? p.positions[r_idx[i]] : 0;
         hi_row[i] = valid[i] ? pos + 1 : 0;
-        lo_row[i] = valid[i] ? first_key(pos, p.window) : 0;
+        lo_row[i] = valid[i] ? range_start<FUSED>(pos, p.window) : 0;
     }
     int range_lo = 0, range_hi = 0, slot = -1;
     if (first >= 0) {
@@ -1052,9 +1060,9 @@ attn_decode_kernel(const AttnParams p) {
         const int pos_last = pos_last_early;
         const int pos_first = first == rows - 1 ? pos_last : p.positions[row0 + first];
         range_hi = pos_last + 1;
-        range_lo = first_key(pos_first, p.window);
+        range_lo = range_start<FUSED>(pos_first, p.window);
         // the splits share out the keys from the window's first tile on
-        const int base = p.window != 0 ? range_lo / KT * KT : 0;
+        const int base = (FUSED == FUSED_NONE ? p.window != 0 : p.window > 0) ? range_lo / KT * KT : 0;
         range_lo = max(range_lo, base + split * p.keys_per_split);
         range_hi = min(range_hi, base + (split + 1) * p.keys_per_split);
     }
@@ -1224,7 +1232,7 @@ attn_decode_kernel(const AttnParams p) {
                     mma_bf16(s[0], qa[kk], b[0], b[1]);
                     mma_bf16(s[1], qa[kk], b[2], b[3]);
                 }
-                if (p.cap.k != 0.f) {
+                if (FUSED == FUSED_NONE && p.cap.k != 0.f) {
 #pragma unroll
                     for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -1309,7 +1317,7 @@ attn_decode_kernel(const AttnParams p) {
             l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 1);
             l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 2);
         }
-        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
+        merge_splits_by_pushing<NR, FUSED != FUSED_HALVES, FUSED == FUSED_NONE>(p, smem_raw, recv, &merge_bar, ms, o, m_run, l_run, G, row0, kvh);
     }
 }
 
@@ -1412,6 +1420,10 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
         tis_set_error("attention: %d query heads per kv head exceed the %d packed rows of this mode", G, mpack);
         return TIS_BAD_SIZE;
     }
+    if (fused && window < 0) {
+        tis_set_error("attention: the rotary encoding is done inside the kernel with windows only, not with chunks");
+        return TIS_BAD_SIZE;
+    }
     if (gate != nullptr && scratch != nullptr) {
         tis_set_error("attention: key splits that merge through scratch memory take no gate");
         return TIS_BAD_SIZE;
@@ -1441,8 +1453,7 @@ static int attn_launch(int mode, const void* q, int q_stride, void* out, int out
     p.fault = fault;
     p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.rope_rot = rope_rot; p.rope_norm = rope_norm; p.rope_eps = rope_eps;
     p.sink = sink;
-    p.cap = soft_cap(softcap, scale);
-    p.gate = (const bf16*)gate; p.ldg = ldg;
+    if (!fused) { p.cap = soft_cap(softcap, scale); p.gate = (const bf16*)gate; p.ldg = ldg; }
     p.plane_w = (fused && write_kv) ? (bf16*)plane : nullptr;
     TIS_TIMELINE_TAKE(p);
     // decode tiles go to the kernel with a producer warp where its layout allows (page segments: two lanes each)

@@ -18,15 +18,17 @@ namespace cluster_reduce {
 
 constexpr int STRIP = 64;             // columns of a strip
 constexpr int CONSUMERS = 128;        // threads that hold accumulators: four warps, 16 columns each
-// EPI_RELU2 .. EPI_TANH: a store through an activation (the square of relu; gelu in its tanh form; silu; tanh), applied to the
+// EPI_RELU2 .. EPI_SILU: a store through an activation (the square of relu; gelu in its tanh form; silu), EPI_TANH likewise (only
+// in kernels that ask for it: the others keep their code), applied to the
 // 32-bit sum
 enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESIDUAL = 2, EPI_RELU2 = 3, EPI_GELU_TANH = 4, EPI_SILU = 5, EPI_TANH = 6 };
 
+template <bool TANH>
 __device__ __forceinline__ float epilogue_act(float x, int epi) {
     if (epi == EPI_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
     if (epi == EPI_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     if (epi == EPI_SILU) return x / (1.f + expf(-x));
-    if (epi == EPI_TANH) return tanhf(x);
+    if (TANH && epi == EPI_TANH) return tanhf(x);
     return x;
 }
 
@@ -131,7 +133,7 @@ struct RowFactorLoads {
 //   pair: [2][64] floats of shared memory; row_factor: [MT * 16] floats (read when e.in_ss is set);
 //   strip: index of the strip (its first column is strip * 64), strips: strips of the product.
 // FORM: the gating of EPI_SWIGLU is the epilogue's `gate`; else silu, with nothing of the other forms in the kernel.
-template <int MT, bool FORM>
+template <int MT, bool FORM, bool TANH = false>
 __device__ __forceinline__ void push_reduce_store(const float (&acc)[MT][2][4], const Epilogue& e, float* recv,
                                                   unsigned long long* recv_bar, float (*pair)[STRIP],
                                                   const float* row_factor, unsigned rank, unsigned ksplit, int strip,
@@ -221,7 +223,7 @@ __device__ __forceinline__ void push_reduce_store(const float (&acc)[MT][2][4], 
         }
         if (e.epi != EPI_SWIGLU) {                      // a plain store, or one through an activation
             if (valid && strip * STRIP + col < e.N)
-                e.out[(size_t)row * e.ldo + strip * STRIP + col] = __float2bfloat16_rn(epilogue_act(sum, e.epi));
+                e.out[(size_t)row * e.ldo + strip * STRIP + col] = __float2bfloat16_rn(epilogue_act<TANH>(sum, e.epi));
         } else {
             // the strip is [32 gate | 32 up]: out column strip*32 + j = gated(gate_j, up_j)
             pair[half][col] = sum;

@@ -50,13 +50,16 @@ struct GemmParams {
     int kc;                       // rows of K per CTA of a cluster (a multiple of BK)
     int stages;                   // ring length: min(tiles per CTA, MAX_STAGES)
     cluster_reduce::Epilogue e;   // rows, columns, where the result goes
-    // several products in one launch (GROUPED kernels): `groups` equal ones of group_cols columns (a multiple of 64), product
+    TIS_TIMELINE_MEMBER           // (instrumented builds only; stamps: 0 entry, 1 weights ordered, 2 dependency wait over,
+                                  //  3 first tile ready, 4 loop done, 5 cluster barrier passed, 6 stored)
+};
+// What the kernels of several products in one launch get besides: the others keep their parameters, and with them their code.
+struct GroupedParams : GemmParams {
+    // `groups` equal ones of group_cols columns (a multiple of 64), product
     // g of rows x + g * x_group and weights w + g * w_group, and behind them one of rows x + groups * x_group and weights
     // `w_last` (N - groups * group_cols columns, row stride ld_last), whose sums pass the epilogue `last_epi`
     int groups, group_cols; size_t x_group, w_group;
     const bf16* w_last; int ld_last, last_epi;
-    TIS_TIMELINE_MEMBER           // (instrumented builds only; stamps: 0 entry, 1 weights ordered, 2 dependency wait over,
-                                  //  3 first tile ready, 4 loop done, 5 cluster barrier passed, 6 stored)
 };
 
 __device__ __forceinline__ void cp16(void* smem, const void* gmem, int bytes) {
@@ -105,7 +108,7 @@ __device__ __forceinline__ void load_x(bf16* xs, const GemmParams& p, int k0, in
 }
 
 // The parameters of the product that the strip of columns from n0 on belongs to (column numbers stay the whole launch's).
-__device__ __forceinline__ GemmParams product_of(const GemmParams& all, int n0) {
+__device__ __forceinline__ GemmParams product_of(const GroupedParams& all, int n0) {
     GemmParams p = all;
     const int g = min(n0 / all.group_cols, all.groups);
     p.x = all.x + (size_t)g * all.x_group;
@@ -119,9 +122,15 @@ __device__ __forceinline__ GemmParams product_of(const GemmParams& all, int n0) 
     return p;
 }
 
+// GROUPED: the kernel of several products in one launch.  The other takes its parameters as they are.
+template <bool GROUPED> struct ParamsOf { typedef GemmParams type; };
+template <> struct ParamsOf<true> { typedef GroupedParams type; };
+__device__ __forceinline__ const GemmParams& params_of(const GemmParams& p) { return p; }
+__device__ __forceinline__ GemmParams params_of(const GroupedParams& p) { return product_of(p, (int)blockIdx.x * BN); }
+
 template <int MT, bool FORM, bool GROUPED = false>
-__global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams all) {
-    const GemmParams p = GROUPED ? product_of(all, (int)blockIdx.x * BN) : all;
+__global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const typename ParamsOf<GROUPED>::type all) {
+    const GemmParams& p = params_of(all);
     namespace cg = cooperative_groups;
     extern __shared__ __align__(16) unsigned char smem[];
     constexpr int W_ELEMS = BK * WROW, X_ELEMS = MT * 16 * XROW;
@@ -251,7 +260,7 @@ __global__ void __launch_bounds__(NTH) gemm_skinny_kernel(const GemmParams all) 
     __syncthreads();                    // row_factor is written (also when this CTA had no tile)
     cluster_reduce::cluster_wait();     // every CTA of the cluster has initialised its barrier
     TIS_STAMP(p, 5);
-    cluster_reduce::push_reduce_store<MT, FORM>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
+    cluster_reduce::push_reduce_store<MT, FORM, GROUPED>(acc, p.e, recv, &recv_bar, pair, row_factor, rank, ksplit, blockIdx.x,
                                           gridDim.x, tid);
     TIS_STAMP(p, 6);
 }
@@ -284,7 +293,7 @@ TIS_API int tis_gemm_skinny_fused(const void* x, int ldx, const void* w, int ldw
         tis_set_error("gemm_skinny: ksplit %d must be 1, 2, 4 or 8", ksplit);
         return TIS_BAD_SIZE;
     }
-    if (epi < EPI_STORE || epi > EPI_TANH) {
+    if (epi < EPI_STORE || epi > EPI_SILU) {
         tis_set_error("gemm_skinny: unknown epilogue %d", epi);
         return TIS_BAD_SIZE;
     }
@@ -376,7 +385,7 @@ TIS_API int tis_gemm_skinny_groups(const void* x, int ldx, size_t x_group, const
         return TIS_BAD_SIZE;
     }
     const int N = groups * group_cols + n_last;
-    GemmParams p = {};
+    GroupedParams p = {};
     p.x = (const bf16*)x; p.ldx = ldx; p.w = (const bf16*)w; p.ldw = group_cols; p.K = K;
     p.e.out = (bf16*)out; p.e.ldo = ldo; p.e.M = M; p.e.N = N; p.e.epi = EPI_STORE; p.e.fault = fault;
     p.e.in_factor = norm_factor(0, 0, 0.f);

@@ -116,7 +116,9 @@ SKINNY_SWIGLU_MAX_ROWS = int(os.environ.get("TIS_SKINNY_SWIGLU_MAX_ROWS", "16"))
 SWAP_SWIGLU_MAX_ROWS = int(os.environ.get("TIS_SWAP_SWIGLU_MAX_ROWS", "32"))
 EPI_STORE, EPI_SWIGLU, EPI_RESIDUAL = 0, 1, 2
 #: a store through an activation, by the activation's name (the weight-streaming products)
-EPI_ACT = {"relu2": 3, "gelu_tanh": 4, "silu": 5, "tanh": 6}
+EPI_ACT = {"relu2": 3, "gelu_tanh": 4, "silu": 5}
+#: the last of several products in one launch (``gemm_side_by_side``) may also pass tanh
+EPI_GROUP_ACT = dict(EPI_ACT, tanh=6)
 #: the norm between two weight-streaming products is folded into them (``ResidualSink`` / ``ScaledRows``);
 #: TIS_FUSED_NORM=0 keeps the norm kernel
 FUSED_NORM = os.environ.get("TIS_FUSED_NORM", "1") != "0"
@@ -498,8 +500,8 @@ def gemm(a, w: torch.Tensor, out: Optional[torch.Tensor] = None, sink: Optional[
             raise KernelError("gemm: an activation and a sink do not go together")
         rows = a.rows if isinstance(a, ScaledRows) else a
         streams = _stream_pays(rows.shape[0], rows.shape[1], w.shape[1]) and rows.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
-        if (_skinny_ok(rows, w) and (streams or _ring_tiles(w.shape[1], rows.shape[1]) <= RING_MAX_TILES)) or \
-                (_skinny_ok(rows, w, STREAM_MAX_ROWS) and streams):
+        if act in EPI_ACT and ((_skinny_ok(rows, w) and (streams or _ring_tiles(w.shape[1], rows.shape[1]) <= RING_MAX_TILES)) or
+                               (_skinny_ok(rows, w, STREAM_MAX_ROWS) and streams)):
             return gemm_skinny(a, w, out, act=act)
         h = gemm(a, w, out)
         return activation(h, h, act)
@@ -771,8 +773,8 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, plane: torch.Tensor, blo
     window = _window_code(window, chunked)
     cap = float(softcap or 0.0)
     ldg = gate.stride(0) if gate is not None else 0
-    if rotary is not None and (cap or gate is not None):
-        raise KernelError("paged_attention: bounded scores and gates go with rows that are rotated already")
+    if rotary is not None and (cap or gate is not None or window < 0):
+        raise KernelError("paged_attention: chunks, bounded scores and gates go with rows that are rotated already")
     scale = 1.0 / math.sqrt(head_dim) if scale is None else float(scale)
     if not scale > 0:
         raise KernelError(f"paged_attention: the scores are multiplied by a positive number, not {scale}")
@@ -1339,7 +1341,7 @@ def gemm_side_by_side(a: torch.Tensor, w: torch.Tensor, w_last: torch.Tensor, ac
         out = torch.empty((n, total), dtype=a.dtype, device=a.device)
         calls["gemm_skinny_groups"] += 1
         _check(lib.tis_gemm_skinny_groups(_p(a), a.stride(0), ctypes.c_size_t(a.stride(1)), _p(w), groups, cols, _p(w_last), last,
-                                          EPI_ACT[act] if act is not None else EPI_STORE, _p(out), out.stride(0), n, k,
+                                          EPI_GROUP_ACT[act] if act is not None else EPI_STORE, _p(out), out.stride(0), n, k,
                                           _ksplit(total, k), _p(tc_fault()), _stream()), lib)
         return out[:, :groups * cols], out[:, groups * cols:]
     out = torch.empty((n, groups * cols), dtype=a.dtype, device=a.device)

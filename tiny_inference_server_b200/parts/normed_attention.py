@@ -137,7 +137,7 @@ class NormedRotaryAttention(Mixer):
         cos, sin, interleaved = (pos.cos, pos.sin, pos.interleaved) if pos is not None else (None, None, True)
         out = torch.empty((n, self.no), dtype=x.dtype, device=x.device)
         gate = proj[:, self.gate_at:self.gate_at + self.num_heads] if self.head_gate else None
-        in_kernel = self.paged and interleaved and not self.whole_norm and not self.softcap and gate is None and ops.rotary_fusable(proj, step, self.num_heads, self.kv_heads, self.dim, pairs=True)
+        in_kernel = self.paged and interleaved and not self.whole_norm and not self.softcap and not self.chunked and gate is None and ops.rotary_fusable(proj, step, self.num_heads, self.kv_heads, self.dim, pairs=True)
         if not in_kernel:
             ops.rotate_norm_store(proj, self.num_heads, 0 if self.reads_cache else self.kv_heads, self.dim, self.v_dim, cos, sin,
                                   interleaved, self.qk_norm, self.eps, binding.k_pages, binding.v_pages, table, step.positions,
