@@ -200,7 +200,8 @@ __device__ __forceinline__ float unit_act(float x, int kind) {
     return x / (1.f + expf(-x));
 }
 
-template <typename T>
+// WEIGH: the units' inputs are weighed (in_weights, n * top).
+template <typename T, bool WEIGH>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ chosen, const T* __restrict__ w_gu,
                    T* __restrict__ hidden, int d, int top, int E, int F, int act, GateForm gate,
@@ -218,7 +219,7 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
     const T* wg = w_gu + (size_t)e * (act >= 0 ? 1 : 2) * F * d;
     const T* wu = wg + (size_t)F * d;
     // a weight on the unit's input multiplies both projections of it
-    const float iw = in_weights != nullptr ? in_weights[pair] : 1.f;
+    const float iw = WEIGH ? in_weights[pair] : 1.f;
     const int j_end = min(F, (int)(blockIdx.y + 1) * MOE_COLS);
     if (act >= 0) {                                        // no gate: two columns are two dot products
         for (int j = blockIdx.y * MOE_COLS + 2 * warp; j < j_end; j += 2 * nw) {
@@ -252,7 +253,8 @@ moe_gate_up_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ cho
 // out[r][c] = sum_k weights[r][k] * (Wd[e_k][c] . hidden[r * top + k])  (+ shared_gate[r] * shared[r][c]);  weights null: 1;
 // w_down (E, d, F).  A CTA per (row, block of COLS output columns).
 // ------------------------------------------------------------------------------------------------------------
-template <typename T>
+// WEIGHTS: the sum is a weighted one.
+template <typename T, bool WEIGHTS>
 __global__ void __launch_bounds__(MOE_THREADS)
 moe_down_kernel(const T* __restrict__ hidden, const int* __restrict__ chosen, const float* __restrict__ weights,
                 const T* __restrict__ w_down, const T* __restrict__ shared, int lds,
@@ -278,7 +280,7 @@ moe_down_kernel(const T* __restrict__ hidden, const int* __restrict__ chosen, co
             for (int j = 0; j < 4; ++j) {
                 const int k = min(k0 + j, top - 1);
                 int e = chosen[(size_t)r * top + k];
-                wt[j] = (k0 + j < top && e >= 0 && e < E) ? (weights != nullptr ? weights[(size_t)r * top + k] : 1.f) : 0.f;
+                wt[j] = (k0 + j < top && e >= 0 && e < E) ? (WEIGHTS ? weights[(size_t)r * top + k] : 1.f) : 0.f;
                 e = min(max(e, 0), E - 1);
                 w[j] = w_down + ((size_t)e * d + c) * F;
                 x4[j] = smem + (size_t)k * F;
@@ -337,9 +339,10 @@ TIS_API int tis_moe_gate_up(int dtype, const void* x, int ldx, const int* chosen
     }
     const size_t smem = sizeof(float) * (size_t)d;
     TIS_DISPATCH_DTYPE(dtype, T, {
-        const int st = set_smem(moe_gate_up_kernel<T>, smem, "moe_gate_up");
+        auto kernel = in_weights != nullptr ? moe_gate_up_kernel<T, true> : moe_gate_up_kernel<T, false>;
+        const int st = set_smem(kernel, smem, "moe_gate_up");
         if (st != TIS_OK) return st;
-        tis_launch(moe_gate_up_kernel<T>, dim3(n * top, (F + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
+        tis_launch(kernel, dim3(n * top, (F + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
                    (const T*)x, ldx, chosen, (const T*)w_gu, (T*)hidden, d, top, E, F, act, gate, in_weights);
     });
     return tis_check_launch("moe_gate_up");
@@ -355,9 +358,10 @@ TIS_API int tis_moe_down(int dtype, const void* hidden, const int* chosen, const
     }
     const size_t smem = sizeof(float) * (size_t)top * F;
     TIS_DISPATCH_DTYPE(dtype, T, {
-        const int st = set_smem(moe_down_kernel<T>, smem, "moe_down");
+        auto kernel = weights != nullptr ? moe_down_kernel<T, true> : moe_down_kernel<T, false>;
+        const int st = set_smem(kernel, smem, "moe_down");
         if (st != TIS_OK) return st;
-        tis_launch(moe_down_kernel<T>, dim3(n, (d + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
+        tis_launch(kernel, dim3(n, (d + MOE_COLS - 1) / MOE_COLS), dim3(MOE_THREADS), smem, stream,
                    (const T*)hidden, chosen, weights, (const T*)w_down, (const T*)shared, lds, shared_gate, (T*)out, d, top,
                    E, F);
     });

@@ -68,8 +68,10 @@ struct Params {
     const int* tile_row0; const int* tile_rows;
     int H, G, page_size, window;
     float scale;
-    SoftCap cap;             // bounds the raw scores (k 0: not)
-    const float* r1; const float* r2;
+    union {                  // (bounded scores have no bias: the two share their place)
+        struct { const float* r1; const float* r2; };
+        SoftCap cap;         // MORE: bounds the raw scores (k 0: not)
+    };
     const float* sink;       // per query head: exp(sink) is one more term of the softmax's denominator (null: none)
     int v_row;               // elements from one value row of a page to the next (VD, or more when the rows are slices)
     int* fault;
@@ -107,6 +109,9 @@ __device__ __forceinline__ void load_tile(const Params& p, int slot, int kvh, in
     }
 }
 
+// MORE: scores may be bounded and the keys may be those of a chunk (and there is no bias); the other kernel knows windows and
+// biases only and keeps its code.
+template <bool MORE>
 __global__ void __launch_bounds__(THREADS, MIN_CTAS)
 window_attention_mma_kernel(const Params p) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -127,7 +132,7 @@ window_attention_mma_kernel(const Params p) {
     const int g = lane >> 2, t4 = lane & 3;
     if (tid == 0) bad = 0;
     const int last = pos0 + nrows - 1;                         // the last key any row of the tile sees
-    const int first = first_key(pos0, p.window);
+    const int first = MORE ? first_key(pos0, p.window) : (p.window > 0 ? max(0, pos0 - p.window + 1) : 0);
     int ntiles = (last - first) / KEYS + 1;
     int kt_begin = 0;
     const int splits = gridDim.z;
@@ -145,7 +150,7 @@ window_attention_mma_kernel(const Params p) {
     const int pos_a = pos0 + m_a / gq, pos_b = pos0 + m_b / gq;
     const int head_a = kvh * gq + m_a % gq, head_b = kvh * gq + m_b % gq;
     float b1_a = 0.f, b2_a = 0.f, b1_b = 0.f, b2_b = 0.f;
-    if (p.r1 != nullptr) {
+    if (!MORE && p.r1 != nullptr) {
         if (row_a) { b1_a = p.r1[head_a]; b2_a = p.r2[head_a]; }
         if (row_b) { b1_b = p.r1[head_b]; b2_b = p.r2[head_b]; }
     }
@@ -180,8 +185,8 @@ window_attention_mma_kernel(const Params p) {
     }
     // positions of the first and last row among this warp's packed rows
     const int w_lo = pos0 + base / gq, w_hi = min(pos0 + (base + 15) / gq, last);
-    const int w_lo_first = first_key(w_lo, p.window), w_hi_first = first_key(w_hi, p.window);
-    const int lo_a = first_key(pos_a, p.window), lo_b = first_key(pos_b, p.window);
+    const int w_lo_first = MORE ? first_key(w_lo, p.window) : 0, w_hi_first = MORE ? first_key(w_hi, p.window) : 0;
+    const int lo_a = MORE ? first_key(pos_a, p.window) : 0, lo_b = MORE ? first_key(pos_b, p.window) : 0;
     for (int kt = kt_begin; kt < ntiles; ++kt) {
         const int stage = (kt - kt_begin) & 1;
         if (kt + 1 < ntiles)
@@ -193,7 +198,8 @@ window_attention_mma_kernel(const Params p) {
         const bf16* vs = vbuf + stage * KEYS * VS;
         const int j0 = first + kt * KEYS;
         // does this warp see any key of the tile?
-        bool any = base < packed && j0 <= w_hi && j0 + KEYS - 1 >= w_lo_first;
+        bool any = base < packed && j0 <= w_hi &&
+                   (MORE ? j0 + KEYS - 1 >= w_lo_first : (p.window <= 0 || j0 + KEYS - 1 > w_lo - p.window));
         if (split_keys) any = any && (kt & 3) == warp;
         if (any) {
             float s[KEYS / 8][4];
@@ -211,8 +217,9 @@ window_attention_mma_kernel(const Params p) {
             }
             // scale, bias, mask; the maximum of each row over the tile.  A tile that every row of the warp sees
             // whole (the usual case inside a window) needs no mask.
-            const bool whole = base + 15 < packed && j0 + KEYS - 1 <= w_lo && j0 >= w_hi_first;
-            if (p.cap.k != 0.f) {
+            const bool whole = base + 15 < packed && j0 + KEYS - 1 <= w_lo &&
+                               (MORE ? j0 >= w_hi_first : (p.window <= 0 || j0 > w_hi - p.window));
+            if (MORE && p.cap.k != 0.f) {
 #pragma unroll
                 for (int n = 0; n < KEYS / 8; ++n)
 #pragma unroll
@@ -226,7 +233,7 @@ window_attention_mma_kernel(const Params p) {
                     for (int e = 0; e < 4; ++e) {
                         const int j = j0 + n * 8 + 2 * t4 + (e & 1);
                         const int pos = (e & 2) ? pos_b : pos_a;
-                        const float v = s[n][e] * p.scale - ((e & 2) ? b1_b : b1_a) * __logf(fmaf((e & 2) ? b2_b : b2_a, (float)(pos - j), 1.f));
+                        const float v = MORE ? s[n][e] * p.scale : s[n][e] * p.scale - ((e & 2) ? b1_b : b1_a) * __logf(fmaf((e & 2) ? b2_b : b2_a, (float)(pos - j), 1.f));
                         s[n][e] = v;
                         mx[e >> 1] = fmaxf(mx[e >> 1], v);
                     }
@@ -238,9 +245,10 @@ window_attention_mma_kernel(const Params p) {
                     for (int e = 0; e < 4; ++e) {
                         const int j = j0 + n * 8 + 2 * t4 + (e & 1);
                         const int pos = (e & 2) ? pos_b : pos_a;
-                        const bool ok = ((e & 2) ? row_b : row_a) && j <= pos && j >= ((e & 2) ? lo_b : lo_a);
+                        const bool ok = ((e & 2) ? row_b : row_a) && j <= pos &&
+                                        (MORE ? j >= ((e & 2) ? lo_b : lo_a) : (p.window <= 0 || j > pos - p.window));
                         float v = -INFINITY;
-                        if (ok) v = s[n][e] * p.scale - ((e & 2) ? b1_b : b1_a) * __logf(fmaf((e & 2) ? b2_b : b2_a, (float)(pos - j), 1.f));
+                        if (ok) v = MORE ? s[n][e] * p.scale : s[n][e] * p.scale - ((e & 2) ? b1_b : b1_a) * __logf(fmaf((e & 2) ? b2_b : b2_a, (float)(pos - j), 1.f));
                         s[n][e] = v;
                         mx[e >> 1] = fmaxf(mx[e >> 1], v);
                     }
@@ -453,6 +461,10 @@ TIS_API int tis_window_attention_mma(const void* q, int ldq, const void* gate, i
                                      const float* r2, int splits, float* partial, const float* sink, int v_row,
                                      int gate_per_head, int* fault, cudaStream_t stream) {
     if (num_tiles <= 0) return TIS_OK;
+    if (r1 != nullptr && (softcap > 0.f || window < 0)) {
+        tis_set_error("window_attention_mma: a bias goes with windows and unbounded scores only");
+        return TIS_BAD_SIZE;
+    }
     if (splits < 1 || splits > 64 || (splits > 1 && partial == nullptr)) {
         tis_set_error("window_attention_mma: %d key splits%s", splits, splits > 1 ? " without scratch" : "");
         return TIS_BAD_SIZE;
@@ -474,14 +486,20 @@ TIS_API int tis_window_attention_mma(const void* q, int ldq, const void* gate, i
     p.v_pages = (const bf16*)v_pages; p.v_page_stride = v_page_stride; p.v_head_stride = v_head_stride;
     p.block_table = block_table; p.bt_stride = bt_stride; p.num_pages = num_pages;
     p.positions = positions; p.row_slot = row_slot; p.tile_row0 = tile_row0; p.tile_rows = tile_rows;
-    p.H = H; p.G = G; p.page_size = page_size; p.window = window; p.scale = scale; p.cap = soft_cap(softcap, scale); p.r1 = r1; p.r2 = r2; p.fault = fault; p.partial = partial; p.sink = sink; p.v_row = v_row;
+    p.H = H; p.G = G; p.page_size = page_size; p.window = window; p.scale = scale;
+    const bool more = softcap > 0.f || window < 0;
+    if (more) p.cap = soft_cap(softcap, scale);
+    else { p.r1 = r1; p.r2 = r2; }
+    p.fault = fault; p.partial = partial; p.sink = sink; p.v_row = v_row;
     const size_t smem = sizeof(bf16) * ((size_t)2 * KEYS * KS + 2 * KEYS * VS);
     static bool attr_set = false;
     if (!attr_set && smem > 48 * 1024) {
-        cudaFuncSetAttribute(window_attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(window_attention_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(window_attention_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         attr_set = true;
     }
-    tis_launch(window_attention_mma_kernel, dim3(num_tiles, G, splits), dim3(THREADS), smem, stream, p);
+    if (more) tis_launch(window_attention_mma_kernel<true>, dim3(num_tiles, G, splits), dim3(THREADS), smem, stream, p);
+    else tis_launch(window_attention_mma_kernel<false>, dim3(num_tiles, G, splits), dim3(THREADS), smem, stream, p);
     int st = tis_check_launch("window_attention_mma");
     if (st != TIS_OK || splits == 1) return st;
     // a step whose keys are split holds one row a tile: H / G packed rows
