@@ -195,7 +195,8 @@ def rel_err(got, ref):
     return float(np.sqrt((d * d).mean()) / max(np.sqrt((r * r).mean()), 1e-9))
 
 
-TOL = {"float32": 1e-4, "bfloat16": 0.1}
+#: (in float32 most positions agree to 1e-6; early tokens whose head outputs nearly cancel before the norm, to 2e-4)
+TOL = {"float32": 3e-4, "bfloat16": 0.1}
 #: The share of positions that may differ by more than the tolerance, and by how much at most: in float32 a router whose scores
 #: at the edge of its choice lie within a rounding of each other; in bfloat16 positions whose scores or decays are steep, or
 #: whose head reads next to nothing of its state before the norm blows it up (a first token whose bonus nearly cancels).
